@@ -13,6 +13,8 @@ A ``ModelSpec`` is plain data.  An architecture's config parser (for example
   layer may be named twice (shared weights; each run gets a cache of its own), and an
   entry may set ``cache_of`` to the index of an earlier *entry* to read that entry's
   cache instead of writing one.
+* ``ScheduleEntry.ahead`` names a *stream step* (``ModelSpec.stream_steps``) that is taken on the stream right before
+  the entry's layer, and the number it is given: a loop of layers begins each pass with one.
 """
 from __future__ import annotations
 
@@ -57,10 +59,12 @@ class LayerSpec:
 
 @dataclass(frozen=True)
 class ScheduleEntry:
-    """One run of ``layers[layer]``; ``cache_of`` names an earlier entry whose cache is read."""
+    """One run of ``layers[layer]``; ``cache_of`` names an earlier entry whose cache is read; ``ahead`` a stream
+    step taken before the layer, with the number it is given."""
 
     layer: int
     cache_of: int | None = None
+    ahead: tuple[str, int] | None = None
 
 
 @dataclass(frozen=True)
@@ -78,8 +82,10 @@ class ModelSpec:
     max_position_embeddings: int
     eos_token_ids: tuple[int, ...] = ()
     stored_dtype: str | None = None
+    stream_steps: Mapping[str, PartSpec] = field(default_factory=dict)
 
     def __post_init__(self) -> None:
+        object.__setattr__(self, "stream_steps", MappingProxyType(dict(self.stream_steps)))
         if not self.layers:
             raise ValueError("a model needs at least one layer")
         if not self.schedule:
@@ -90,6 +96,8 @@ class ModelSpec:
                     f"schedule[{index}] names layer {entry.layer}, "
                     f"but the model has {len(self.layers)} layers"
                 )
+            if entry.ahead is not None and entry.ahead[0] not in self.stream_steps:
+                raise ValueError(f"schedule[{index}] is begun by {entry.ahead[0]!r}, which is no stream step of the model")
             if entry.cache_of is not None:
                 if not 0 <= entry.cache_of < index:
                     raise ValueError(
@@ -107,4 +115,16 @@ def default_schedule(num_layers: int) -> tuple[ScheduleEntry, ...]:
     return tuple(ScheduleEntry(layer=i) for i in range(num_layers))
 
 
-__all__ = ["LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "default_schedule"]
+def looped_schedule(num_layers: int, start: int, stop: int, times: int, step: str | None = None) -> tuple[ScheduleEntry, ...]:
+    """Layers in order, those of ``[start, stop)`` ``times`` times in a row, each run with a cache of its own;
+    ``step``: the stream step that begins every pass, given the pass's number."""
+    if not 0 <= start < stop <= num_layers or times < 1:
+        raise ValueError(f"a loop over layers [{start}, {stop}) of {num_layers}, {times} times, is none")
+    entries = [ScheduleEntry(layer=i) for i in range(start)]
+    for number in range(times):
+        entries += [ScheduleEntry(layer=i, ahead=(step, number) if step is not None and i == start else None)
+                    for i in range(start, stop)]
+    return tuple(entries + [ScheduleEntry(layer=i) for i in range(stop, num_layers)])
+
+
+__all__ = ["LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "default_schedule", "looped_schedule"]

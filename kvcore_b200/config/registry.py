@@ -124,6 +124,9 @@ def _register_stock_architectures() -> None:
     from .rubuvik import ARCHITECTURE as RUBUVIK, RubuvikConfig
 
     register_architecture(RUBUVIK, lambda raw: RubuvikConfig.from_dict(raw).to_model_spec())
+    from .mamevik import ARCHITECTURE as MAMEVIK, MamevikConfig
+
+    register_architecture(MAMEVIK, lambda raw: MamevikConfig.from_dict(raw).to_model_spec())
 
 
 _register_stock_architectures()

@@ -173,6 +173,12 @@ struct KvbTrace {
 #define KVB_TAG_GELU_MUL 45
 #define KVB_TAG_LIGHTNING_PREPARE 46
 #define KVB_TAG_LIGHTNING_SCAN 47
+#define KVB_TAG_SSM_SCAN 48
+#define KVB_TAG_SSM_PREPARE 49
+#define KVB_TAG_GROUP_NORM 50
+#define KVB_TAG_ADD_ROWS 51
+#define KVB_TAG_EMBED_PAIRS 52
+#define KVB_TAG_SOFTCAP 53
 
 // 1 when launches should carry the programmatic-serialization attribute (set by the host side).
 extern "C" int kvb_pdl_enabled();

@@ -8,7 +8,8 @@
 //   [rank | rot].  The query rows [heads, width + rot] get the same turn on their last `rot` entries,
 //   written behind the `rank` entries of the attention's query rows [heads, rank + rot]; the first
 //   `rank` entries of those rows (the query carried into the latent space) are copied from `q_latent`
-//   when given, else left as the caller filled them.
+//   when given, else left as the caller filled them.  (A mixer without position entries whose queries need
+//   nothing done calls it for the cached rows alone.)
 //
 //   head_norm_kv_write (attention with several score maps a head).  q and k are cut into vectors of
 //   `dim` entries (one per head and map); each gets an RMS norm of its own with one weight shared by
@@ -129,7 +130,8 @@ extern "C" int kvb_latent_prepare(const void* kv_rows, long long kv_stride, cons
                                   long long ql_head_stride, void* q_out, int tokens, int heads, int rank, int rot,
                                   int lead, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
-  KVB_REQUIRE(rank > 0 && rot >= 0 && heads > 0 && heads < 65535 && dims >= 0 && dims <= rot && dims % 2 == 0 &&
+  // no heads: only the cached rows are written
+  KVB_REQUIRE(rank > 0 && rot >= 0 && heads >= 0 && heads < 65535 && dims >= 0 && dims <= rot && dims % 2 == 0 &&
               lead > 0, "latent_prepare: bad sizes");
   int* status = kvb_status_word();
   KVB_REQUIRE(status != nullptr, "latent_prepare: no status word");

@@ -3,7 +3,8 @@
 //
 //   route:   z = W_router x in 32-bit (one warp per expert row, lane-strided k in a fixed order, butterfly sum);
 //            scores = sigmoid(z) or softmax(z); the `top` largest (lowest index among equals); weights are
-//            the chosen scores, optionally divided by their sum.  Optionally the choice goes by
+//            the chosen scores, optionally divided by their sum.  A third way scores with z itself and weights the
+//            chosen experts by the softmax over their logits alone.  Optionally z has a bias, the choice goes by
 //            score + correction[e] (the weights stay the scores), only experts of the `keep` best of `groups`
 //            equal groups of neighbouring experts can be chosen (a group's score: its largest choice score),
 //            and the weights are multiplied by a constant.  Extra rows (a shared expert's gate) are
@@ -16,7 +17,8 @@
 //            products in ascending k, so a pair's result depends on nothing else in the batch.
 //            a(p, k) = A[p / a_row_div, k] (* pair weight, rounded to the storage type): the weight
 //            multiplies the expert's INPUT.  GATED: w holds gate rows [0, N) and up rows [N, 2N) and
-//            out = silu(gate) * up.
+//            out = silu(gate) * up, or with g = min(gate, limit), u = clamp(up, -limit, limit):
+//            out = g * sigmoid(alpha g) * (u + shift).
 //   gemv:    the same two products for a handful of pairs in bf16, bound by the bytes of the chosen
 //            experts' matrices (no padded tiles).
 //   gather:  the pairs' input rows expert by expert at a common stride, for one batched library product
@@ -39,7 +41,8 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS)
 moe_route_kernel(int* __restrict__ ids_out, float* __restrict__ weights_out, float* __restrict__ gate_out,
                  const T* __restrict__ x, long long x_stride, const float* __restrict__ router,
                  const float* __restrict__ gate_rows, int tokens, int E, int R, int K, int top, int score_mode,
-                 int renormalize, const float* __restrict__ correction, int groups, int keep, float weight_scale) {
+                 int renormalize, const float* __restrict__ correction, int groups, int keep, float weight_scale,
+                 const float* __restrict__ bias) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_MOE_ROUTE);
   extern __shared__ __align__(16) unsigned char route_smem[];
   T* xs = reinterpret_cast<T*>(route_smem);                                   // [TPB][K]
@@ -90,9 +93,11 @@ moe_route_kernel(int* __restrict__ ids_out, float* __restrict__ weights_out, flo
   const int token = token0 + warp;                    // warp t finishes token t of the block
   float* sc = scores + warp * (E + R);
   for (int r = lane; r < R; r += 32) gate_out[(size_t)token * R + r] = 1.0f / (1.0f + expf(-sc[E + r]));
+  if (bias != nullptr)
+    for (int e = lane; e < E; e += 32) sc[e] += bias[e];
   if (score_mode == 0) {
     for (int e = lane; e < E; e += 32) sc[e] = 1.0f / (1.0f + expf(-sc[e]));
-  } else {
+  } else if (score_mode == 1) {
     float m = -INFINITY;
     for (int e = lane; e < E; e += 32) m = fmaxf(m, sc[e]);
     m = warp_max(m);
@@ -143,11 +148,15 @@ moe_route_kernel(int* __restrict__ ids_out, float* __restrict__ weights_out, flo
       if (kept[e / per] == 0.0f) ch[e] = -INFINITY;
     __syncwarp();
   }
-  float chosen_sum = 0.0f;
+  float chosen_sum = 0.0f, first_logit = 0.0f;
   for (int slot = 0; slot < top; ++slot) {
     float best; int best_e;
     arg_max(ch, E, best, best_e);
-    const float weight = sc[best_e];
+    float weight = sc[best_e];
+    if (score_mode == 2) {                            // softmax over the chosen logits
+      if (slot == 0) first_logit = weight;
+      weight = expf(weight - first_logit);
+    }
     if (lane == 0) {
       ids_out[(size_t)token * top + slot] = best_e;
       weights_out[(size_t)token * top + slot] = weight;
@@ -168,36 +177,38 @@ template <typename T, int TPB>
 static int launch_moe_route(int* ids_out, float* weights_out, float* gate_out, const void* x, long long x_stride,
                             const float* router, const float* gate_rows, int tokens, int E, int R, int K, int top,
                             int score_mode, int renormalize, const float* correction, int groups, int keep,
-                            float weight_scale, cudaStream_t stream) {
+                            float weight_scale, const float* bias, cudaStream_t stream) {
   const size_t smem = (size_t)TPB * K * sizeof(T) + (size_t)TPB * (2 * E + R + 2 * groups) * sizeof(float);
   KVB_REQUIRE(smem <= 200 * 1024, "moe_route: the tokens' rows and scores do not fit in shared memory");
   if (smem > 48 * 1024)
     KVB_CHECK_CUDA(cudaFuncSetAttribute(moe_route_kernel<T, TPB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   KVB_CHECK_CUDA(kvb_launch((moe_route_kernel<T, TPB>), dim3((tokens + TPB - 1) / TPB), dim3(MOE_ROUTE_THREADS), smem,
                             stream, true, ids_out, weights_out, gate_out, (const T*)x, x_stride, router, gate_rows,
-                            tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale));
+                            tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale,
+                            bias));
   return 0;
 }
 
 extern "C" int kvb_moe_route(int* ids_out, float* weights_out, float* gate_out, const void* x, long long x_stride,
                              const float* router, const float* gate_rows, int tokens, int E, int R, int K, int top,
                              int score_mode, int renormalize, const float* correction, int groups, int keep,
-                             float weight_scale, int dtype, cudaStream_t stream) {
+                             float weight_scale, const float* bias, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   KVB_REQUIRE(E > 0 && K > 0 && top > 0 && top <= E, "moe_route: need 0 < top <= experts");
   KVB_REQUIRE(groups > 0 && E % groups == 0 && keep > 0 && keep <= groups && (long long)keep * (E / groups) >= top,
               "moe_route: the kept groups of experts must hold the experts to choose");
   KVB_REQUIRE(R >= 0 && (R == 0 || (gate_rows != nullptr && gate_out != nullptr)), "moe_route: gate rows need their weights and output");
-  KVB_REQUIRE(score_mode == 0 || score_mode == 1, "moe_route: unknown score function");
+  KVB_REQUIRE(score_mode >= 0 && score_mode <= 2, "moe_route: unknown score function");
+  if (score_mode == 2) renormalize = 1;
   // a prompt's tokens go eight a block; a few tokens one a block, for the parallelism
   const bool many = tokens >= 256 && (size_t)8 * K * (dtype == KVB_F32 ? 4 : 2) <= 96 * 1024;
   int rc;
   if (dtype == KVB_F32)
-    rc = many ? launch_moe_route<float, 8>(ids_out, weights_out, gate_out, x, x_stride, router, gate_rows, tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale, stream)
-              : launch_moe_route<float, 1>(ids_out, weights_out, gate_out, x, x_stride, router, gate_rows, tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale, stream);
+    rc = many ? launch_moe_route<float, 8>(ids_out, weights_out, gate_out, x, x_stride, router, gate_rows, tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale, bias, stream)
+              : launch_moe_route<float, 1>(ids_out, weights_out, gate_out, x, x_stride, router, gate_rows, tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale, bias, stream);
   else
-    rc = many ? launch_moe_route<bf16, 8>(ids_out, weights_out, gate_out, x, x_stride, router, gate_rows, tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale, stream)
-              : launch_moe_route<bf16, 1>(ids_out, weights_out, gate_out, x, x_stride, router, gate_rows, tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale, stream);
+    rc = many ? launch_moe_route<bf16, 8>(ids_out, weights_out, gate_out, x, x_stride, router, gate_rows, tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale, bias, stream)
+              : launch_moe_route<bf16, 1>(ids_out, weights_out, gate_out, x, x_stride, router, gate_rows, tokens, E, R, K, top, score_mode, renormalize, correction, groups, keep, weight_scale, bias, stream);
   if (rc) return rc;
   KVB_CHECK_LAUNCH();
   return 0;
@@ -275,11 +286,25 @@ __device__ __forceinline__ float moe_silu<float>(float x) { return x / (1.0f + e
 template <>
 __device__ __forceinline__ float moe_silu<bf16>(float x) { return kvb_silu_for_bf16(x); }
 
+// How an expert joins its two branches: silu(gate) * up, or (limit > 0) the bounded form.
+struct MoeJoin { float alpha, limit, shift; };
+
+// As the separate kernels would: both products rounded, then (silu) the activation rounded and the product taken.
+template <typename T>
+__device__ __forceinline__ float moe_join(float gate, float up, const MoeJoin& join) {
+  const float g = to_float(from_float<T>(gate)), u = to_float(from_float<T>(up));
+  if (join.limit > 0.0f) {
+    const float gc = fminf(g, join.limit), uc = fminf(fmaxf(u, -join.limit), join.limit);
+    return gc / (1.0f + expf(-join.alpha * gc)) * (uc + join.shift);
+  }
+  return to_float(from_float<T>(moe_silu<T>(g))) * u;
+}
+
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(T* __restrict__ out, const T* __restrict__ a, long long a_stride, int a_row_div,
                 const float* __restrict__ pair_weight, const T* __restrict__ w, const int* __restrict__ sorted,
-                const int* __restrict__ tile_expert, const int* __restrict__ meta, int N, int K) {
+                const int* __restrict__ tile_expert, const int* __restrict__ meta, int N, int K, MoeJoin join) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_MOE_GEMM);
   if ((int)blockIdx.x >= meta[0]) return;
   __shared__ float as[MOE_BK][MOE_BM + 1];
@@ -336,25 +361,23 @@ moe_gemm_kernel(T* __restrict__ out, const T* __restrict__ a, long long a_stride
     const int n = n0 + c0 + j;
     if (n >= N) continue;
     float v = acc[j];
-    if (GATED) {
-      // as the separate kernels would: both products rounded, the activation rounded, then the product
-      const float g = to_float(from_float<T>(acc[j])), u = to_float(from_float<T>(acc_up[j]));
-      v = to_float(from_float<T>(moe_silu<T>(g))) * u;
-    }
+    if (GATED) v = moe_join<T>(acc[j], acc_up[j], join);
     out[(size_t)pair * N + n] = from_float<T>(v);
   }
 }
 
 extern "C" int kvb_moe_gemm(void* out, const void* a, long long a_stride, int a_row_div, const float* pair_weight,
                             const void* w, const int* sorted, const int* tile_expert, const int* meta, int max_tiles,
-                            int N, int K, int gated, int dtype, cudaStream_t stream) {
+                            int N, int K, int gated, float alpha, float limit, float shift, int dtype,
+                            cudaStream_t stream) {
+  const MoeJoin join = {alpha, limit, shift};
   if (max_tiles == 0) return 0;
   KVB_REQUIRE(N > 0 && K > 0 && a_row_div > 0, "moe_gemm: empty product");
   dim3 grid(max_tiles, (N + MOE_BN - 1) / MOE_BN);
   KVB_REQUIRE(grid.y <= 65535, "moe_gemm: too many output columns for one launch");
 #define KVB_MOE_GEMM(T_, G_)                                                                                  \
   KVB_CHECK_CUDA(kvb_launch((moe_gemm_kernel<T_, G_>), grid, dim3(256), 0, stream, true, (T_*)out, (const T_*)a, \
-                            a_stride, a_row_div, pair_weight, (const T_*)w, sorted, tile_expert, meta, N, K))
+                            a_stride, a_row_div, pair_weight, (const T_*)w, sorted, tile_expert, meta, N, K, join))
   if (dtype == KVB_F32) { if (gated) KVB_MOE_GEMM(float, true); else KVB_MOE_GEMM(float, false); }
   else { if (gated) KVB_MOE_GEMM(bf16, true); else KVB_MOE_GEMM(bf16, false); }
 #undef KVB_MOE_GEMM
@@ -372,7 +395,7 @@ template <bool GATED>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long long a_stride, int a_row_div,
                 const float* __restrict__ pair_weight, const bf16* __restrict__ w, const int* __restrict__ ids,
-                int E, int N, int K, int* status) {
+                int E, int N, int K, int* status, MoeJoin join) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_MOE_GEMM);
   extern __shared__ __align__(16) unsigned char gemv_smem[];
   bf16* xs = reinterpret_cast<bf16*>(gemv_smem);
@@ -424,16 +447,16 @@ moe_gemv_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long long a_
     float v = lane == 0 ? acc[0] : lane == 1 ? acc[1] : lane == 2 ? acc[2] : acc[3];
     if (GATED) {
       const float u = lane == 0 ? acc[4 % ROWS] : lane == 1 ? acc[5 % ROWS] : lane == 2 ? acc[6 % ROWS] : acc[7 % ROWS];
-      const float g = to_float(from_float<bf16>(v));
-      v = to_float(from_float<bf16>(moe_silu<bf16>(g))) * to_float(from_float<bf16>(u));
+      v = moe_join<bf16>(v, u, join);
     }
     out[(size_t)pair * N + n0 + lane] = from_float<bf16>(v);
   }
 }
 
 extern "C" int kvb_moe_gemv(void* out, const void* a, long long a_stride, int a_row_div, const float* pair_weight,
-                            const void* w, const int* ids, int pairs, int E, int N, int K, int gated,
-                            cudaStream_t stream) {
+                            const void* w, const int* ids, int pairs, int E, int N, int K, int gated, float alpha,
+                            float limit, float shift, cudaStream_t stream) {
+  const MoeJoin join = {alpha, limit, shift};
   if (pairs == 0) return 0;
   KVB_REQUIRE(N > 0 && K > 0 && K % 8 == 0 && a_stride % 8 == 0 && a_row_div > 0, "moe_gemv: K and the row stride must be multiples of 8");
   KVB_REQUIRE(aligned16(a) && aligned16(w), "moe_gemv: operands must be 16-byte aligned");
@@ -448,7 +471,7 @@ extern "C" int kvb_moe_gemv(void* out, const void* a, long long a_stride, int a_
     if (smem > 48 * 1024)                                                                                      \
       KVB_CHECK_CUDA(cudaFuncSetAttribute(moe_gemv_kernel<G_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
     KVB_CHECK_CUDA(kvb_launch((moe_gemv_kernel<G_>), grid, dim3(256), smem, stream, true, (bf16*)out, (const bf16*)a, \
-                              a_stride, a_row_div, pair_weight, (const bf16*)w, ids, E, N, K, status));        \
+                              a_stride, a_row_div, pair_weight, (const bf16*)w, ids, E, N, K, status, join));  \
   } while (0)
   if (gated) KVB_MOE_GEMV(true); else KVB_MOE_GEMV(false);
 #undef KVB_MOE_GEMV
@@ -471,7 +494,7 @@ __global__ void __launch_bounds__(256)
 moe_gemv_rows_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long long a_stride, int a_row_div,
                      const float* __restrict__ pair_weight, const bf16* __restrict__ w,
                      const int* __restrict__ sorted, const int* __restrict__ tile_expert,
-                     const int* __restrict__ meta, int N, int K) {
+                     const int* __restrict__ meta, int N, int K, MoeJoin join) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_MOE_GEMM);
   extern __shared__ __align__(16) unsigned char gemv_smem[];
   bf16* xs = reinterpret_cast<bf16*>(gemv_smem);            // [MOE_GEMV_ROWS][K]
@@ -550,10 +573,7 @@ moe_gemv_rows_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long lo
       }
   const int pair = lane < MOE_GEMV_ROWS * CPW ? pair_of[r] : -1;
   if (pair >= 0 && n0 + c < N) {
-    if (GATED) {
-      const float g = to_float(from_float<bf16>(v));
-      v = to_float(from_float<bf16>(moe_silu<bf16>(g))) * to_float(from_float<bf16>(u));
-    }
+    if (GATED) v = moe_join<bf16>(v, u, join);
     out[(size_t)pair * N + n0 + c] = from_float<bf16>(v);
   }
   }
@@ -561,7 +581,9 @@ moe_gemv_rows_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long lo
 
 extern "C" int kvb_moe_gemv_rows(void* out, const void* a, long long a_stride, int a_row_div, const float* pair_weight,
                                  const void* w, const int* sorted, const int* tile_expert, const int* meta,
-                                 int max_tiles, int N, int K, int gated, cudaStream_t stream) {
+                                 int max_tiles, int N, int K, int gated, float alpha, float limit, float shift,
+                                 cudaStream_t stream) {
+  const MoeJoin join = {alpha, limit, shift};
   if (max_tiles == 0) return 0;
   KVB_REQUIRE(N > 0 && K > 0 && K % 8 == 0 && a_stride % 8 == 0 && a_row_div > 0, "moe_gemv_rows: K and the row stride must be multiples of 8");
   KVB_REQUIRE(aligned16(a) && aligned16(w), "moe_gemv_rows: operands must be 16-byte aligned");
@@ -576,7 +598,7 @@ extern "C" int kvb_moe_gemv_rows(void* out, const void* a, long long a_stride, i
       KVB_CHECK_CUDA(cudaFuncSetAttribute(moe_gemv_rows_kernel<G_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
     KVB_CHECK_CUDA(kvb_launch((moe_gemv_rows_kernel<G_>), grid, dim3(256), smem, stream, true, (bf16*)out,     \
                               (const bf16*)a, a_stride, a_row_div, pair_weight, (const bf16*)w, sorted,        \
-                              tile_expert, meta, N, K));                                                       \
+                              tile_expert, meta, N, K, join));                                                 \
   } while (0)
   if (gated) KVB_MOE_GEMV_ROWS(true); else KVB_MOE_GEMV_ROWS(false);
 #undef KVB_MOE_GEMV_ROWS

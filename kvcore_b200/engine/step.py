@@ -88,6 +88,7 @@ class StepContext:
         self.host_query_lens: list[int] = []
         self.host_context_lens: list[int] = []
         self.host_state_slots: list[int] = []
+        self.embedding_state: torch.Tensor | None = None   # ``[slots, *shape]`` of the embedding's own ``StateSpec``
         self._shared: dict = {}
 
     def shared(self, key, make):
@@ -108,7 +109,7 @@ class CacheStorage:
     Per group one tensor ``[entries, planes, pages, heads, page_size, width]`` as the group's
     ``CacheSpec`` has it (keys at plane 0, values at plane 1 for attention): every entry of the
     group stores a page id's tokens in its own slice.  Per schedule entry with a ``StateSpec``
-    one tensor ``[slots, *shape]``.
+    one tensor ``[slots, *shape]``; one more if the embedding keeps state of its own.
     """
 
     def __init__(
@@ -154,6 +155,11 @@ class CacheStorage:
                                           dtype=req.block_state_spec.dtype, device=device)
                 self.state_tensors.append(block_state)
             self.layer_caches.append(LayerCache(group_id, planes, owner, state, page_size, block_state))
+        self.embedding_state: torch.Tensor | None = None
+        spec = model.embedding_state_spec()
+        if spec is not None:
+            self.embedding_state = torch.zeros((num_slots, *spec.shape), dtype=spec.dtype, device=device)
+            self.state_tensors.append(self.embedding_state)
 
     # what "poison" writes into freed pages: large enough that a read of a position nobody wrote
     # changes the logits by orders of magnitude, finite so that a masked probability of exactly
@@ -442,6 +448,7 @@ class StepFunction:
         ctx.host_query_lens = query_lens
         ctx.host_context_lens = context_lens
         ctx.host_state_slots = slots
+        ctx.embedding_state = self.storage.embedding_state
         return ctx
 
     # ---- the step ------------------------------------------------------------------------------

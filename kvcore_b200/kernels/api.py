@@ -52,12 +52,14 @@ def ensure_built(verbose: bool = False) -> str:
                            _int, _int, _float, _int, _int, _int, _int, _vp],
         "kvb_glu_clamped": [_vp, _vp, _int, _int, _float, _float, _float, _int, _vp],
         "kvb_moe_route": [_vp, _vp, _vp, _vp, _ll, _vp, _vp, _int, _int, _int, _int, _int, _int, _int, _vp, _int, _int,
-                          _float, _int, _vp],
+                          _float, _vp, _int, _vp],
         "kvb_moe_align": [_vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _vp],
-        "kvb_moe_gemv": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _int, _int, _int, _int, _int, _vp],
-        "kvb_moe_gemv_rows": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _vp],
+        "kvb_moe_gemv": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _int, _int, _int, _int, _int, _float, _float, _float, _vp],
+        "kvb_moe_gemv_rows": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _float, _float,
+                              _float, _vp],
         "kvb_moe_gather": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _int, _int, _vp, _int, _int, _vp],
-        "kvb_moe_gemm": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _int, _vp],
+        "kvb_moe_gemm": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _float, _float, _float,
+                         _int, _vp],
         "kvb_moe_combine": [_vp, _vp, _int, _int, _vp, _vp, _vp, _vp, _int, _int, _int, _vp],
         "kvb_flash_paged_attention": [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _int, _vp, _vp, _int, _int, _int,
                                       _int, _int, _int, _int, _float, _int, _int, _vp, _vp, _vp],
@@ -96,6 +98,15 @@ def ensure_built(verbose: bool = False) -> str:
         "kvb_gated_rms_norm": [_vp, _ll, _vp, _vp, _ll, _vp, _int, _int, _int, _float, _float, _int, _int, _vp],
         "kvb_lightning_scan": [_vp, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _ll, _ll, _vp, _vp, _int, _int, _int, _int, _int,
                                _float, _int, _vp],
+        "kvb_ssm_prepare": [_vp, _ll, _vp, _ll, _vp, _int, _vp, _vp, _ll, _ll, _vp, _vp, _vp, _vp, _vp, _int, _int, _int,
+                            _int, _int, _int, _vp],
+        "kvb_ssm_scan": [_vp, _vp, _ll, _vp, _vp, _ll, _ll, _vp, _vp, _int, _int, _int, _int, _int, _int, _vp],
+        "kvb_gated_group_norm": [_vp, _ll, _vp, _vp, _ll, _vp, _int, _int, _int, _float, _int, _vp],
+        "kvb_stream_add_rows": [_vp, _vp, _int, _vp, _vp, _vp, _int, _vp, _vp, _vp, _float, _vp, _vp, _int, _int, _int,
+                                _int, _vp],
+        "kvb_embed_pairs": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _ll, _ll, _ll, _float,
+                            _int, _vp],
+        "kvb_softcap": [_vp, _ll, _float, _float, _vp],
         "kvb_gelu_mul": [_vp, _vp, _vp, _ll, _int, _int, _int, _int, _vp],
         "kvb_turn_norm_kv_write": [_vp, _ll, _vp, _int, _vp, _vp, _int, _float, _vp, _vp, _vp, _int, _vp, _int, _int,
                                    _int, _int, _int, _int, _int, _int, _float, _int, _vp, _ll, _vp, _int, _vp],
@@ -673,13 +684,15 @@ _stream_scratch: dict[int, torch.Tensor] = {}
 TRACE_TAGS = {27: "rms_norm_shift", 28: "stream_add_norm", 29: "attention_dims_rows", 30: "latent_prepare",
               31: "head_norm_kv_write", 32: "maps_combine", 33: "sigmoid_gate_mul", 34: "flash_dims",
               35: "flash_dims_combine", 36: "gather_cached_rows", 37: "gla_scan", 38: "delta_scan", 39: "conv_prepare",
-              40: "gated_rms_norm", 41: "turn_norm_kv_write", 42: "head_gate", 43: "embed_scaled", 44: "gla_prepare", 45: "gelu_mul", 46: "lightning_prepare", 47: "lightning_scan", 25: "kept_first_merge", 26: "moe_gather", 17: "layer_norm", 18: "stream_add", 19: "qk_prepare", 20: "glu_clamped", 21: "moe_route",
+              40: "gated_rms_norm", 41: "turn_norm_kv_write", 42: "head_gate", 43: "embed_scaled", 44: "gla_prepare", 45: "gelu_mul", 46: "lightning_prepare", 47: "lightning_scan", 48: "ssm_scan",
+              49: "ssm_prepare", 50: "gated_group_norm", 51: "stream_add_rows", 52: "embed_pairs", 53: "softcap", 25: "kept_first_merge", 26: "moe_gather", 17: "layer_norm", 18: "stream_add", 19: "qk_prepare", 20: "glu_clamped", 21: "moe_route",
               22: "moe_align", 23: "moe_gemm", 24: "moe_combine", 1: "gather_rows", 2: "rmsnorm", 3: "silu_mul", 4: "rope_table", 5: "rope_kv_write", 6: "attention_rows",
               7: "flash_paged", 8: "flash_combine", 9: "flash_decode_tma", 10: "flash_decode_combine",
               11: "flash_prefill_tc5", 12: "gemm_f32", 13: "gemm_stream", 14: "sample", 16: "feed_tokens"}
 _TRACE_UNITS = ("elementwise", "attention_decode_tma", "attention_flash", "attention_generic",
                 "attention_prefill_tc5", "gemm_f32", "sampling", "gemm_stream", "layer_norm", "qk_prepare", "moe", "attention_kept_first",
-                "stream_norm", "attention_dims", "mixer_prepare", "attention_flash_dims", "recurrence", "turn_norm")
+                "stream_norm", "attention_dims", "mixer_prepare", "attention_flash_dims", "recurrence", "turn_norm",
+                "state_space", "stream_rows")
 _trace_buffer: torch.Tensor | None = None
 
 
@@ -802,7 +815,7 @@ def linear(
         else:
             out = torch.mm(x, weight.t()).float()
         if bias is not None:
-            out = out + bias.float()
+            out.add_(bias)
         return out
     return torch.nn.functional.linear(x, weight, bias)
 
@@ -1037,6 +1050,65 @@ def stream_add_norm(x: torch.Tensor, a: torch.Tensor, weight: torch.Tensor, eps:
     return (out, avg) if rounded is None else (out, avg, narrow)
 
 
+def stream_add_rows(x: torch.Tensor, a, *, weight: torch.Tensor | None = None, eps: float = 0.0,
+                    out_dtype: torch.dtype | None = None, token_rows: torch.Tensor | None = None,
+                    origin: torch.Tensor | None = None, keep: bool = True) -> tuple:
+    """``X = x + a`` on the 32-bit stream ``x [T, width]``, ``a`` a sub-layer's output ``[T, width]`` or the rows its
+    experts left (``ExpertRows``: summed per token in ascending slot, weights still pending included), or None.  Returns
+    ``(X, y, packed)``: ``X`` is ``x`` updated in place (``keep`` False or ``token_rows`` given: ``x`` stays and
+    ``X`` is None); ``y = X * rsqrt(mean(X^2) + eps) * weight`` in ``out_dtype`` (with ``weight``, else None);
+    ``packed [T, 2 * width]`` = ``[X | origin]`` in ``out_dtype`` (with ``origin``, a stream of the same shape, else
+    None).  ``token_rows`` (int32): only those tokens, the outputs compact and in their order."""
+    experts = a if isinstance(a, ExpertRows) else None
+    rows = a if experts is None else experts.rows
+    _check(x, "x", dtype=torch.float32)
+    tokens, width = x.shape
+    if rows is not None:
+        _check(rows, "a")
+    if rows is not None and (rows.dim() != 2 or rows.shape[1] != width):
+        raise KernelError(f"stream_add_rows: rows {tuple(rows.shape)} do not match the stream {tuple(x.shape)}")
+    top, row_of_pair, pair_weight = 1, None, None
+    if experts is not None:
+        top, row_of_pair, pair_weight = experts.top, experts.row_of_pair, experts.pending_weights
+        for name, t, kind in (("row_of_pair", row_of_pair, torch.int32), ("pending weights", pair_weight, torch.float32)):
+            if t is not None:
+                _check(t, name, dtype=kind)
+                if t.numel() != tokens * top:
+                    raise KernelError(f"stream_add_rows: {t.numel()} {name} for {tokens} x {top} pairs")
+    if rows is None:
+        top, keep = 0, False
+        if out_dtype is None:
+            raise KernelError("stream_add_rows: without anything to add the type of the outputs must be given")
+    elif row_of_pair is None and rows.shape[0] != tokens * top:
+        raise KernelError(f"stream_add_rows: {rows.shape[0]} rows for {tokens} tokens of {top}")
+    dtype = out_dtype or rows.dtype
+    count = tokens
+    if token_rows is not None:
+        _check(token_rows, "token_rows", dtype=torch.int32)
+        count, keep = token_rows.numel(), False
+    normed = packed = None
+    weight_code = _F32
+    if weight is not None:
+        _check(weight, "weight")
+        if weight.numel() != width:
+            raise KernelError(f"stream_add_rows: weight has {weight.numel()} entries for rows of width {width}")
+        weight_code = _dtype_code(weight)
+        normed = torch.empty((count, width), dtype=dtype, device=x.device)
+    if origin is not None:
+        _check(origin, "origin", dtype=torch.float32)
+        if origin.shape != x.shape:
+            raise KernelError("stream_add_rows: origin does not match the stream")
+        packed = torch.empty((count, 2 * width), dtype=dtype, device=x.device)
+    code = _BF16 if dtype == torch.bfloat16 else _F32
+    _call("kvb_stream_add_rows", x.data_ptr(), None if rows is None else rows.data_ptr(), int(top),
+          None if row_of_pair is None else row_of_pair.data_ptr(), None if pair_weight is None else pair_weight.data_ptr(),
+          None if token_rows is None else token_rows.data_ptr(), count, x.data_ptr() if keep else None,
+          None if normed is None else normed.data_ptr(), None if weight is None else weight.data_ptr(), float(eps),
+          None if packed is None else packed.data_ptr(), None if origin is None else origin.data_ptr(), width,
+          code if rows is None else _dtype_code(rows), code, weight_code, _stream())
+    return (x if keep else None), normed, packed
+
+
 def attention_dims(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, table: torch.Tensor, ctx, *,
                    value_heads: int, group: int, maps: int, key_width: int, value_width: int, page_size: int,
                    num_pages: int, key_strides: tuple[int, int, int], value_strides: tuple[int, int, int], scale: float,
@@ -1227,6 +1299,26 @@ def latent_prepare(kv_rows: torch.Tensor, norm_weight: torch.Tensor, eps: float,
           int(q_width), *latent, q_out.data_ptr(), tokens, heads, rank, rot, lead, _dtype_code(kv_rows), _stream())
 
 
+def latent_cache_write(kv_rows: torch.Tensor, norm_weight: torch.Tensor, eps: float, ctx, table: torch.Tensor,
+                       cache: torch.Tensor) -> None:
+    """``latent_prepare`` for a mixer without position entries, whose queries need nothing done: the RMS norm of
+    ``kv_rows [T, rank]`` (a view) with ``norm_weight``, written into the tokens' places of
+    ``cache [pages, 1, page, rank]``."""
+    _check(kv_rows, "kv_rows", contiguous=False)
+    _check(cache, "cache", dtype=kv_rows.dtype)
+    _check(norm_weight, "norm_weight", dtype=kv_rows.dtype)
+    tokens, rank = kv_rows.shape
+    num_pages, one, page_size, width = cache.shape
+    if one != 1 or width != rank or norm_weight.numel() != rank or (tokens and kv_rows.stride(1) != 1):
+        raise KernelError(f"latent_cache_write: rows {tuple(kv_rows.shape)} / cache {tuple(cache.shape)} do not fit")
+    if ctx.positions.numel() != tokens:
+        raise KernelError(f"latent_cache_write: {ctx.positions.numel()} positions for {tokens} tokens")
+    _call("kvb_latent_prepare", kv_rows.data_ptr(), kv_rows.stride(0), norm_weight.data_ptr(), float(eps), None, 0,
+          ctx.positions.data_ptr(), ctx.req_index.data_ptr(), table.data_ptr(), table.stride(0), cache.data_ptr(),
+          page_size, num_pages, 1, None, 0, 0, 0, None, 0, 0, None, tokens, 0, rank, 0, rank, _dtype_code(kv_rows),
+          _stream())
+
+
 def gather_cached_rows(cache: torch.Tensor, table: torch.Tensor, src_req: torch.Tensor, src_pos: torch.Tensor,
                        col0: int, cols: int, out: torch.Tensor, *, copies: int = 1, head_stride: int = 0) -> None:
     """Columns ``[col0, col0 + cols)`` of the cached rows of the tokens ``(src_req[n], src_pos[n])`` (request row
@@ -1299,8 +1391,7 @@ def sigmoid_gate_mul(o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
 
 def heads_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
     """A product per head: ``x [T, H, K]`` (a view; last stride 1) with ``weight [H, N, K]`` -> ``[T, H, N]``
-    (a view when the batched library product made it; into ``out``, a view with last stride 1, on the 32-bit
-    path).  float32: this package's own FMA kernel, head by head; bfloat16: one batched library product."""
+    (a view when the batched library product made it; into ``out``, a view with last stride 1, when given).  float32: this package's own FMA kernel, head by head; bfloat16: one batched library product."""
     _check(x, "x", contiguous=False)
     _check(weight, "weight", dtype=x.dtype)
     tokens, heads, k = x.shape
@@ -1316,11 +1407,12 @@ def heads_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor | None
             _call("kvb_gemm_f32", out[:, h].data_ptr(), x[:, h].data_ptr(), weight[h].data_ptr(), None, tokens, n, k,
                   x.stride(0), out.stride(0), _stream())
         return out
-    result = torch.bmm(x.transpose(0, 1), weight.transpose(1, 2)).transpose(0, 1)
-    if out is not None:
-        out.copy_(result)
+    if out is not None:                     # the library writes the rows where they belong
+        if tuple(out.shape) != (tokens, heads, n) or out.stride(2) != 1:
+            raise KernelError(f"heads_linear: out {tuple(out.shape)} does not fit")
+        torch.bmm(x.transpose(0, 1), weight.transpose(1, 2), out=out.transpose(0, 1))
         return out
-    return result
+    return torch.bmm(x.transpose(0, 1), weight.transpose(1, 2)).transpose(0, 1)
 
 
 QK_NORM_MODES = {None: 0, "none": 0, "projection": 1, "head": 2}
@@ -1335,6 +1427,51 @@ def embed_scaled(table: torch.Tensor, ids: torch.Tensor, scale: float) -> torch.
     _call("kvb_embed_scaled", out.data_ptr(), table.data_ptr(), ids.data_ptr(), ids.numel(), table.shape[0],
           table.shape[1], float(scale), _dtype_code(table), _stream())
     return out
+
+
+def embed_pairs(table: torch.Tensor, ids: torch.Tensor, *, pairs: torch.Tensor | None = None, mul_prev: int = 0,
+                mul_cur: int = 0, weight: torch.Tensor | None = None, eps: float = 0.0,
+                state: torch.Tensor | None = None, ctx=None) -> torch.Tensor:
+    """The first value of a 32-bit residual stream, ``[T, width]``: ``table[ids]``, plus (``pairs``
+    ``[buckets + 1, width]``) the row ``(id in front * mul_prev + id * mul_cur) mod buckets`` of a second table, for
+    a request's first token its last row; then (``weight``, 32-bit) an RMS norm of the sum.  The id in front of a
+    request's portion is its word of ``state [slots, 1]`` (int32), which this call brings up to date."""
+    _check(table, "table")
+    _check(ids, "ids", dtype=torch.int32)
+    tokens, (vocab, width) = ids.numel(), table.shape
+    batch = (None, None, None, None, None)
+    buckets = 0
+    if pairs is not None:
+        _check(pairs, "pairs", dtype=table.dtype)
+        if pairs.dim() != 2 or pairs.shape[1] != width or pairs.shape[0] < 2:
+            raise KernelError(f"embed_pairs: pair table {tuple(pairs.shape)} does not match rows of width {width}")
+        if state is None or ctx is None:
+            raise KernelError("embed_pairs: a pair table needs the state and the step's context")
+        _check(state, "state", dtype=torch.int32)
+        if state.numel() != state.shape[0] or ctx.positions.numel() != tokens:
+            raise KernelError(f"embed_pairs: state {tuple(state.shape)} is not one word a slot")
+        buckets = pairs.shape[0] - 1
+        # below 2^31 times an id (also below 2^31), so that the row's number stays inside 64 bits
+        if max(abs(int(mul_prev)), abs(int(mul_cur))) >= 1 << 31:
+            raise KernelError("embed_pairs: the factors of a pair must lie inside 32 bits")
+        batch = (ctx.positions.data_ptr(), ctx.req_index.data_ptr(), ctx.query_start.data_ptr(),
+                 ctx.state_slots.data_ptr(), state.data_ptr())
+    if weight is not None:
+        _check(weight, "weight", dtype=torch.float32)
+        if weight.numel() != width:
+            raise KernelError(f"embed_pairs: weight has {weight.numel()} entries for rows of width {width}")
+    out = torch.empty((tokens, width), dtype=torch.float32, device=table.device)
+    _call("kvb_embed_pairs", out.data_ptr(), table.data_ptr(), None if pairs is None else pairs.data_ptr(),
+          None if weight is None else weight.data_ptr(), ids.data_ptr(), *batch, tokens, vocab, width, buckets,
+          int(mul_prev), int(mul_cur), float(eps), _dtype_code(table), _stream())
+    return out
+
+
+def softcap(logits: torch.Tensor, scale: float, cap: float) -> torch.Tensor:
+    """``cap * tanh(logits * scale / cap)`` in place (32-bit)."""
+    _check(logits, "logits", dtype=torch.float32)
+    _call("kvb_softcap", logits.data_ptr(), logits.numel(), float(scale), float(cap), _stream())
+    return logits
 
 
 def turn_norm_kv_write(rows: torch.Tensor, inv_freq: torch.Tensor | None, rot: int, ctx, table: torch.Tensor,
@@ -1541,6 +1678,80 @@ def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
     return out
 
 
+def ssm_row_width(heads: int, groups: int, dim: int, value_dim: int) -> int:
+    """32-bit entries of a token's prepared row ``[B | C | x | dt | decay]``, rounded up to 16 bytes."""
+    return (2 * groups * dim + heads * value_dim + 2 * heads + 3) & ~3
+
+
+def ssm_prepare(rows: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, ctx,
+                a_log: torch.Tensor, dt_bias: torch.Tensor, *, heads: int, groups: int, dim: int, value_dim: int,
+                state_offset: int) -> torch.Tensor:
+    """What a selective state-space mixer does to its projections before the scan.  ``rows`` (a view; last stride 1):
+    the channels ``[x: heads * value_dim | B: groups * dim | C: groups * dim]``, then a column a head for the step
+    size.  The channels pass a causal convolution over time (``taps [channels, K]`` 32-bit, the last tap on the
+    current token, plus ``bias``; the ``K - 1`` inputs in front of a portion are the request's
+    ``state[slot, state_offset:]`` as ``[K - 1, channels]``, brought up to date by this call) and SiLU;
+    ``dt = softplus(step + dt_bias)``, ``decay = exp(-exp(a_log) * dt)``.  Returns 32-bit rows
+    ``[B | C | x | dt | decay]`` (``ssm_row_width`` entries)."""
+    channels = heads * value_dim + 2 * groups * dim
+    _check(rows, "rows", contiguous=False)
+    for name, t, count in (("bias", bias, channels), ("a_log", a_log, heads), ("dt_bias", dt_bias, heads)):
+        _check(t, name, dtype=torch.float32)
+        if t.numel() != count:
+            raise KernelError(f"ssm_prepare: {name} has {t.numel()} entries, not {count}")
+    _check(taps, "taps", dtype=torch.float32)
+    if rows.stride(1) != 1 or taps.dim() != 2 or taps.shape[0] != channels or not 1 <= taps.shape[1] <= 9:
+        raise KernelError(f"ssm_prepare: taps {tuple(taps.shape)} for {channels} channels (1 to 9 taps)")
+    if rows.shape[1] < channels + heads:
+        raise KernelError(f"ssm_prepare: rows {tuple(rows.shape)} do not hold the channels and the step sizes")
+    _state_row(state, state_offset, channels * (taps.shape[1] - 1))
+    tokens = rows.shape[0]
+    out = torch.empty((tokens, ssm_row_width(heads, groups, dim, value_dim)), dtype=torch.float32, device=rows.device)
+    _call("kvb_ssm_prepare", out.data_ptr(), out.stride(0), rows.data_ptr(), rows.stride(0), taps.data_ptr(),
+          taps.shape[1], bias.data_ptr(), state.data_ptr(), state.stride(0), state_offset, ctx.req_index.data_ptr(),
+          ctx.query_start.data_ptr(), ctx.state_slots.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), tokens,
+          ctx.num_reqs, heads, heads * value_dim, channels, _dtype_code(rows), _stream(),
+          kernels=2 if taps.shape[1] > 1 and tokens != ctx.num_reqs else 1)
+    return out
+
+
+def ssm_scan(prepared: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, ctx, *, heads: int, groups: int, dim: int,
+             value_dim: int, state_offset: int = 0) -> torch.Tensor:
+    """The selective state-space recurrence over the step's tokens, request by request in order, on what
+    ``ssm_prepare`` left: ``S <- decay_t S + B_t (dt_t x_t)^T``, ``o_t = S^T C_t + skip[h] x_t`` (head ``h`` reads
+    group ``h // (heads / groups)`` of B and C).  ``state [slots, n]`` holds ``S`` column by column
+    (``[heads, value_dim, dim]``) at ``state_offset``.  Returns ``o [T, heads, value_dim]`` 32-bit."""
+    _check(prepared, "prepared", dtype=torch.float32)
+    _check(skip, "skip", dtype=torch.float32)
+    if prepared.dim() != 2 or prepared.shape[1] != ssm_row_width(heads, groups, dim, value_dim) or skip.numel() != heads:
+        raise KernelError(f"ssm_scan: prepared rows {tuple(prepared.shape)} do not match the head layout")
+    _state_row(state, state_offset, heads * dim * value_dim)
+    out = torch.empty((prepared.shape[0], heads, value_dim), dtype=torch.float32, device=prepared.device)
+    _call("kvb_ssm_scan", out.data_ptr(), prepared.data_ptr(), prepared.stride(0), skip.data_ptr(), state.data_ptr(),
+          state.stride(0), state_offset, ctx.query_start.data_ptr(), ctx.state_slots.data_ptr(), prepared.shape[0],
+          ctx.num_reqs, heads, groups, dim, value_dim, _stream())
+    return out
+
+
+def gated_group_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                     groups: int) -> torch.Tensor:
+    """The gate first, then the norm: ``v = o * silu(gate)`` over a token's whole read-out, cut into ``groups`` equal
+    parts, ``out = v / sqrt(mean of the part's v^2 + eps) * weight``.  ``o [T, ...]`` 32-bit (``width`` entries a
+    token), ``gate`` and ``out [T, width]`` views of the activation type, ``weight [width]`` 32-bit."""
+    _check(o, "o", dtype=torch.float32)
+    _check(gate, "gate", contiguous=False)
+    _check(out, "out", dtype=gate.dtype, contiguous=False)
+    _check(weight, "weight", dtype=torch.float32)
+    tokens, width = gate.shape
+    if (o.numel() != tokens * width or tuple(out.shape) != (tokens, width) or weight.numel() != width or groups <= 0
+            or width % groups or (tokens and (gate.stride(1) != 1 or out.stride(1) != 1))):
+        raise KernelError(f"gated_group_norm: gate {tuple(gate.shape)} / out {tuple(out.shape)} / weight do not fit "
+                          f"o {tuple(o.shape)} in {groups} parts")
+    _call("kvb_gated_group_norm", out.data_ptr(), out.stride(0), o.data_ptr(), gate.data_ptr(), gate.stride(0),
+          weight.data_ptr(), tokens, groups, width // groups, float(eps), _dtype_code(out), _stream())
+    return out
+
+
 def gelu_mul(z: torch.Tensor, rows: torch.Tensor, column: int) -> torch.Tensor:
     """``gelu_tanh(z) * rows[:, column:column + dim]`` for ``z [T, dim]``, in 32-bit with one rounding;
     ``rows [T, n]`` of the same type (a table's rows of the step's tokens)."""
@@ -1624,14 +1835,16 @@ def glu_clamped(gate_up: torch.Tensor, *, alpha: float, limit: float, shift: flo
     return out
 
 
-MOE_SCORE_MODES = {"sigmoid": 0, "softmax": 1}
+# "softmax_chosen": the choice goes by the logits, the weights are the softmax over the chosen logits alone
+MOE_SCORE_MODES = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
 
 
 def moe_route(x: torch.Tensor, router: torch.Tensor, top: int, *, score: str = "sigmoid", renormalize: bool = False,
               gate_rows: torch.Tensor | None = None, correction: torch.Tensor | None = None, group_count: int = 1,
-              group_keep: int = 1, weight_scale: float = 1.0) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor | None]:
-    """Router of a mixture of experts on ``x [T, K]``: 32-bit logits with the 32-bit matrix ``router [E, K]``,
-    scores by ``score``, the ``top`` largest per token.  ``correction [E]`` (32-bit): the choice goes by
+              group_keep: int = 1, weight_scale: float = 1.0,
+              bias: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor | None]:
+    """Router of a mixture of experts on ``x [T, K]``: 32-bit logits with the 32-bit matrix ``router [E, K]`` (plus
+    ``bias [E]``, 32-bit), scores by ``score``, the ``top`` largest per token.  ``correction [E]`` (32-bit): the choice goes by
     ``score + correction``, the weights stay the scores.  ``group_count`` / ``group_keep``: the experts form
     equal groups of neighbours, a group's score is its largest choice score, and only experts of the
     ``group_keep`` best groups can be chosen.  ``weight_scale`` multiplies the weights.  Returns ``(ids [T, top] int32, weights [T, top] float32,
@@ -1655,6 +1868,10 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, top: int, *, score: str = "
         _check(correction, "correction", dtype=torch.float32)
         if correction.numel() != experts:
             raise KernelError(f"moe_route: {correction.numel()} corrections for {experts} experts")
+    if bias is not None:
+        _check(bias, "bias", dtype=torch.float32)
+        if bias.numel() != experts:
+            raise KernelError(f"moe_route: {bias.numel()} biases for {experts} experts")
     if (group_count <= 0 or experts % group_count or not 0 < group_keep <= group_count
             or group_keep * (experts // group_count) < top):
         raise KernelError(f"moe_route: {group_keep} of {group_count} groups of {experts} experts must hold {top} experts")
@@ -1662,7 +1879,7 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, top: int, *, score: str = "
           x.data_ptr(), x.stride(0), router.data_ptr(), None if gate_rows is None else gate_rows.data_ptr(),
           tokens, experts, extra, k, int(top), MOE_SCORE_MODES[score], int(bool(renormalize)),
           None if correction is None else correction.data_ptr(), int(group_count), int(group_keep), float(weight_scale),
-          _dtype_code(x), _stream())
+          None if bias is None else bias.data_ptr(), _dtype_code(x), _stream())
     return ids, weights, gates
 
 
@@ -1677,12 +1894,12 @@ MOE_GEMV_SINGLE_PAIRS = int(os.environ.get("KVCORE_B200_MOE_GEMV_SINGLE_PAIRS", 
 class ExpertRows:
     """What ``moe_experts`` leaves for ``moe_combine``: the experts' outputs ``rows [R, N]``, where the row of
     pair ``t * top + s`` is that index itself (``row_of_pair`` None) or ``row_of_pair[t * top + s]``, and
-    weights still to be applied (``pending_weights`` [T * top], or None)."""
+    weights still to be applied (``pending_weights`` [T * top], or None).  ``top``: pairs of a token."""
 
-    __slots__ = ("rows", "row_of_pair", "pending_weights")
+    __slots__ = ("rows", "row_of_pair", "pending_weights", "top")
 
-    def __init__(self, rows, row_of_pair=None, pending_weights=None):
-        self.rows, self.row_of_pair, self.pending_weights = rows, row_of_pair, pending_weights
+    def __init__(self, rows, row_of_pair=None, pending_weights=None, top=None):
+        self.rows, self.row_of_pair, self.pending_weights, self.top = rows, row_of_pair, pending_weights, top
 
 
 class ExpertGrouping:
@@ -1737,12 +1954,13 @@ def moe_path(x: torch.Tensor, pairs: int, ff: int) -> str:
 
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_up: torch.Tensor,
                 down: torch.Tensor, *, weight_on_input: bool, path: str | None = None,
-                grouping: ExpertGrouping | None = None) -> ExpertRows:
+                grouping: ExpertGrouping | None = None, join: tuple | None = None) -> ExpertRows:
     """The chosen experts of every token: for pair ``t * top + s`` with ``e = ids[t, s]``,
     ``down[e] @ (silu(gate[e] @ a) * (up[e] @ a))``.  ``weight_on_input``: ``a = weights[t, s] * x[t]``
     (rounded to the storage type).  Otherwise ``a = x[t]`` and the weight multiplies the output (the rows
     that enter the last product, or the sum in ``moe_combine``: that product is linear).
-    ``gate_up [E, 2F, K]`` (gate rows first), ``down [E, N, F]``.
+    ``gate_up [E, 2F, K]`` (gate rows first), ``down [E, N, F]``.  ``join = (alpha, limit, shift)``: the branches
+    join as in ``glu_clamped`` instead of ``silu(gate) * up``.
 
     Three ways, by ``path`` (default: by type and size).  "tiles": grouped products of this library, one
     accumulator per output in ascending k (all of float32: bit-equal under any batching).  "stream": bf16,
@@ -1763,6 +1981,15 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
         raise KernelError("moe_experts: the experts' matrices do not match the input")
     pairs = tokens * top
     code = _dtype_code(x)
+    if join is not None and not join[1] > 0:
+        raise KernelError(f"moe_experts: the branches' limit must be positive, got {join[1]}")
+    joined = (0.0, 0.0, 0.0) if join is None else tuple(float(v) for v in join)
+
+    def activate(both: torch.Tensor) -> torch.Tensor:
+        if join is None:
+            return silu_mul(both, 0)
+        return glu_clamped(both, alpha=joined[0], limit=joined[1], shift=joined[2])
+
     if path is None:
         path = moe_path(x, pairs, ff)
     if path == "stream" and pairs > MOE_GEMV_SINGLE_PAIRS and pairs >= 4 * experts:
@@ -1771,22 +1998,22 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
         hidden = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
         _call("kvb_moe_gemv_rows", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,
               weights.data_ptr() if weight_on_input else None, gate_up.data_ptr(), g.sorted_pairs.data_ptr(),
-              g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, ff, k, 1, _stream())
+              g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, ff, k, 1, *joined, _stream())
         out = torch.empty((pairs, n), dtype=x.dtype, device=x.device)
         _call("kvb_moe_gemv_rows", out.data_ptr(), hidden.data_ptr(), hidden.stride(0), 1,
               None if weight_on_input else weights.data_ptr(), down.data_ptr(), g.sorted_pairs.data_ptr(),
-              g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, n, ff, 0, _stream())
-        return ExpertRows(out)
+              g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, n, ff, 0, *joined, _stream())
+        return ExpertRows(out, top=top)
     if path == "stream":
         hidden = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
         _call("kvb_moe_gemv", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,
               weights.data_ptr() if weight_on_input else None, gate_up.data_ptr(), ids.data_ptr(), pairs, experts,
-              ff, k, 1, _stream())
+              ff, k, 1, *joined, _stream())
         out = torch.empty((pairs, n), dtype=x.dtype, device=x.device)
         _call("kvb_moe_gemv", out.data_ptr(), hidden.data_ptr(), hidden.stride(0), 1,
               None if weight_on_input else weights.data_ptr(), down.data_ptr(), ids.data_ptr(), pairs, experts,
-              n, ff, 0, _stream())
-        return ExpertRows(out)
+              n, ff, 0, *joined, _stream())
+        return ExpertRows(out, top=top)
     library = path == "library"
     if grouping is None or (library and grouping.expert_begin is None):
         grouping = moe_group(ids, experts, for_library=library)
@@ -1807,7 +2034,7 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
         # fewer pairs multiplies zero rows; with one expert far fuller than the rest, expert by expert instead)
         if experts * stride <= 2 * capacity + experts * 64:
             both = torch.bmm(gathered, gate_up.transpose(1, 2))
-            hidden = silu_mul(both.view(experts * stride, two_ff), 0).view(experts, stride, ff)
+            hidden = activate(both.view(experts * stride, two_ff)).view(experts, stride, ff)
             out = torch.bmm(hidden, down.transpose(1, 2)).view(experts * stride, n)
         else:
             # an expert's rows rounded up to 64 as well (the rows beyond its pairs are zeros): few shapes again
@@ -1816,22 +2043,22 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
             for e in range(experts):
                 if counts[e]:
                     torch.mm(gathered[e, : counts[e]], gate_up[e].t(), out=both[e, : counts[e]])
-            hidden = silu_mul(both.view(experts * stride, two_ff), 0).view(experts, stride, ff)
+            hidden = activate(both.view(experts * stride, two_ff)).view(experts, stride, ff)
             out = torch.empty((experts, stride, n), dtype=x.dtype, device=x.device)
             for e in range(experts):
                 if counts[e]:
                     torch.mm(hidden[e, : counts[e]], down[e].t(), out=out[e, : counts[e]])
             out = out.view(experts * stride, n)
-        return ExpertRows(out, row_of_pair, None if weight_on_input else weights.reshape(-1))
+        return ExpertRows(out, row_of_pair, None if weight_on_input else weights.reshape(-1), top)
     hidden = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
     _call("kvb_moe_gemm", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,
           weights.data_ptr() if weight_on_input else None, gate_up.data_ptr(), sorted_pairs.data_ptr(),
-          tile_expert.data_ptr(), meta.data_ptr(), max_tiles, ff, k, 1, code, _stream())
+          tile_expert.data_ptr(), meta.data_ptr(), max_tiles, ff, k, 1, *joined, code, _stream())
     out = torch.empty((pairs, n), dtype=x.dtype, device=x.device)
     _call("kvb_moe_gemm", out.data_ptr(), hidden.data_ptr(), hidden.stride(0), 1,
           None if weight_on_input else weights.data_ptr(), down.data_ptr(), sorted_pairs.data_ptr(),
-          tile_expert.data_ptr(), meta.data_ptr(), max_tiles, n, ff, 0, code, _stream())
-    return ExpertRows(out)
+          tile_expert.data_ptr(), meta.data_ptr(), max_tiles, n, ff, 0, *joined, code, _stream())
+    return ExpertRows(out, top=top)
 
 
 def moe_combine(expert_out, tokens: int, top: int, shared: torch.Tensor | None = None,

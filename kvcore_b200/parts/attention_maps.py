@@ -15,7 +15,9 @@ projection ``dkv`` gives ``kv_rank`` latent entries (RMS-normed with a weight: t
 cached.  The scores are taken in the latent space: ``q_h . (W_uk[h] c) = (W_uk[h]^T q_h) . c``, so the
 attention runs with one key head of ``kv_rank + rot_dim`` entries whose first ``kv_rank`` entries are also
 the values, and ``W_uv[h]`` is applied to the attention's output.  The softmax has a learned sink per head;
-the heads' outputs are gated by ``sigmoid(W_g x)`` before the output projection.
+the heads' outputs are gated by ``sigmoid(W_g x)`` before the output projection.  ``window``: a query sees that many
+trailing positions (its own included).  With ``rot_dim`` 0 there is no position entry, and the carried query is used
+where the product left it.
 
 Long portions of prompts (bfloat16, at least ``LatentAttention.expand_min_tokens`` tokens) take the other
 reading of the same product: the latents of the request's whole context are fetched from the cache and
@@ -134,8 +136,11 @@ class LatentAttention(Mixer):
 
     def __init__(self, *, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, value_dim: int,
                  kv_rank: int, scale: float, eps: float, rot_base: float, rot_dims: int, name: str,
-                 sink: bool = True, gate: bool = True, tensor_names: dict | None = None,
+                 sink: bool = True, gate: bool = True, window: int | None = None, tensor_names: dict | None = None,
                  dtype: torch.dtype, device: torch.device) -> None:
+        if window is not None and window <= 0:
+            raise ValueError(f"window must be positive when set, got {window}")
+        self.window = None if window is None else int(window)
         if min(num_heads, head_dim, value_dim, kv_rank) <= 0 or rot_dim < 0:
             raise ValueError("latent attention needs positive heads, head_dim, value_dim and kv_rank")
         if rot_dims % 2 or not 0 <= rot_dims <= rot_dim:
@@ -169,7 +174,7 @@ class LatentAttention(Mixer):
         self.inv_freq = table if torch.device(device).type == "meta" else table.to(device)
 
     def cache_spec(self) -> CacheSpec:
-        return CacheSpec(1, 1, self.kv_cols)
+        return CacheSpec(1, 1, self.kv_cols, self.window)
 
     def _tensor(self, key: str) -> str:
         return f"{self.name}.{self.tensor_names[key]}"
@@ -226,20 +231,23 @@ class LatentAttention(Mixer):
         def plan():
             # per step, shared by the model's latent layers: which cached rows to fetch, and a table that
             # addresses the fetched rows as pages of one token (row 0 stands for the null page)
-            totals = [c + n for c, n in zip(ctx.host_context_lens[:count], ctx.host_query_lens[:count])]
-            longest, rows_needed = max(totals), sum(totals)
+            # behind a window only what the portion's first token sees is fetched (earlier pages may be gone)
+            contexts, lens = ctx.host_context_lens[:count], ctx.host_query_lens[:count]
+            spans = [(0 if self.window is None else max(0, c - self.window + 1), c + n) for c, n in zip(contexts, lens)]
+            totals = [end - start for start, end in spans]
+            longest, rows_needed = max(end for _, end in spans), sum(totals)
             req = torch.repeat_interleave(torch.arange(count, dtype=torch.int32), torch.tensor(totals))
-            pos = torch.cat([torch.arange(n, dtype=torch.int32) for n in totals])
+            pos = torch.cat([torch.arange(start, end, dtype=torch.int32) for start, end in spans])
             row_table = torch.zeros((count, longest), dtype=torch.int32)
             begin = 1
-            for index, n in enumerate(totals):
-                row_table[index, :n] = torch.arange(begin, begin + n, dtype=torch.int32)
-                begin += n
+            for index, (start, end) in enumerate(spans):
+                row_table[index, start:end] = torch.arange(begin, begin + end - start, dtype=torch.int32)
+                begin += end - start
             packed = torch.cat([req, pos, row_table.view(-1)]).to(q.device, non_blocking=True)
             return (packed[:rows_needed], packed[rows_needed:2 * rows_needed],
                     packed[2 * rows_needed:].view(count, longest), rows_needed)
 
-        src_req, src_pos, row_table, rows_needed = ctx.shared(("carried_up_rows", count), plan)
+        src_req, src_pos, row_table, rows_needed = ctx.shared(("carried_up_rows", count, self.window), plan)
         latents = torch.empty((rows_needed + 1, rank), dtype=q.dtype, device=q.device)
         latents[0].zero_()
         K.gather_cached_rows(plane, table, src_req, src_pos, 0, rank, latents[1:])
@@ -252,7 +260,29 @@ class LatentAttention(Mixer):
         K.attention_dims(queries, carried, carried.view(-1)[d + r:], row_table, K.api._RequestRun(ctx, 0, count),
                          value_heads=heads, group=1, maps=1, key_width=d + r, value_width=v, page_size=1,
                          num_pages=rows_needed + 1, key_strides=strides, value_strides=strides, scale=self.scale,
-                         sink=self.sink_f32, out=out[:tokens])
+                         sink=self.sink_f32, window=self.window, out=out[:tokens])
+
+    def _turned_queries(self, rows, q, kv_rows, ctx, table, plane, cache, first: int, latent_q: torch.Tensor):
+        """Every token's latent row into the cache; the queries of the first ``first`` tokens (long portions) as heads
+        of their own (the unturned part as projected, then the turned part), those of the other tokens carried into
+        the latent space, with the turned part behind, in their rows of ``latent_q``.  Returns the former (or None)."""
+        heads, rank, tokens = self.num_heads, self.kv_rank, rows.shape[0]
+        carried = queries = None
+        if rows.dtype == torch.float32:
+            K.heads_linear(q[:, :, : self.head_dim], self.uk_t, out=latent_q[:, :, :rank])
+        elif first < tokens:
+            carried = K.heads_linear(q[first:, :, : self.head_dim], self.uk_t)
+        rest = ctx if not first else _TokenRange(ctx, first, tokens)
+        if first:
+            queries = torch.empty((first, heads, self.head_dim + self.rot_dim), dtype=rows.dtype, device=rows.device)
+            K.latent_prepare(kv_rows[:first], self.kv_norm_weight, self.eps, self.inv_freq, self.rot_dims,
+                             _TokenRange(ctx, 0, first), table, plane, q[:first], self.head_dim, queries,
+                             q_latent=q[:first, :, : self.head_dim], write=cache.owner)
+        if first < tokens:
+            K.latent_prepare(kv_rows[first:], self.kv_norm_weight, self.eps, self.inv_freq, self.rot_dims, rest,
+                             table, plane, q[first:], self.head_dim, latent_q[first:], q_latent=carried,
+                             write=cache.owner)
+        return queries
 
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
         if self.sink is not None and self.sink_f32 is None:
@@ -267,31 +297,27 @@ class LatentAttention(Mixer):
         long_count = self._long_requests(ctx, rows)
         first = sum(ctx.host_query_lens[:long_count]) if long_count else 0      # tokens of the long portions
         # the attention's queries: the head's query carried into the latent space, then its turned part
-        latent_q = torch.empty((tokens, heads, width), dtype=rows.dtype, device=rows.device)
-        carried = None
-        if rows.dtype == torch.float32:
-            K.heads_linear(q[:, :, : self.head_dim], self.uk_t, out=latent_q[:, :, :rank])
-        elif first < tokens:
-            carried = K.heads_linear(q[first:, :, : self.head_dim], self.uk_t)
-        # every token's latent row goes into the cache here; the long portions' queries stay heads of their
-        # own: the unturned part as projected, then the turned part
-        rest = ctx if not first else _TokenRange(ctx, first, tokens)
-        queries = None
-        if first:
-            queries = torch.empty((first, heads, self.head_dim + self.rot_dim), dtype=rows.dtype, device=rows.device)
-            K.latent_prepare(kv_rows[:first], self.kv_norm_weight, self.eps, self.inv_freq, self.rot_dims,
-                             _TokenRange(ctx, 0, first), table, plane, q[:first], self.head_dim, queries,
-                             q_latent=q[:first, :, : self.head_dim], write=cache.owner)
-        if first < tokens:
-            K.latent_prepare(kv_rows[first:], self.kv_norm_weight, self.eps, self.inv_freq, self.rot_dims, rest,
-                             table, plane, q[first:], self.head_dim, latent_q[first:], q_latent=carried,
-                             write=cache.owner)
+        queries = latent_q = None
+        if not self.rot_dim:
+            if cache.owner:
+                K.latent_cache_write(kv_rows, self.kv_norm_weight, self.eps, ctx, table, plane)
+            queries = q[:first]
+            if not first:
+                latent_q = K.heads_linear(q, self.uk_t)
+            elif first < tokens:                       # rows of the whole step, of which the short portions' are used
+                latent_q = torch.empty((tokens, heads, rank), dtype=rows.dtype, device=rows.device)
+                K.heads_linear(q[first:], self.uk_t, out=latent_q[first:])
+        else:
+            latent_q = torch.empty((tokens, heads, width), dtype=rows.dtype, device=rows.device)
+            queries = self._turned_queries(rows, q, kv_rows, ctx, table, plane, cache, first, latent_q)
         strides = (page * width, 0, width)
         if not first:
             mixed = K.attention_dims(latent_q, plane, plane, table, ctx, value_heads=1, group=heads, maps=1,
                                      key_width=width, value_width=rank, page_size=page, num_pages=num_pages,
-                                     key_strides=strides, value_strides=strides, scale=self.scale, sink=self.sink_f32)
-            out = K.heads_linear(mixed, self.uv)                   # [T, heads, value_dim]
+                                     key_strides=strides, value_strides=strides, scale=self.scale, window=self.window,
+                                     sink=self.sink_f32)
+            out = None if self.g_cols else torch.empty((tokens, heads, self.value_dim), dtype=rows.dtype, device=rows.device)
+            out = K.heads_linear(mixed, self.uv, out=out)          # [T, heads, value_dim]
         else:
             out = torch.empty((tokens, heads, self.value_dim), dtype=rows.dtype, device=rows.device)
             self._attend_carried_up(queries, ctx, table, plane, long_count, out)
@@ -300,7 +326,7 @@ class LatentAttention(Mixer):
                 K.attention_dims(latent_q, plane, plane, table[long_count:], K.api._RequestRun(ctx, long_count, ctx.num_reqs),
                                  value_heads=1, group=heads, maps=1, key_width=width, value_width=rank, page_size=page,
                                  num_pages=num_pages, key_strides=strides, value_strides=strides, scale=self.scale,
-                                 sink=self.sink_f32, out=mixed)
+                                 window=self.window, sink=self.sink_f32, out=mixed)
                 K.heads_linear(mixed[first:], self.uv, out=out[first:])
         if self.g_cols:
             out = K.sigmoid_gate_mul(out, rows[:, self.q_cols + self.kv_cols :])

@@ -13,6 +13,8 @@ none knows the model it sits in.  What each kind must provide:
   fixed-size per-request state; ``None`` if none).  ``cache`` is the ``LayerCache`` of the
   schedule entry being run.
 * **FeedForward**: ``forward(x [T,E], ctx) -> [T,E]``.
+* **StreamStep**: ``forward(h, residual, origin, number, ctx) -> residual``; what is done to the whole stream between
+  two layers (``origin``: the embedded tokens as they entered the stream, 32-bit).
 * **Block**: ``forward(h, residual, ctx, cache) -> (h, residual)``; arranges norms, mixer and
   feed-forward.  ``residual`` is ``None`` before the first block.
 
@@ -193,6 +195,11 @@ class Block(Part):
         raise NotImplementedError
 
 
+class StreamStep(Part):
+    def forward(self, h: Any, residual: torch.Tensor | None, origin: torch.Tensor, number: int, ctx: Any) -> torch.Tensor:
+        raise NotImplementedError
+
+
 class PartFactory(Protocol):
     def __call__(self, *, dtype: torch.dtype, device: torch.device, **params: Any) -> Part: ...
 
@@ -238,6 +245,7 @@ FEED_FORWARDS = PartRegistry("feed-forward")
 BLOCKS = PartRegistry("block")
 EMBEDDINGS = PartRegistry("embedding")
 LM_HEADS = PartRegistry("lm head")
+STREAM_STEPS = PartRegistry("stream step")
 
 
 def collect_slots(parts: Iterable[Part]) -> list[WeightSlot]:
@@ -263,7 +271,9 @@ __all__ = [
     "Part",
     "PartRegistry",
     "PositionEncoding",
+    "STREAM_STEPS",
     "StateSpec",
+    "StreamStep",
     "WeightSlot",
     "collect_slots",
 ]

@@ -1,5 +1,5 @@
-"""Arrangements of one layer: pre-norm mixer and feed-forward in sequence on a deferred residual, side
-by side on a 32-bit stream, or in sequence on a 32-bit stream with a norm on both sides of each.
+"""Arrangements of one layer: pre-norm mixer and feed-forward in sequence on a deferred residual (of the
+activation type, or a 32-bit stream), side by side on a 32-bit stream, or in sequence on a 32-bit stream with a norm on both sides of each.
 
 As the reference's decoder layer (kvcore/model/models/llama3.py:124-142): the running
 ``residual`` and the last sub-layer output ``h`` stay separate and are summed inside the
@@ -70,6 +70,50 @@ class PreNormResidualBlock(Block):
                 x, residual = self.feed_forward_norm.forward_residual(a, residual)
             h = self.feed_forward.forward(x, ctx)
         return h, residual
+
+
+class PreNormStreamBlock(PreNormResidualBlock):
+    """``x <- x + mixer(norm_a(x))``, then ``x <- x + ff(norm_b(x))`` on one 32-bit stream (a layer may have no
+    feed-forward).  A sub-layer's output goes unsummed to the norm behind it, which adds it to the stream and norms
+    the sum in one kernel; the experts of a mixture leave their rows for that kernel to weight and sum.
+
+    In the ``(h, residual)`` pair that runs through the blocks this block returns ``(its last sub-layer's output or
+    its experts' rows, stream)``."""
+
+    takes_expert_rows = True
+
+    def __init__(self, *, layer: LayerSpec, unused_tensors: tuple = (), dtype: torch.dtype, device: torch.device) -> None:
+        self.unused_tensors = tuple(unused_tensors)
+        self.mixer_norm = NORMS.build(layer.norms["mixer_norm"], dtype=dtype, device=device)
+        self.mixer = MIXERS.build(layer.mixer, dtype=dtype, device=device)
+        self.feed_forward = self.feed_forward_norm = None
+        if layer.feed_forward is not None:
+            self.feed_forward_norm = NORMS.build(layer.norms["feed_forward_norm"], dtype=dtype, device=device)
+            self.feed_forward = FEED_FORWARDS.build(layer.feed_forward, dtype=dtype, device=device)
+
+    def parts(self):
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward)
+                     if p is not None)
+
+    def ignorable_tensor_names(self) -> list[str]:
+        return PreNormResidualBlock.ignorable_tensor_names(self) + list(self.unused_tensors)
+
+    def forward(self, h, residual, ctx, cache):
+        if residual is None:                       # the embedded tokens start the stream
+            residual, h = (h if h.dtype == torch.float32 else K.stream_add(h)), Summed(None)
+        elif residual.dtype != torch.float32:      # a block in front kept its stream in the activation type
+            residual = K.stream_add(residual)
+        if isinstance(h, Summed):
+            x = self.mixer_norm.forward(residual)
+        else:
+            x, residual = self.mixer_norm.forward_residual(h, residual)
+        h = self.mixer.forward(x, ctx, cache)
+        if self.feed_forward is None:
+            return h, residual
+        x, residual = self.feed_forward_norm.forward_residual(h, residual)
+        unsummed = getattr(self.feed_forward, "forward_rows", None)
+        h = None if unsummed is None else unsummed(x, ctx)
+        return (self.feed_forward.forward(x, ctx) if h is None else h), residual
 
 
 class ParallelResidualBlock(Block):
@@ -279,7 +323,8 @@ class SandwichResidualBlock(Block):
 
 
 BLOCKS.register("prenorm_residual", PreNormResidualBlock)
+BLOCKS.register("prenorm_stream", PreNormStreamBlock)
 BLOCKS.register("sandwich_residual", SandwichResidualBlock)
 BLOCKS.register("parallel_residual", ParallelResidualBlock)
 
-__all__ = ["ParallelResidualBlock", "PreNormResidualBlock", "SandwichResidualBlock"]
+__all__ = ["ParallelResidualBlock", "PreNormResidualBlock", "PreNormStreamBlock", "SandwichResidualBlock"]

@@ -14,8 +14,9 @@ import torch
 from .. import kernels as K
 from ..config.model_spec import ModelSpec
 from . import (attention, attention_maps, block, embedding, mlp, moe, norm, recurrent, rope,  # noqa: F401
-               side_by_side)                                                                 # (register the stock parts)
-from .base import BLOCKS, EMBEDDINGS, LM_HEADS, NORMS, CacheSpec, StateSpec, Summed, WeightSlot
+               side_by_side, stream_steps)                                                   # (register the stock parts)
+from .base import (BLOCKS, EMBEDDINGS, LM_HEADS, NORMS, STREAM_STEPS, CacheSpec, StateSpec, Summed,
+                   WeightSlot)
 
 
 @dataclass(frozen=True)
@@ -48,6 +49,8 @@ class DecoderModel:
             tied_weight = self.embedding.weight
         self.lm_head = LM_HEADS.build(spec.lm_head, tied_weight=tied_weight, dtype=dtype, device=device)
         self.schedule = spec.schedule
+        self.stream_steps = {name: STREAM_STEPS.build(part, dtype=dtype, device=device)
+                             for name, part in spec.stream_steps.items()}
 
     @property
     def graph_safe(self) -> bool:
@@ -56,7 +59,7 @@ class DecoderModel:
 
     # ---- weights -------------------------------------------------------------------------
     def _parts(self):
-        return [self.embedding, *self.blocks, self.final_norm, self.lm_head]
+        return [self.embedding, *self.blocks, *self.stream_steps.values(), self.final_norm, self.lm_head]
 
     def weight_slots(self) -> list[WeightSlot]:
         slots: list[WeightSlot] = []
@@ -104,21 +107,45 @@ class DecoderModel:
             )
         return out
 
+    def embedding_state_spec(self) -> StateSpec | None:
+        """Per-request state the embedding itself keeps (the token in front, where it reads it)."""
+        spec = getattr(self.embedding, "state_spec", None)
+        return None if spec is None else spec()
+
     # ---- the forward pass of one step --------------------------------------------------------
     def forward(self, ctx, caches) -> tuple[torch.Tensor, torch.Tensor]:
         """Run the step's tokens through every schedule entry; returns ``(h, residual)``."""
-        h = self.embedding.forward(ctx.token_ids)
-        residual = None
+        embed_step = getattr(self.embedding, "forward_step", None)
+        h = self.embedding.forward(ctx.token_ids) if embed_step is None else embed_step(ctx)
+        residual = origin = None
+        if self.stream_steps:
+            # what the stream started as: the blocks add to the stream in place, so it is kept apart from it
+            # (unless a step replaces the stream ahead of the first block)
+            origin = h if h.dtype == torch.float32 else K.stream_add(h)
+            if self.schedule[0].ahead is None:
+                h = origin.clone()
         # per-token inputs of the layers themselves: gathered once, every block reads its own columns
         side_rows = getattr(self.embedding, "side_rows", None)
         if side_rows is not None and getattr(self.embedding, "side_weight", None) is not None:
             ctx.shared("token_side_rows", lambda: side_rows(ctx.token_ids))
         for index, entry in enumerate(self.schedule):
-            h, residual = self.blocks[entry.layer].forward(h, residual, ctx, caches[index])
+            block = self.blocks[entry.layer]
+            if entry.ahead is not None:
+                name, number = entry.ahead
+                residual = self.stream_steps[name].forward(h, residual, origin, number, ctx)
+                h = Summed(None)
+            elif isinstance(h, K.ExpertRows) and not getattr(block, "takes_expert_rows", False):
+                residual, h = K.stream_add_rows(residual, h)[0], Summed(None)
+            h, residual = block.forward(h, residual, ctx, caches[index])
         return h, residual
 
     def compute_logits(self, h: torch.Tensor, residual: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
         """32-bit logits ``[len(rows), V]`` of the token rows ``rows`` (int32 indices)."""
+        forward_rows = getattr(self.final_norm, "forward_rows", None)
+        if forward_rows is not None and residual.dtype == torch.float32 and not isinstance(h, Summed):
+            return self.lm_head.forward(forward_rows(h, residual, rows))
+        if isinstance(h, K.ExpertRows):
+            residual, h = K.stream_add_rows(residual, h)[0], Summed(None)
         residual_rows = K.gather_rows(residual, rows)
         if isinstance(h, Summed):      # the last sub-layer has added its output into the residual itself
             normed = self.final_norm.forward(residual_rows)

@@ -2,7 +2,8 @@
 feed-forwards per token; an optional shared expert runs for every token.
 
     z = router x                      (32-bit logits; the router matrix is kept in 32-bit)
-    s = sigmoid(z)  or  softmax(z)    (``score``)
+    s = sigmoid(z)  or  softmax(z)    (``score``; ``router_bias``: z has a bias ``[experts]``, 32-bit)
+             or ``score="softmax_chosen"``: s = z, and the weights are the softmax over the chosen logits alone
     chosen = the top_k largest s; weights = their s, divided by their sum if ``renormalize``
              ``choice_correction``: the choice goes by ``s + c`` with a tensor ``c [experts]``, the weights stay
              the chosen experts' ``s``; ``group_count`` / ``group_keep``: the experts form ``group_count`` equal
@@ -12,7 +13,8 @@ feed-forwards per token; an optional shared expert runs for every token.
                          or   w_e * expert_e(x)        (``weight_on="output"``)
     y += sigmoid(g . x) * shared(x)   (``shared`` given; ``shared_gate`` False: plain sum)
 
-    expert(a) = down(silu(gate a) * (up a)), no biases.
+    expert(a) = down(silu(gate a) * (up a)), no biases; or with ``join = (alpha, limit, shift)``
+                down(g * sigmoid(alpha g) * (u + shift)), g = min(gate a, limit), u = clamp(up a, -limit, limit)
 
 The experts' matrices are stacked ``[E, 2F, K]`` (gate rows, then up rows) and ``[E, K, F]``; the
 (token, expert) pairs are grouped by expert on the device and the two products run as grouped
@@ -30,7 +32,7 @@ from .base import FEED_FORWARDS, FeedForward, WeightSlot
 
 class RoutedExperts(FeedForward):
     DEFAULT_TENSOR_NAMES = {
-        "router": "router", "shared_gate": "shared_gate", "correction": "correction",
+        "router": "router", "router_bias": "router.b", "shared_gate": "shared_gate", "correction": "correction",
         # expert tensors: formatted with the expert's index
         "gate": "experts.{index}.gate_proj.weight", "up": "experts.{index}.up_proj.weight",
         "down": "experts.{index}.down_proj.weight",
@@ -40,12 +42,13 @@ class RoutedExperts(FeedForward):
                  score: str = "sigmoid", renormalize: bool = False, weight_on: str = "input",
                  shared: PartSpec | None = None, shared_gate: bool = False, weight_scale: float = 1.0,
                  choice_correction: bool = False, group_count: int = 1, group_keep: int = 1,
+                 router_bias: bool = False, join: tuple | None = None,
                  tensor_names: dict | None = None, dtype: torch.dtype, device: torch.device) -> None:
         self.hidden_size, self.num_experts = int(hidden_size), int(num_experts)
         self.top_k, self.expert_size = int(top_k), int(expert_size)
         if not 0 < self.top_k <= self.num_experts:
             raise ValueError(f"top_k {top_k} must lie in [1, num_experts {num_experts}]")
-        if score not in ("sigmoid", "softmax"):
+        if score not in ("sigmoid", "softmax", "softmax_chosen"):
             raise ValueError(f"unknown router score {score!r}")
         if weight_on not in ("input", "output"):
             raise ValueError(f"weight_on must be 'input' or 'output', got {weight_on!r}")
@@ -54,12 +57,16 @@ class RoutedExperts(FeedForward):
         if (self.group_count <= 0 or self.num_experts % self.group_count or not 0 < self.group_keep <= self.group_count
                 or self.group_keep * (self.num_experts // self.group_count) < self.top_k):
             raise ValueError(f"{group_keep} of {group_count} equal groups of {num_experts} experts must hold top_k {top_k}")
+        if join is not None and (len(join) != 3 or not join[1] > 0):
+            raise ValueError(f"join is (alpha, limit, shift) with a positive limit, got {join!r}")
+        self.join = None if join is None else tuple(float(v) for v in join)
         self.name = name
         self.tensor_names = dict(self.DEFAULT_TENSOR_NAMES)
         self.tensor_names.update(tensor_names or {})
         experts, ff, hidden = self.num_experts, self.expert_size, self.hidden_size
         self.router_weight = torch.empty(experts, hidden, dtype=torch.float32, device=device)
         self.correction = torch.empty(experts, dtype=torch.float32, device=device) if choice_correction else None
+        self.router_bias = torch.empty(experts, dtype=torch.float32, device=device) if router_bias else None
         self.gate_up_weight = torch.empty(experts, 2 * ff, hidden, dtype=dtype, device=device)
         self.down_weight = torch.empty(experts, hidden, ff, dtype=dtype, device=device)
         self.shared = None if shared is None else FEED_FORWARDS.build(shared, dtype=dtype, device=device)
@@ -78,6 +85,8 @@ class RoutedExperts(FeedForward):
     def weight_slots(self) -> list[WeightSlot]:
         ff = self.expert_size
         slots = [WeightSlot(self._tensor("router"), self.router_weight)]
+        if self.router_bias is not None:
+            slots.append(WeightSlot(self._tensor("router_bias"), self.router_bias, init="zeros"))
         if self.correction is not None:
             slots.append(WeightSlot(self._tensor("correction"), self.correction, init="zeros"))
         for e in range(self.num_experts):
@@ -106,16 +115,24 @@ class RoutedExperts(FeedForward):
         routed = K.moe_route(x, self.router_weight, self.top_k, score=self.score,
                              renormalize=self.renormalize, gate_rows=self.shared_gate_weight,
                              correction=self.correction, group_count=self.group_count, group_keep=self.group_keep,
-                             weight_scale=self.weight_scale)
+                             weight_scale=self.weight_scale, bias=self.router_bias)
         grouping = None
         if K.moe_path(x, x.shape[0] * self.top_k, self.expert_size) == "library":
             grouping = K.moe_group(routed[0], self.num_experts, for_library=True)
         return routed, grouping
 
-    def forward(self, x: torch.Tensor, ctx, prepared=None) -> torch.Tensor:
+    def _expert_rows(self, x: torch.Tensor, ctx, prepared):
         (ids, weights, gates), grouping = prepared if prepared is not None else self.prepare(x, ctx)
-        pairs = K.moe_experts(x, ids, weights, self.gate_up_weight, self.down_weight,
-                              weight_on_input=self.weight_on == "input", grouping=grouping)
+        return gates, K.moe_experts(x, ids, weights, self.gate_up_weight, self.down_weight,
+                                    weight_on_input=self.weight_on == "input", grouping=grouping, join=self.join)
+
+    def forward_rows(self, x: torch.Tensor, ctx):
+        """The chosen experts' rows, for a block whose next norm weights and sums them into the stream (None: a
+        shared expert wants a sum of its own)."""
+        return None if self.shared is not None else self._expert_rows(x, ctx, None)[1]
+
+    def forward(self, x: torch.Tensor, ctx, prepared=None) -> torch.Tensor:
+        gates, pairs = self._expert_rows(x, ctx, prepared)
         shared = None if self.shared is None else self.shared.forward(x, ctx)
         return K.moe_combine(pairs, x.shape[0], self.top_k, shared, gates)
 

@@ -107,9 +107,18 @@ class RMSNormStream(Norm):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         return K.rms_norm_shift(x, self.weight, self.eps, self.dtype)
 
-    def forward_residual(self, h: torch.Tensor, residual: torch.Tensor):
-        residual = K.stream_add(residual, h) if residual.dtype == torch.float32 else residual.add_(h)
-        return self.forward(residual), residual
+    def forward_residual(self, h, residual: torch.Tensor):
+        """``h``: a sub-layer's output, or the rows its experts left (``ExpertRows``, a 32-bit stream only)."""
+        if residual.dtype != torch.float32:
+            residual = residual.add_(h)
+            return self.forward(residual), residual
+        residual, y, _ = K.stream_add_rows(residual, h, weight=self.weight, eps=self.eps, out_dtype=self.dtype)
+        return y, residual
+
+    def forward_rows(self, h, residual: torch.Tensor, token_rows: torch.Tensor) -> torch.Tensor:
+        """``norm(residual + h)`` of some tokens of a 32-bit stream, which stays as it is."""
+        return K.stream_add_rows(residual, h, weight=self.weight, eps=self.eps, out_dtype=self.dtype,
+                                 token_rows=token_rows)[1]
 
     def as_rms_scale(self):
         return self.weight, self.eps

@@ -21,6 +21,12 @@ convolution.  Both mixers keep ``S`` column by column (``[heads, value_dim, head
 ``a`` a head (a constant of the model) and ``q``, ``k``, ``v`` passed through SiLU; the heads' read-outs are
 RMS-normed together (one weight over all heads' values) and multiplied by ``sigmoid(W_g x)``.
 
+``SelectiveStateSpace`` (the second Mamba's mixer): one projection gives ``[z | x | B | C | step sizes]``; x, B and C
+pass a short causal convolution with a bias and SiLU; ``dt = softplus(step + dt_bias)``; per head (a group of heads
+shares B and C) ``S <- exp(-exp(A_log) dt) S + dt B x^T``, ``y = S^T C + D x``; y times ``silu(z)`` is RMS-normed in
+``norm_groups`` equal parts of all heads' values.  The state of a request is ``S`` and the last ``taps - 1`` inputs of
+the convolution.
+
 Decays, step sizes, unit norms, the state, the read-out and the norm behind it are 32-bit whatever the
 activation type.
 """
@@ -249,8 +255,72 @@ class LightningAttention(ProjectedMixer):
                          out, scale, gate_act="sigmoid")
 
 
+class SelectiveStateSpace(ProjectedMixer):
+    graph_safe = True
+
+    DEFAULT_TENSOR_NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "A_log": "A_log",
+                            "D": "D", "norm": "norm", "o": "o"}
+
+    def __init__(self, *, hidden_size: int, num_heads: int, num_groups: int, state_dim: int, value_dim: int,
+                 conv_taps: int, norm_groups: int, eps: float, name: str, tensor_names: dict | None = None,
+                 dtype: torch.dtype, device: torch.device) -> None:
+        if min(num_heads, num_groups, state_dim, value_dim) <= 0 or num_heads % num_groups:
+            raise ValueError(f"num_heads {num_heads} must be a positive multiple of num_groups {num_groups}")
+        if norm_groups <= 0 or (num_heads * value_dim) % norm_groups:
+            raise ValueError(f"{num_heads} x {value_dim} values do not fall into {norm_groups} equal parts")
+        if not 1 <= conv_taps <= 9:
+            raise ValueError(f"the short convolution has 1 to 9 taps, got {conv_taps}")
+        if state_dim > 512:
+            raise ValueError(f"state_dim {state_dim} exceeds the state kernel's 512 key channels")
+        self.hidden_size, self.num_heads, self.num_groups = int(hidden_size), int(num_heads), int(num_groups)
+        self.state_dim, self.value_dim, self.conv_taps = int(state_dim), int(value_dim), int(conv_taps)
+        self.norm_groups, self.eps, self.name = int(norm_groups), float(eps), name
+        self.tensor_names = dict(self.DEFAULT_TENSOR_NAMES)
+        self.tensor_names.update(tensor_names or {})
+        self.inner = self.num_heads * self.value_dim
+        self.channels = self.inner + 2 * self.num_groups * self.state_dim      # what passes the convolution: x, B, C
+        self.projected = self.inner + self.channels + self.num_heads           # z, the channels, the step sizes
+        self.in_rows = _round8(self.projected)
+        self.out_cols = self.inner
+        self._allocate(dtype, device)
+        f32 = dict(dtype=torch.float32, device=device)
+        self.taps = torch.empty(self.channels, self.conv_taps, **f32)
+        self.conv_bias = torch.empty(self.channels, **f32)
+        self.dt_bias, self.a_log, self.skip = (torch.empty(self.num_heads, **f32) for _ in range(3))
+        self.norm_weight = torch.empty(self.inner, **f32)
+        self.matrix_floats = _round4(self.num_heads * self.state_dim * self.value_dim)
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec((_round4(self.matrix_floats + self.channels * (self.conv_taps - 1)),), torch.float32)
+
+    def _tensor(self, key: str) -> str:
+        return f"{self.name}.{self.tensor_names[key]}"
+
+    def weight_slots(self) -> list[WeightSlot]:
+        return [
+            WeightSlot(self._tensor("in"), self.in_weight[:self.projected]),
+            WeightSlot(self._tensor("conv"), self.taps),
+            WeightSlot(self._tensor("conv_bias"), self.conv_bias, init="zeros"),
+            WeightSlot(self._tensor("dt_bias"), self.dt_bias, init="zeros"),
+            WeightSlot(self._tensor("A_log"), self.a_log, init="zeros"),
+            WeightSlot(self._tensor("D"), self.skip, init="ones"),
+            WeightSlot(self._tensor("norm"), self.norm_weight, init="ones"),
+            WeightSlot(self._tensor("o"), self.o_weight),
+        ]
+
+    def mix_rows(self, rows, ctx, cache, out, scale: float = 1.0) -> None:
+        if scale != 1.0:
+            raise ValueError(f"{self.name}: the norm behind the state-space read-out takes no factor")
+        sizes = dict(heads=self.num_heads, groups=self.num_groups, dim=self.state_dim, value_dim=self.value_dim)
+        prepared = K.ssm_prepare(rows[:, self.inner:], self.taps, self.conv_bias, cache.state, ctx, self.a_log,
+                                 self.dt_bias, state_offset=self.state_offset + self.matrix_floats, **sizes)
+        o = K.ssm_scan(prepared, self.skip, cache.state, ctx, state_offset=self.state_offset, **sizes)
+        K.gated_group_norm(o, rows[:, :self.inner], self.norm_weight, self.eps, out, self.norm_groups)
+
+
+MIXERS.register("selective_state_space", SelectiveStateSpace)
 MIXERS.register("gated_linear_attention", GatedLinearAttention)
 MIXERS.register("lightning_attention", LightningAttention)
 MIXERS.register("gated_delta_rule", GatedDeltaRule)
 
-__all__ = ["GatedDeltaRule", "GatedLinearAttention", "LightningAttention", "ProjectedMixer"]
+__all__ = ["GatedDeltaRule", "GatedLinearAttention", "LightningAttention", "ProjectedMixer", "SelectiveStateSpace"]

@@ -207,6 +207,51 @@ def stream_add_norm(x, a, weight, eps, *, out=None, stack=None, depth=0, coeffs=
     return out, avg
 
 
+def stream_add_rows(x, a, *, weight=None, eps=0.0, out_dtype=None, token_rows=None, origin=None, keep=True):
+    tokens, width = x.shape
+    total = x
+    if a is not None:
+        if hasattr(a, "rows"):                      # the rows of the chosen experts, as the product hands them on
+            pairs = a.rows.float()
+            if a.row_of_pair is not None:
+                pairs = pairs[a.row_of_pair.long()]
+            if a.pending_weights is not None:
+                pairs = pairs * a.pending_weights.reshape(-1, 1)
+        else:
+            pairs = a.float()
+        total = x + pairs.reshape(tokens, -1, width).sum(1)
+    dtype = out_dtype or (a.rows if hasattr(a, "rows") else a).dtype
+    keep = keep and token_rows is None and a is not None
+    if keep:
+        total = x.copy_(total)
+    picked = slice(None) if token_rows is None else token_rows.long()
+    normed = None if weight is None else (_rms(total[picked], eps) * weight.float()).to(dtype)
+    packed = None if origin is None else torch.cat([total[picked], origin[picked]], 1).to(dtype)
+    return (x if keep else None), normed, packed
+
+
+def embed_pairs(table, ids, *, pairs=None, mul_prev=0, mul_cur=0, weight=None, eps=0.0, state=None, ctx=None):
+    x = table[ids.long()].float()
+    if pairs is not None:
+        buckets = pairs.shape[0] - 1
+        starts = [int(v) for v in ctx.query_start]
+        rows = []
+        for r in range(ctx.num_reqs):
+            slot = int(ctx.state_slots[r])
+            before = int(state[slot, 0])
+            for t in range(starts[r], starts[r + 1]):
+                token = int(ids[t])
+                rows.append((before * mul_prev + token * mul_cur) % buckets if int(ctx.positions[t]) > 0 else buckets)
+                before = token
+            state[slot, 0] = before
+        x = x + pairs[torch.tensor(rows, device=pairs.device)].float()
+    return x if weight is None else _rms(x, eps) * weight
+
+
+def softcap(logits, scale, cap):
+    return logits.copy_(cap * torch.tanh(logits * scale / cap))
+
+
 def gelu_mul(z, rows, column):
     zf = z.float()
     gelu = 0.5 * zf * (1.0 + torch.tanh(0.7978845608028654 * (zf + 0.044715 * zf ** 3)))
@@ -282,6 +327,16 @@ def latent_prepare(kv_rows, norm_weight, eps, inv_freq, dims, ctx, table, cache,
         q_out[t, :, lead:] = turn(q[t, :, q_width:].float(), pos).to(q_out.dtype)
         if q_latent is not None:
             q_out[t, :, :lead] = q_latent[t]
+
+
+def latent_cache_write(kv_rows, norm_weight, eps, ctx, table, cache):
+    page_size = cache.shape[2]
+    normed = (_rms(kv_rows, eps) * norm_weight.float()).to(cache.dtype)
+    for t in range(kv_rows.shape[0]):
+        pos = int(ctx.positions[t])
+        page = int(table[int(ctx.req_index[t]), pos // page_size])
+        assert page > 0, "write through the null page"
+        cache[page, 0, pos % page_size] = normed[t]
 
 
 def gather_cached_rows(cache, table, src_req, src_pos, col0, cols, out, *, copies=1, head_stride=0):
@@ -378,9 +433,11 @@ def glu_clamped(gate_up, *, alpha, limit, shift):
 
 
 def moe_route(x, router, top, *, score="sigmoid", renormalize=False, gate_rows=None, correction=None,
-              group_count=1, group_keep=1, weight_scale=1.0):
+              group_count=1, group_keep=1, weight_scale=1.0, bias=None):
     z = x.float() @ router.float().T
-    scores = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, dim=-1)
+    if bias is not None:
+        z = z + bias.float()
+    scores = {"sigmoid": torch.sigmoid(z), "softmax": torch.softmax(z, dim=-1), "softmax_chosen": z}[score]
     tokens, experts = scores.shape
     ids = torch.empty(tokens, top, dtype=torch.int32, device=x.device)
     weights = torch.empty(tokens, top, dtype=torch.float32, device=x.device)
@@ -401,7 +458,9 @@ def moe_route(x, router, top, *, score="sigmoid", renormalize=False, gate_rows=N
         ids[:, slot] = index
         weights[:, slot] = scores[rows, index]
         left[rows, index] = -float("inf")
-    if renormalize:
+    if score == "softmax_chosen":
+        weights = torch.softmax(weights, -1)
+    elif renormalize:
         weights = weights / weights.sum(-1, keepdim=True)
     weights = weights * weight_scale
     gates = None if gate_rows is None else torch.sigmoid(x.float() @ gate_rows.float().T)
@@ -412,7 +471,7 @@ def moe_path(x, pairs, ff):
     return "tiles"
 
 
-def moe_experts(x, ids, weights, gate_up, down, *, weight_on_input, path=None, grouping=None):
+def moe_experts(x, ids, weights, gate_up, down, *, weight_on_input, path=None, grouping=None, join=None):
     tokens, top = ids.shape
     ff = gate_up.shape[1] // 2
     out = torch.empty(tokens * top, down.shape[1], dtype=x.dtype, device=x.device)
@@ -422,7 +481,12 @@ def moe_experts(x, ids, weights, gate_up, down, *, weight_on_input, path=None, g
             a = (w * x[t].float()).to(x.dtype).float() if weight_on_input else x[t].float()
             g = (gate_up[e, :ff].float() @ a).to(x.dtype).float()
             u = (gate_up[e, ff:].float() @ a).to(x.dtype).float()
-            hidden = ((g * torch.sigmoid(g)).to(x.dtype).float() * u).to(x.dtype).float()
+            if join is None:
+                hidden = ((g * torch.sigmoid(g)).to(x.dtype).float() * u).to(x.dtype).float()
+            else:
+                alpha, limit, shift = join
+                g, u = g.clamp(max=limit), u.clamp(min=-limit, max=limit)
+                hidden = (g * torch.sigmoid(alpha * g) * (u + shift)).to(x.dtype).float()
             if not weight_on_input:
                 hidden = (w * hidden).to(x.dtype).float()
             out[t * top + s] = (down[e].float() @ hidden).to(x.dtype)
@@ -607,6 +671,53 @@ def gated_rms_norm(o, gate, weight, eps, out, scale=1.0, *, gate_act="silu"):
     return out
 
 
+def ssm_prepare(rows, taps, bias, state, ctx, a_log, dt_bias, *, heads, groups, dim, value_dim, state_offset):
+    inner, gn = heads * value_dim, groups * dim
+    channels, num_taps = taps.shape
+    keep = num_taps - 1
+    x = rows[:, :channels].float()
+    out = torch.zeros((rows.shape[0], (channels + 2 * heads + 3) // 4 * 4), dtype=torch.float32, device=rows.device)
+    for _, begin, end, slot in _request_ranges(ctx):
+        held = state[slot, state_offset:state_offset + channels * keep].reshape(keep, channels)
+        history = torch.cat([held.clone(), x[begin:end]])
+        acc = bias.repeat(end - begin, 1)
+        for j in range(num_taps):
+            acc = acc + history[j:j + end - begin] * taps[:, j]
+        y = acc * torch.sigmoid(acc)
+        out[begin:end, :2 * gn], out[begin:end, 2 * gn:channels] = y[:, inner:], y[:, :inner]
+        if keep:
+            state[slot, state_offset:state_offset + channels * keep] = history[-keep:].reshape(-1)
+    dt = torch.nn.functional.softplus(rows[:, channels:channels + heads].float() + dt_bias, threshold=1e6)
+    out[:, channels:channels + heads] = dt
+    out[:, channels + heads:channels + 2 * heads] = torch.exp(-torch.exp(a_log) * dt)
+    return out
+
+
+def ssm_scan(prepared, skip, state, ctx, *, heads, groups, dim, value_dim, state_offset=0):
+    tokens, gn, n = prepared.shape[0], groups * dim, heads * dim * value_dim
+    share = torch.arange(heads, device=prepared.device) // (heads // groups)
+    B = prepared[:, :gn].reshape(tokens, groups, dim)[:, share]
+    C = prepared[:, gn:2 * gn].reshape(tokens, groups, dim)[:, share]
+    x = prepared[:, 2 * gn:2 * gn + heads * value_dim].reshape(tokens, heads, value_dim)
+    dt, decay = prepared[:, 2 * gn + heads * value_dim:][:, :2 * heads].split(heads, 1)
+    out = torch.empty((tokens, heads, value_dim), dtype=torch.float32, device=prepared.device)
+    for _, begin, end, slot in _request_ranges(ctx):
+        S = state[slot, state_offset:state_offset + n].reshape(heads, value_dim, dim).transpose(1, 2).clone()   # kept column by column
+        for t in range(begin, end):
+            S = S * decay[t][:, None, None] + B[t][:, :, None] * (dt[t][:, None] * x[t])[:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S, C[t]) + skip[:, None] * x[t]
+        state[slot, state_offset:state_offset + n] = S.transpose(1, 2).reshape(n)
+    return out
+
+
+def gated_group_norm(o, gate, weight, eps, out, groups):
+    tokens, width = gate.shape
+    g = gate.float()
+    v = (o.reshape(tokens, width) * g * torch.sigmoid(g)).reshape(tokens, groups, width // groups)
+    out.copy_((_rms(v, eps).reshape(tokens, width) * weight).to(out.dtype))
+    return out
+
+
 # ---- sampling: the same counter-based noise as the CUDA kernel --------------------------------
 def philox4x32_10(counter, key):
     c = [np.uint64(x) for x in counter]
@@ -666,6 +777,7 @@ _NAMES = [
     "rms_norm_shift", "stream_add_norm", "attention_dims", "latent_prepare", "head_norm_kv_write", "maps_combine",
     "sigmoid_gate_mul", "heads_linear", "gather_cached_rows",
     "embed_scaled", "turn_norm_kv_write", "head_gate", "gla_scan", "conv_prepare", "delta_scan", "gated_rms_norm",
+    "latent_cache_write", "stream_add_rows", "embed_pairs", "softcap", "ssm_prepare", "ssm_scan", "gated_group_norm",
     "lightning_scan", "gelu_mul", "layer_norm", "stream_add", "qk_prepare", "glu_clamped", "moe_route", "moe_experts", "moe_combine", "moe_path",
 ]
 
