@@ -696,6 +696,26 @@ def rubuvik_config(size: dict, kinds: str) -> dict:
             "embedding": {"scale": 24.0}, "residual_mult": 0.6, "token_side": {"dim": 256}, "layers": layers}
 
 
+def mamevik_config(size: dict, kinds: str, loop: tuple[int, int, int]) -> dict:
+    """A Mamevik config.json.  ``kinds``: a letter per layer, "s" the selective state space (an inner width of the
+    stream's, heads of 64 values, a state of 128, eight groups, four taps), "l" latent attention (Llama's heads, a
+    latent of 512, a window of 1,024).  Every layer has a mixture of experts without a shared one (chosen experts
+    together as wide as Llama's feed-forward).  ``loop``: start, stop, times."""
+    moe = {"kind": "moe", "expert": {"ff": size["ff"] // size["top"], "limit": 7.0},
+           "router": {"experts": size["experts"], "top": size["top"]}}
+    layers = []
+    for kind in kinds:
+        if kind == "s":
+            mixer = {"heads": size["width"] // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+        else:
+            mixer = {"heads": size["heads"], "dim": size["dim"], "vdim": size["dim"], "kv_rank": 512,
+                     "scale": size["dim"] ** -0.5, "mask": {"size": 1024}}
+        layers.append({"type": "mamba2" if kind == "s" else "latent_attention", "mixer": mixer, "mlp": moe})
+    return {"architecture": "Mamevik", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5},
+            "embedding": {"bigram": {"buckets": size["vocab"] - 1, "mul_prev": 31, "mul_cur": 17}}, "layers": layers,
+            "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]}, "logit_scale": 0.25, "logit_softcap": 30.0}
+
+
 def llama_config(size: dict) -> dict:
     return dict(LLAMA_31_8B, hidden_size=size["width"], intermediate_size=size["ff"], num_hidden_layers=DESIGN_LAYERS,
                 num_attention_heads=size["heads"], num_key_value_heads=size["kv_heads"], head_dim=size["dim"],
@@ -754,6 +774,15 @@ def compare_designs(args) -> int:
                 "rubuvik_attention": rubuvik_config(size, "ab"),
                 "rubuvik_moe": rubuvik_config(size, "m"),
                 "rubuvik_mixed": rubuvik_config(size, "lmbl"),
+            })
+        elif args.designs_of == "mamevik":
+            models.update({
+                "dutivik_linear": dutivik_config(size, "g"),
+                "pipesun_latent": pipesun_config(size, "l"),
+                "rubuvik_moe": rubuvik_config(size, "m"),
+                "mamevik_state": mamevik_config(size, "ssss", (0, 4, 1)),
+                "mamevik_latent": mamevik_config(size, "llll", (0, 4, 1)),
+                "mamevik_mixed": mamevik_config(size, "sll", (1, 2, 2)),      # one layer twice: four runs
             })
         elif args.designs_of == "dutivik":
             models.update({
@@ -837,7 +866,7 @@ def main() -> int:
     parser.add_argument("--designs", action="store_true",
                         help="instead: Toposun (dense and mixture feed-forward) beside a Llama of equal layer sizes, "
                              "prefill and decode throughput and each kernel's share of a step; prints a line of its own")
-    parser.add_argument("--designs-of", default="toposun", choices=["toposun", "pipesun", "dutivik", "rubuvik"],
+    parser.add_argument("--designs-of", default="toposun", choices=["toposun", "pipesun", "dutivik", "rubuvik", "mamevik"],
                         help="which design --designs sets beside Llama")
     parser.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES), help="one size of --designs")
     args = parser.parse_args()
