@@ -17,12 +17,14 @@
 
 #define SSM_THREADS 128
 #define SSM_RUN 16             // tokens a thread walks
+#define SSM_AHEAD 4            // of which it loads this many at once
 #define SSM_MAX_TAPS 9
 
 template <typename T, int N>
 struct __align__(N * sizeof(T)) SsmPiece { T v[N]; };
 
-__device__ __forceinline__ float ssm_silu(float x) { return x / (1.0f + expf(-x)); }
+// (where exp(-x) runs out of range, x below -88, the quotient is a zero: what is lost is smaller than 1e-36)
+__device__ __forceinline__ float ssm_silu(float x) { return __fdividef(x, 1.0f + expf(-x)); }
 
 // N channels a thread; K: taps the window is made for (the model's taps, right-aligned; the places in front are zero).
 template <typename T, int N, int K>
@@ -60,52 +62,63 @@ ssm_prepare_kernel(float* __restrict__ out, long long out_stride, const T* __res
   }
   // x goes behind B and C
   float* o = out + (c < x_channels ? bc + c : c - x_channels);
-  for (int t = t_begin; t < t_end; ++t) {
-    const int req = req_index[t], back = t - query_start[req];
-    if (t == t_begin || back == 0) {
-      const float* held = state + (size_t)state_slots[req] * state_stride + state_offset + c;
+  const T* src = rows + c;
+  int end = t_begin;                                 // where the request of the token in hand ends
+  float* held = nullptr;
+  for (int t0 = t_begin; t0 < t_end; t0 += SSM_AHEAD) {
+    SsmPiece<T, N> in[SSM_AHEAD];                    // a few tokens' loads in flight together
 #pragma unroll
-      for (int j = 0; j < K - 1; ++j) {
-        const int ago = K - 1 - j;                   // window[j] is the input `ago` tokens back
-        if (ago > keep) {
+    for (int u = 0; u < SSM_AHEAD; ++u)
+      if (t0 + u < t_end) in[u] = *reinterpret_cast<const SsmPiece<T, N>*>(src + (size_t)(t0 + u) * row_stride);
 #pragma unroll
-          for (int i = 0; i < N; ++i) window[j][i] = 0.0f;
-        } else if (ago <= back) {
-          const SsmPiece<T, N> in = *reinterpret_cast<const SsmPiece<T, N>*>(rows + (size_t)(t - ago) * row_stride + c);
+    for (int u = 0; u < SSM_AHEAD; ++u) {
+      const int t = t0 + u;
+      if (t >= t_end) break;
+      if (t == end) {                                // the run's first token, or a portion's
+        const int req = req_index[t], back = t - query_start[req];
+        end = query_start[req + 1];
+        held = state + (size_t)state_slots[req] * state_stride + state_offset + c;
 #pragma unroll
-          for (int i = 0; i < N; ++i) window[j][i] = to_float(in.v[i]);
-        } else {
-          const SsmPiece<float, N> in = *reinterpret_cast<const SsmPiece<float, N>*>(held + (size_t)(keep - (ago - back)) * channels);
+        for (int j = 0; j < K - 1; ++j) {
+          const int ago = K - 1 - j;                 // window[j] is the input `ago` tokens back
+          if (ago > keep) {
 #pragma unroll
-          for (int i = 0; i < N; ++i) window[j][i] = in.v[i];
+            for (int i = 0; i < N; ++i) window[j][i] = 0.0f;
+          } else if (ago <= back) {
+            const SsmPiece<T, N> was = *reinterpret_cast<const SsmPiece<T, N>*>(src + (size_t)(t - ago) * row_stride);
+#pragma unroll
+            for (int i = 0; i < N; ++i) window[j][i] = to_float(was.v[i]);
+          } else {
+            const SsmPiece<float, N> was = *reinterpret_cast<const SsmPiece<float, N>*>(held + (size_t)(keep - (ago - back)) * channels);
+#pragma unroll
+            for (int i = 0; i < N; ++i) window[j][i] = was.v[i];
+          }
         }
       }
-    }
-    const SsmPiece<T, N> in = *reinterpret_cast<const SsmPiece<T, N>*>(rows + (size_t)t * row_stride + c);
-    SsmPiece<float, N> y;
+      SsmPiece<float, N> y;
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-      float acc = b[i];
+      for (int i = 0; i < N; ++i) {
+        float acc = b[i];
 #pragma unroll
-      for (int j = 0; j < K - 1; ++j) acc = fmaf(w[j][i], window[j][i], acc);
-      const float x = to_float(in.v[i]);
-      acc = fmaf(w[K - 1][i], x, acc);
-      y.v[i] = ssm_silu(acc);
+        for (int j = 0; j < K - 1; ++j) acc = fmaf(w[j][i], window[j][i], acc);
+        const float x = to_float(in[u].v[i]);
+        acc = fmaf(w[K - 1][i], x, acc);
+        y.v[i] = ssm_silu(acc);
 #pragma unroll
-      for (int j = 0; j + 1 < K - 1; ++j) window[j][i] = window[j + 1][i];
-      window[K - 2][i] = x;
-    }
-    *reinterpret_cast<SsmPiece<float, N>*>(o + (size_t)t * out_stride) = y;
-    if (single) {                                    // one token a request: nobody else reads what was held
-      float* held = state + (size_t)state_slots[req] * state_stride + state_offset + c;
+        for (int j = 0; j + 1 < K - 1; ++j) window[j][i] = window[j + 1][i];
+        window[K - 2][i] = x;
+      }
+      *reinterpret_cast<SsmPiece<float, N>*>(o + (size_t)t * out_stride) = y;
+      if (single) {                                  // one token a request: nobody else reads what was held
 #pragma unroll
-      for (int j = 0; j < K - 1; ++j) {
-        const int place = j - (K - num_taps);
-        if (place >= 0) {
-          SsmPiece<float, N> moved;
+        for (int j = 0; j < K - 1; ++j) {
+          const int place = j - (K - num_taps);
+          if (place >= 0) {
+            SsmPiece<float, N> moved;
 #pragma unroll
-          for (int i = 0; i < N; ++i) moved.v[i] = window[j][i];
-          *reinterpret_cast<SsmPiece<float, N>*>(held + (size_t)place * channels) = moved;
+            for (int i = 0; i < N; ++i) moved.v[i] = window[j][i];
+            *reinterpret_cast<SsmPiece<float, N>*>(held + (size_t)place * channels) = moved;
+          }
         }
       }
     }
@@ -232,12 +245,24 @@ gated_group_norm_kernel(T* __restrict__ out, long long out_stride, const float* 
     for (int j = 0; j < N; ++j) v[j] = a.v[j] * ssm_silu(to_float(z.v[j]));
   };
   float kept[GN_PIECES][N];
+  SsmPiece<float, N> as[GN_PIECES], ws[GN_PIECES];
+  SsmPiece<T, N> zs[GN_PIECES];
   float ss = 0.0f;
+#pragma unroll
+  for (int s = 0; s < GN_PIECES; ++s) {              // every load of the kept pieces in flight together
+    const int i = (lane + s * lanes) * N;
+    if (i < width) {
+      as[s] = *reinterpret_cast<const SsmPiece<float, N>*>(src + i);
+      zs[s] = *reinterpret_cast<const SsmPiece<T, N>*>(g + i);
+      ws[s] = *reinterpret_cast<const SsmPiece<float, N>*>(wt + i);
+    }
+  }
 #pragma unroll
   for (int s = 0; s < GN_PIECES; ++s) {
     const int i = (lane + s * lanes) * N;
     if (i < width) {
-      gated(i, kept[s]);
+#pragma unroll
+      for (int j = 0; j < N; ++j) kept[s][j] = as[s].v[j] * ssm_silu(to_float(zs[s].v[j]));
 #pragma unroll
       for (int j = 0; j < N; ++j) ss = fmaf(kept[s][j], kept[s][j], ss);
     }
@@ -249,8 +274,7 @@ gated_group_norm_kernel(T* __restrict__ out, long long out_stride, const float* 
     for (int j = 0; j < N; ++j) ss = fmaf(v[j], v[j], ss);
   }
   const float inv = 1.0f / sqrtf((WARP ? warp_sum(ss) : block_sum(ss, scratch)) / (float)width + eps);
-  auto put = [&](int i, const float (&v)[N]) {
-    const SsmPiece<float, N> w = *reinterpret_cast<const SsmPiece<float, N>*>(wt + i);
+  auto put = [&](int i, const float (&v)[N], const SsmPiece<float, N>& w) {
     SsmPiece<T, N> r;
 #pragma unroll
     for (int j = 0; j < N; ++j) r.v[j] = from_float<T>(v[j] * inv * w.v[j]);
@@ -259,12 +283,12 @@ gated_group_norm_kernel(T* __restrict__ out, long long out_stride, const float* 
 #pragma unroll
   for (int s = 0; s < GN_PIECES; ++s) {
     const int i = (lane + s * lanes) * N;
-    if (i < width) put(i, kept[s]);
+    if (i < width) put(i, kept[s], ws[s]);
   }
   for (int i = (lane + GN_PIECES * lanes) * N; i < width; i += lanes * N) {
     float v[N];
     gated(i, v);
-    put(i, v);
+    put(i, v, *reinterpret_cast<const SsmPiece<float, N>*>(wt + i));
   }
 }
 

@@ -1,7 +1,7 @@
 // Kernels of a model that keeps a 32-bit residual stream and leaves a sub-layer's output to the norm behind it.
 //
 //   stream_add_rows: X = x + a per token, where a is a sub-layer's output row, the weighted sum of the rows that a
-//   token's chosen experts left (ascending slot), or nothing.  From X, as asked: X itself (the new stream), its RMS norm
+//   token's chosen experts left (ascending slot), one row for all tokens, or nothing.  From X, as asked: X itself (the new stream), its RMS norm
 //   y = X * rsqrt(mean(X^2) + eps) * w in the activation type, and the row [X | x0] in the activation type (the
 //   input of a product that reads the stream together with what it was at the start).  With a list of token rows
 //   only those are worked on and the outputs are compact.
@@ -26,6 +26,7 @@ struct AddRowsParams {
   const float* x;                                    // [tokens, width]
   const void* rows; int top;                         // row of pair (token, slot): row_of_pair[pair], or pair itself
   const int* row_of_pair; const float* pair_weight;  // weights 1 without a list
+  int one_row;                                       // every token's row is row 0
   const int* token_rows;                             // tokens to work on, or null: all
   float* stream;                                     // [tokens, width] or null
   void* normed; const void* weight; float eps;       // [count, width] or null
@@ -42,15 +43,20 @@ stream_add_rows_kernel(const AddRowsParams p) {
   const int width = p.width;
   const float* x = p.x + (size_t)t * width;
   const T* rows = (const T*)p.rows;
-  auto summed = [&](int i, float (&v)[N]) {
+  // the row and the weight of a slot of this token (row < 0: none)
+  auto slot_row = [&](int slot, float& w) {
+    const long long pair = (long long)t * p.top + slot;
+    w = p.pair_weight != nullptr ? p.pair_weight[pair] : 1.0f;
+    return p.row_of_pair != nullptr ? (long long)p.row_of_pair[pair] : p.one_row ? 0ll : pair;
+  };
+  auto summed = [&](int i, float (&v)[N]) {          // one piece of the sum: what the registers do not hold
     float a[N];
 #pragma unroll
     for (int j = 0; j < N; ++j) a[j] = 0.0f;
     for (int slot = 0; slot < p.top; ++slot) {
-      const long long pair = (long long)t * p.top + slot;
-      const long long row = p.row_of_pair != nullptr ? p.row_of_pair[pair] : pair;
+      float w;
+      const long long row = slot_row(slot, w);
       if (row < 0) continue;
-      const float w = p.pair_weight != nullptr ? p.pair_weight[pair] : 1.0f;
       const RowPiece<T, N> r = *reinterpret_cast<const RowPiece<T, N>*>(rows + (size_t)row * width + i);
 #pragma unroll
       for (int j = 0; j < N; ++j) a[j] = fmaf(w, to_float(r.v[j]), a[j]);
@@ -80,15 +86,47 @@ stream_add_rows_kernel(const AddRowsParams p) {
 #pragma unroll
     for (int j = 0; j < N; ++j) ss = fmaf(v[j], v[j], ss);
   };
+  // the kept pieces: the stream's, the weights' and a slot's loads are each in flight together
+  RowPiece<float, N> xs[SR_PIECES];
+  RowPiece<W, N> ws[SR_PIECES];
 #pragma unroll
   for (int s = 0; s < SR_PIECES; ++s) {
     const int i = (threadIdx.x + s * SR_THREADS) * N;
-    if (i < width) summed(i, kept[s]);
+#pragma unroll
+    for (int j = 0; j < N; ++j) kept[s][j] = 0.0f;
+    if (i < width) {
+      xs[s] = *reinterpret_cast<const RowPiece<float, N>*>(x + i);
+      if (p.normed != nullptr) ws[s] = *reinterpret_cast<const RowPiece<W, N>*>((const W*)p.weight + i);
+    }
+  }
+#pragma unroll 2
+  for (int slot = 0; slot < p.top; ++slot) {
+    float w;
+    const long long row = slot_row(slot, w);
+    if (row < 0) continue;
+    RowPiece<T, N> r[SR_PIECES];
+#pragma unroll
+    for (int s = 0; s < SR_PIECES; ++s) {
+      const int i = (threadIdx.x + s * SR_THREADS) * N;
+      if (i < width) r[s] = *reinterpret_cast<const RowPiece<T, N>*>(rows + (size_t)row * width + i);
+    }
+#pragma unroll
+    for (int s = 0; s < SR_PIECES; ++s) {
+      const int i = (threadIdx.x + s * SR_THREADS) * N;
+      if (i < width) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) kept[s][j] = fmaf(w, to_float(r[s].v[j]), kept[s][j]);
+      }
+    }
   }
 #pragma unroll
   for (int s = 0; s < SR_PIECES; ++s) {
     const int i = (threadIdx.x + s * SR_THREADS) * N;
-    if (i < width) first_pass(i, kept[s]);
+    if (i < width) {
+#pragma unroll
+      for (int j = 0; j < N; ++j) kept[s][j] = xs[s].v[j] + kept[s][j];
+      first_pass(i, kept[s]);
+    }
   }
   // rows wider than the registers hold: the sum goes through `stream`, which the same thread reads again
   const int rest = (threadIdx.x + SR_PIECES * SR_THREADS) * N;
@@ -101,8 +139,7 @@ stream_add_rows_kernel(const AddRowsParams p) {
   const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + p.eps);
   const W* weight = (const W*)p.weight;
   OUT* dst = (OUT*)p.normed + (size_t)n * width;
-  auto put = [&](int i, const float (&v)[N]) {
-    const RowPiece<W, N> w = *reinterpret_cast<const RowPiece<W, N>*>(weight + i);
+  auto put = [&](int i, const float (&v)[N], const RowPiece<W, N>& w) {
     RowPiece<OUT, N> r;
 #pragma unroll
     for (int j = 0; j < N; ++j) r.v[j] = from_float<OUT>(v[j] * inv * to_float(w.v[j]));
@@ -111,7 +148,7 @@ stream_add_rows_kernel(const AddRowsParams p) {
 #pragma unroll
   for (int s = 0; s < SR_PIECES; ++s) {
     const int i = (threadIdx.x + s * SR_THREADS) * N;
-    if (i < width) put(i, kept[s]);
+    if (i < width) put(i, kept[s], ws[s]);
   }
   for (int i = rest; i < width; i += SR_THREADS * N) {
     float v[N];
@@ -122,13 +159,13 @@ stream_add_rows_kernel(const AddRowsParams p) {
     } else {
       summed(i, v);
     }
-    put(i, v);
+    put(i, v, *reinterpret_cast<const RowPiece<W, N>*>(weight + i));
   }
 }
 
 // The sum goes into `stream` (which may be x itself) when given; `token_rows` (count entries) only without `stream`.
 extern "C" int kvb_stream_add_rows(const float* x, const void* rows, int top, const int* row_of_pair,
-                                   const float* pair_weight, const int* token_rows, int count, float* stream,
+                                   const float* pair_weight, int one_row, const int* token_rows, int count, float* stream,
                                    void* normed, const void* weight, float eps, void* packed, const float* origin,
                                    int width, int dtype, int out_dtype, int weight_dtype, cudaStream_t cuda_stream) {
   if (count == 0) return 0;
@@ -138,7 +175,7 @@ extern "C" int kvb_stream_add_rows(const float* x, const void* rows, int top, co
   KVB_REQUIRE(token_rows == nullptr || stream == nullptr, "stream_add_rows: a list of tokens leaves the stream alone");
   AddRowsParams p;
   p.x = x; p.rows = rows; p.top = top; p.row_of_pair = row_of_pair; p.pair_weight = pair_weight;
-  p.token_rows = token_rows; p.stream = stream; p.normed = normed; p.weight = weight; p.eps = eps; p.packed = packed;
+  p.one_row = one_row; p.token_rows = token_rows; p.stream = stream; p.normed = normed; p.weight = weight; p.eps = eps; p.packed = packed;
   p.origin = origin; p.width = width;
   const bool quads = width % 4 == 0 && aligned16(x) && aligned16(rows) && (stream == nullptr || aligned16(stream)) &&
                      (normed == nullptr || (aligned16(normed) && aligned16(weight))) &&

@@ -102,7 +102,7 @@ def ensure_built(verbose: bool = False) -> str:
                             _int, _int, _int, _vp],
         "kvb_ssm_scan": [_vp, _vp, _ll, _vp, _vp, _ll, _ll, _vp, _vp, _int, _int, _int, _int, _int, _int, _vp],
         "kvb_gated_group_norm": [_vp, _ll, _vp, _vp, _ll, _vp, _int, _int, _int, _float, _int, _vp],
-        "kvb_stream_add_rows": [_vp, _vp, _int, _vp, _vp, _vp, _int, _vp, _vp, _vp, _float, _vp, _vp, _int, _int, _int,
+        "kvb_stream_add_rows": [_vp, _vp, _int, _vp, _vp, _int, _vp, _int, _vp, _vp, _vp, _float, _vp, _vp, _int, _int, _int,
                                 _int, _vp],
         "kvb_embed_pairs": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _ll, _ll, _ll, _float,
                             _int, _vp],
@@ -1053,8 +1053,9 @@ def stream_add_norm(x: torch.Tensor, a: torch.Tensor, weight: torch.Tensor, eps:
 def stream_add_rows(x: torch.Tensor, a, *, weight: torch.Tensor | None = None, eps: float = 0.0,
                     out_dtype: torch.dtype | None = None, token_rows: torch.Tensor | None = None,
                     origin: torch.Tensor | None = None, keep: bool = True) -> tuple:
-    """``X = x + a`` on the 32-bit stream ``x [T, width]``, ``a`` a sub-layer's output ``[T, width]`` or the rows its
-    experts left (``ExpertRows``: summed per token in ascending slot, weights still pending included), or None.  Returns
+    """``X = x + a`` on the 32-bit stream ``x [T, width]``, ``a`` a sub-layer's output ``[T, width]``, one row for all
+    tokens ``[1, width]``, the rows a sub-layer's experts left (``ExpertRows``: summed per token in ascending slot,
+    weights still pending included), or None.  Returns
     ``(X, y, packed)``: ``X`` is ``x`` updated in place (``keep`` False or ``token_rows`` given: ``x`` stays and
     ``X`` is None); ``y = X * rsqrt(mean(X^2) + eps) * weight`` in ``out_dtype`` (with ``weight``, else None);
     ``packed [T, 2 * width]`` = ``[X | origin]`` in ``out_dtype`` (with ``origin``, a stream of the same shape, else
@@ -1079,7 +1080,7 @@ def stream_add_rows(x: torch.Tensor, a, *, weight: torch.Tensor | None = None, e
         top, keep = 0, False
         if out_dtype is None:
             raise KernelError("stream_add_rows: without anything to add the type of the outputs must be given")
-    elif row_of_pair is None and rows.shape[0] != tokens * top:
+    elif row_of_pair is None and rows.shape[0] != tokens * top and not (experts is None and rows.shape[0] == 1):
         raise KernelError(f"stream_add_rows: {rows.shape[0]} rows for {tokens} tokens of {top}")
     dtype = out_dtype or rows.dtype
     count = tokens
@@ -1102,7 +1103,7 @@ def stream_add_rows(x: torch.Tensor, a, *, weight: torch.Tensor | None = None, e
     code = _BF16 if dtype == torch.bfloat16 else _F32
     _call("kvb_stream_add_rows", x.data_ptr(), None if rows is None else rows.data_ptr(), int(top),
           None if row_of_pair is None else row_of_pair.data_ptr(), None if pair_weight is None else pair_weight.data_ptr(),
-          None if token_rows is None else token_rows.data_ptr(), count, x.data_ptr() if keep else None,
+          int(experts is None and rows is not None and rows.shape[0] == 1), None if token_rows is None else token_rows.data_ptr(), count, x.data_ptr() if keep else None,
           None if normed is None else normed.data_ptr(), None if weight is None else weight.data_ptr(), float(eps),
           None if packed is None else packed.data_ptr(), None if origin is None else origin.data_ptr(), width,
           code if rows is None else _dtype_code(rows), code, weight_code, _stream())

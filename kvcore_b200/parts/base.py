@@ -13,7 +13,7 @@ none knows the model it sits in.  What each kind must provide:
   fixed-size per-request state; ``None`` if none).  ``cache`` is the ``LayerCache`` of the
   schedule entry being run.
 * **FeedForward**: ``forward(x [T,E], ctx) -> [T,E]``.
-* **StreamStep**: ``forward(h, residual, origin, number, ctx) -> residual``; what is done to the whole stream between
+* **StreamStep**: ``forward(h, residual, origin, number, ctx) -> (h, residual)``; what is done to the whole stream between
   two layers (``origin``: the embedded tokens as they entered the stream, 32-bit).
 * **Block**: ``forward(h, residual, ctx, cache) -> (h, residual)``; arranges norms, mixer and
   feed-forward.  ``residual`` is ``None`` before the first block.
@@ -196,7 +196,8 @@ class Block(Part):
 
 
 class StreamStep(Part):
-    def forward(self, h: Any, residual: torch.Tensor | None, origin: torch.Tensor, number: int, ctx: Any) -> torch.Tensor:
+    def forward(self, h: Any, residual: torch.Tensor | None, origin: torch.Tensor, number: int,
+                ctx: Any) -> tuple[Any, torch.Tensor]:
         raise NotImplementedError
 
 

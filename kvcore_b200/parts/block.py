@@ -80,7 +80,7 @@ class PreNormStreamBlock(PreNormResidualBlock):
     In the ``(h, residual)`` pair that runs through the blocks this block returns ``(its last sub-layer's output or
     its experts' rows, stream)``."""
 
-    takes_expert_rows = True
+    takes_rows = True          # ``h`` may be experts' rows, or one row for all tokens
 
     def __init__(self, *, layer: LayerSpec, unused_tensors: tuple = (), dtype: torch.dtype, device: torch.device) -> None:
         self.unused_tensors = tuple(unused_tensors)

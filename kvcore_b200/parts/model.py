@@ -132,10 +132,11 @@ class DecoderModel:
             block = self.blocks[entry.layer]
             if entry.ahead is not None:
                 name, number = entry.ahead
-                residual = self.stream_steps[name].forward(h, residual, origin, number, ctx)
-                h = Summed(None)
-            elif isinstance(h, K.ExpertRows) and not getattr(block, "takes_expert_rows", False):
-                residual, h = K.stream_add_rows(residual, h)[0], Summed(None)
+                h, residual = self.stream_steps[name].forward(h, residual, origin, number, ctx)
+            if residual is not None and not isinstance(h, Summed) and not getattr(block, "takes_rows", False):
+                # rows that only the norm behind them knows how to add: experts' rows, one row for all tokens
+                if isinstance(h, K.ExpertRows) or h.shape != residual.shape:
+                    residual, h = K.stream_add_rows(residual, h)[0], Summed(None)
             h, residual = block.forward(h, residual, ctx, caches[index])
         return h, residual
 

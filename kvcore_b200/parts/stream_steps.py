@@ -2,7 +2,8 @@
 
 ``RecallOrigin``: ``x <- W [x; x_0] + step[n]`` with ``x_0`` the embedded tokens as they entered the stream and ``n``
 the number the schedule gives it (a loop of layers that share their weights begins each of its passes with it).
-The stream is 32-bit; the product reads it (and ``x_0``) in the activation type and leaves a 32-bit stream.
+The stream is 32-bit; the product reads it (and ``x_0``) in the activation type and leaves a 32-bit stream, and
+``step[n]`` (one row for all tokens) is left to the norm behind it to add.
 """
 from __future__ import annotations
 
@@ -34,7 +35,7 @@ class RecallOrigin(StreamStep):
             residual = K.stream_add(residual)
         pending = None if isinstance(h, Summed) else h
         both = K.stream_add_rows(residual, pending, out_dtype=self.dtype, origin=origin, keep=False)[2]
-        return K.linear(both, self.weight, self.steps[number], out_dtype=torch.float32)
+        return self.steps[number:number + 1], K.linear(both, self.weight, out_dtype=torch.float32)
 
 
 STREAM_STEPS.register("recall_origin", RecallOrigin)

@@ -219,6 +219,8 @@ def stream_add_rows(x, a, *, weight=None, eps=0.0, out_dtype=None, token_rows=No
                 pairs = pairs * a.pending_weights.reshape(-1, 1)
         else:
             pairs = a.float()
+            if a.shape[0] == 1:                     # one row for all tokens
+                pairs = pairs.expand(tokens, width)
         total = x + pairs.reshape(tokens, -1, width).sum(1)
     dtype = out_dtype or (a.rows if hasattr(a, "rows") else a).dtype
     keep = keep and token_rows is None and a is not None

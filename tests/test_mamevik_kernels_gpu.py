@@ -178,6 +178,11 @@ def test_sum_norm_and_packing_of_the_stream(width, dtype):
         assert out[0] is None and out[1] is None and torch.equal(before, x)
         total = x if addend is None else x + a.float()
         assert torch.equal(out[2], torch.cat([total, origin], 1).to(dtype))
+    # one row for all tokens
+    row = a[2:3].contiguous()
+    stream_one, y_one, _ = K().stream_add_rows(x.clone(), row, weight=w, eps=1e-5)
+    stream_all, y_all, _ = K().stream_add_rows(x.clone(), row.expand(tokens, width).contiguous(), weight=w, eps=1e-5)
+    assert torch.equal(stream_one, stream_all) and torch.equal(y_one, y_all)
     # some tokens only
     rows = torch.tensor([5, 0, 3], dtype=torch.int32, device=DEV)
     before = x.clone()
