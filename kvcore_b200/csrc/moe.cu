@@ -20,7 +20,7 @@
 //            out = silu(gate) * up, or with g = min(gate, limit), u = clamp(up, -limit, limit):
 //            out = g * sigmoid(alpha g) * (u + shift).
 //   gemv:    the same two products for a handful of pairs in bf16, bound by the bytes of the chosen
-//            experts' matrices (no padded tiles).
+//            experts' matrices (no padded tiles); for more pairs, a tile's pairs share one pass (stream_rows).
 //   gather:  the pairs' input rows expert by expert at a common stride, for one batched library product
 //            over all experts.
 //   combine: y[token] = sum over slots of out[row of (token, slot)] (ascending slot, 32-bit)
@@ -479,129 +479,142 @@ extern "C" int kvb_moe_gemv(void* out, const void* a, long long a_stride, int a_
   return 0;
 }
 
-// The same for a few hundred pairs: the pairs of one expert share one pass over its matrices.  grid (N / 128,
-// 2 * tiles): a block takes one half (8 rows) of a tile of the grouped order (moe_align), holds those pairs'
-// input rows in shared memory and gives each warp 2 output columns (GATED: 2 gate and 2 up rows) for all
-// 8 rows, 8 such groups of 16 columns one after the other; a weight vector is loaded once and used for every
-// row, the staged rows for 128 columns.  (Four columns a warp cost 176 registers and left one block a
-// multiprocessor; one group of columns a block spent more bytes on staging the rows than on weights.)
-#define MOE_GEMV_ROWS 8
-#define MOE_GEMV_ROWS_CPW 2                                  // output columns a warp (GATED: that many gate and up rows)
-#define MOE_GEMV_ROWS_COLS (8 * MOE_GEMV_ROWS_CPW)           // output columns of one group: 8 warps
-#define MOE_GEMV_ROWS_GROUPS 8                               // groups of columns a block walks with the rows it staged
+// The same for up to a few hundred pairs, grouped by expert (moe_align): the pairs of an expert's tile of MOE_BM rows
+// share one pass over its matrices, multiplied by mma.sync m16n8k16 (32-bit accumulation).  grid (columns, tiles): a
+// block of 8 warps holds the tile's input rows (weighted and rounded) in shared memory, a slab of MR_SLAB columns of K
+// at a time; each warp owns two groups of 8 weight rows (GATED: the gate and the up rows of 8 outputs, else 16 outputs)
+// and streams them from global memory straight into its B fragments, the next 128 columns of K in flight while the
+// current ones are multiplied.  A thread's 16 bytes of a weight row (8 neighbouring k) serve two k-steps: which k a
+// fragment place stands for does not matter as long as the A fragments use the same one, so both take theirs from the
+// same 8 neighbouring entries.  Bound by the weights it reads, each expert's once.
+#define MR_SLAB 2048
+#define MR_PITCH (MR_SLAB + 32)          // rows 64 bytes apart modulo 128: the fragment loads meet no bank conflict
+#define MR_STEP 128                      // columns of K between two rounds of loads: four 16-byte pieces a row and thread
+#define MR_PIECES (MR_STEP / 32)
+
+__device__ __forceinline__ void mr_mma(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3, unsigned b0,
+                                       unsigned b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
 template <bool GATED>
-__global__ void __launch_bounds__(256)
-moe_gemv_rows_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long long a_stride, int a_row_div,
-                     const float* __restrict__ pair_weight, const bf16* __restrict__ w,
-                     const int* __restrict__ sorted, const int* __restrict__ tile_expert,
-                     const int* __restrict__ meta, int N, int K, MoeJoin join) {
+__global__ void __launch_bounds__(256, 2)
+moe_stream_rows_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long long a_stride, int a_row_div,
+                       const float* __restrict__ pair_weight, const bf16* __restrict__ w,
+                       const int* __restrict__ sorted, const int* __restrict__ tile_expert,
+                       const int* __restrict__ meta, int N, int K, MoeJoin join) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_MOE_GEMM);
-  extern __shared__ __align__(16) unsigned char gemv_smem[];
-  bf16* xs = reinterpret_cast<bf16*>(gemv_smem);            // [MOE_GEMV_ROWS][K]
-  __shared__ int pair_of[MOE_GEMV_ROWS];
-  const int tile = blockIdx.y >> 1, half = blockIdx.y & 1;
+  extern __shared__ __align__(16) unsigned char rows_smem[];
+  bf16* as = reinterpret_cast<bf16*>(rows_smem);             // [MOE_BM][MR_PITCH]
+  __shared__ int pair_of[MOE_BM];
+  const int tile = blockIdx.y;
   if (tile >= meta[0]) return;
-  const int first = sorted[tile * MOE_BM + half * MOE_GEMV_ROWS];
-  if (first < 0) return;                                     // a run fills its tiles from the front
-  if (threadIdx.x < MOE_GEMV_ROWS) pair_of[threadIdx.x] = sorted[tile * MOE_BM + half * MOE_GEMV_ROWS + threadIdx.x];
-  __syncthreads();
+  if (threadIdx.x < MOE_BM) pair_of[threadIdx.x] = sorted[tile * MOE_BM + threadIdx.x];
   const int expert = tile_expert[tile];
-  for (int i = threadIdx.x * 8; i < MOE_GEMV_ROWS * K; i += 256 * 8) {
-    const int r = i / K, k = i % K;
-    const int pair = pair_of[r];
-    Vec16<bf16> v;
-    if (pair >= 0) {
-      v.load(a + (size_t)(pair / a_row_div) * a_stride + k);
-      if (pair_weight != nullptr) {
-        const float scale = pair_weight[pair];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) v.set(j, v.get(j) * scale);
-      }
-    } else {
-      v.raw = make_uint4(0, 0, 0, 0);
-    }
-    v.store(xs + i);
-  }
-  __syncthreads();
-  constexpr int CPW = MOE_GEMV_ROWS_CPW;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
   const bf16* we = w + (size_t)expert * (GATED ? 2 : 1) * N * K;
-  constexpr int COLS = GATED ? 2 * CPW : CPW;
-  // the staged rows serve MOE_GEMV_ROWS_GROUPS groups of columns, one after the other
-  for (int group = 0; group < MOE_GEMV_ROWS_GROUPS; ++group) {
-  const int n0 = (blockIdx.x * MOE_GEMV_ROWS_GROUPS + group) * MOE_GEMV_ROWS_COLS + warp * CPW;
-  if (n0 >= N) break;                                        // uniform over the warp
-  const bf16* cols[COLS];
-  float acc[COLS][MOE_GEMV_ROWS];
+  const int n0 = (blockIdx.x * 8 + warp) * (GATED ? 8 : 16);   // the warp's first output
+  const bf16* rows[2];
 #pragma unroll
-  for (int c = 0; c < COLS; ++c) {
-    const int n = min(n0 + (c % CPW), N - 1) + (c >= CPW ? N : 0);
-    cols[c] = we + (size_t)n * K;
-#pragma unroll
-    for (int r = 0; r < MOE_GEMV_ROWS; ++r) acc[c][r] = 0.0f;
+  for (int c = 0; c < 2; ++c) {
+    const int n = min(n0 + g + (GATED ? 0 : 8 * c), N - 1);    // outputs beyond N compute a copy that nobody stores
+    rows[c] = we + (size_t)(n + (GATED ? c * N : 0)) * K + q * 8;
   }
-  for (int k = lane * 8; k < K; k += 32 * 8) {
-    Vec16<bf16> wv[COLS];
+  float acc[2][4];
 #pragma unroll
-    for (int c = 0; c < COLS; ++c) wv[c].load(cols[c] + k);
+  for (int c = 0; c < 2; ++c) acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.0f;
+  for (int k0 = 0; k0 < K; k0 += MR_SLAB) {
+    const int kn = min(MR_SLAB, K - k0), steps = (kn + MR_STEP - 1) / MR_STEP;
+    __syncthreads();                                         // pair_of is there; the slab in front is spent
+    const int chunks = steps * (MR_STEP / 8);
+    for (int i = threadIdx.x; i < MOE_BM * chunks; i += 256) {
+      const int r = i / chunks, k = (i - r * chunks) * 8, pair = pair_of[r];
+      Vec16<bf16> v;
+      v.raw = make_uint4(0, 0, 0, 0);
+      if (pair >= 0 && k < kn) {
+        v.load(a + (size_t)(pair / a_row_div) * a_stride + k0 + k);
+        if (pair_weight != nullptr) {
+          const float scale = pair_weight[pair];
 #pragma unroll
-    for (int r = 0; r < MOE_GEMV_ROWS; ++r) {
-      Vec16<bf16> x;
-      x.load(xs + (size_t)r * K + k);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const float xv = x.get(j);
-#pragma unroll
-        for (int c = 0; c < COLS; ++c) acc[c][r] = fmaf(wv[c].get(j), xv, acc[c][r]);
+          for (int j = 0; j < 8; ++j) v.set(j, v.get(j) * scale);
+        }
       }
+      v.store(as + r * MR_PITCH + k);
+    }
+    __syncthreads();
+    auto fetch = [&](int step, uint4 (&b)[2][MR_PIECES]) {
+#pragma unroll
+      for (int u = 0; u < MR_PIECES; ++u) {
+        const int k = step * MR_STEP + u * 32;
+#pragma unroll
+        for (int c = 0; c < 2; ++c)
+          b[c][u] = k + q * 8 < kn ? __ldcs(reinterpret_cast<const uint4*>(rows[c] + k0 + k)) : make_uint4(0, 0, 0, 0);
+      }
+    };
+    auto multiply = [&](int step, const uint4 (&b)[2][MR_PIECES]) {
+      const bf16* lo = as + g * MR_PITCH + step * MR_STEP + q * 8;
+#pragma unroll
+      for (int u = 0; u < MR_PIECES; ++u) {
+        const uint4 x = *reinterpret_cast<const uint4*>(lo + u * 32);
+        const uint4 y = *reinterpret_cast<const uint4*>(lo + 8 * MR_PITCH + u * 32);
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          mr_mma(acc[c], x.x, y.x, x.y, y.y, b[c][u].x, b[c][u].y);
+          mr_mma(acc[c], x.z, y.z, x.w, y.w, b[c][u].z, b[c][u].w);
+        }
+      }
+    };
+    uint4 even[2][MR_PIECES], odd[2][MR_PIECES];
+    fetch(0, even);
+    for (int step = 0; step < steps; step += 2) {
+      if (step + 1 < steps) fetch(step + 1, odd);
+      multiply(step, even);
+      if (step + 2 < steps) fetch(step + 2, even);
+      if (step + 1 < steps) multiply(step + 1, odd);
     }
   }
+  // a thread holds outputs 2 q and 2 q + 1 of rows g and g + 8
 #pragma unroll
-  for (int c = 0; c < COLS; ++c)
+  for (int half = 0; half < 2; ++half) {
+    const int pair = pair_of[g + 8 * half];
+    if (pair < 0) continue;
 #pragma unroll
-    for (int r = 0; r < MOE_GEMV_ROWS; ++r) acc[c][r] = warp_sum(acc[c][r]);
-  // lane (r, c) = (lane / CPW, lane % CPW) of the first 8 * CPW lanes writes one output
-  const int r = lane / CPW, c = lane % CPW;
-  float v = 0.0f, u = 0.0f;
+    for (int c = 0; c < (GATED ? 1 : 2); ++c)
 #pragma unroll
-  for (int rr = 0; rr < MOE_GEMV_ROWS; ++rr)
-#pragma unroll
-    for (int cc = 0; cc < CPW; ++cc)
-      if (rr == r && cc == c) {
-        v = acc[cc][rr];
-        if (GATED) u = acc[(cc + CPW) % COLS][rr];
+      for (int j = 0; j < 2; ++j) {
+        const int n = n0 + c * 8 + 2 * q + j;
+        const float v = acc[c][2 * half + j];
+        if (n < N) out[(size_t)pair * N + n] = from_float<bf16>(GATED ? moe_join<bf16>(v, acc[1][2 * half + j], join) : v);
       }
-  const int pair = lane < MOE_GEMV_ROWS * CPW ? pair_of[r] : -1;
-  if (pair >= 0 && n0 + c < N) {
-    if (GATED) v = moe_join<bf16>(v, u, join);
-    out[(size_t)pair * N + n0 + c] = from_float<bf16>(v);
-  }
   }
 }
 
-extern "C" int kvb_moe_gemv_rows(void* out, const void* a, long long a_stride, int a_row_div, const float* pair_weight,
-                                 const void* w, const int* sorted, const int* tile_expert, const int* meta,
-                                 int max_tiles, int N, int K, int gated, float alpha, float limit, float shift,
-                                 cudaStream_t stream) {
+extern "C" int kvb_moe_stream_rows(void* out, const void* a, long long a_stride, int a_row_div, const float* pair_weight,
+                                   const void* w, const int* sorted, const int* tile_expert, const int* meta,
+                                   int max_tiles, int N, int K, int gated, float alpha, float limit, float shift,
+                                   cudaStream_t stream) {
   const MoeJoin join = {alpha, limit, shift};
   if (max_tiles == 0) return 0;
-  KVB_REQUIRE(N > 0 && K > 0 && K % 8 == 0 && a_stride % 8 == 0 && a_row_div > 0, "moe_gemv_rows: K and the row stride must be multiples of 8");
-  KVB_REQUIRE(aligned16(a) && aligned16(w), "moe_gemv_rows: operands must be 16-byte aligned");
-  KVB_REQUIRE(2 * (long long)max_tiles <= 65535, "moe_gemv_rows: too many tiles for one launch");
-  const size_t smem = (size_t)MOE_GEMV_ROWS * K * sizeof(bf16);
-  KVB_REQUIRE(smem <= 200 * 1024, "moe_gemv_rows: the input rows do not fit in shared memory");
-  const int block_cols = MOE_GEMV_ROWS_COLS * MOE_GEMV_ROWS_GROUPS;
-  dim3 grid((N + block_cols - 1) / block_cols, 2 * max_tiles);
-#define KVB_MOE_GEMV_ROWS(G_)                                                                                 \
+  KVB_REQUIRE(N > 0 && K > 0 && K % 8 == 0 && a_stride % 8 == 0 && a_row_div > 0, "moe_stream_rows: K and the row stride must be multiples of 8");
+  KVB_REQUIRE(aligned16(a) && aligned16(w), "moe_stream_rows: operands must be 16-byte aligned");
+  KVB_REQUIRE(max_tiles <= 65535, "moe_stream_rows: too many tiles for one launch");
+  const int smem = MOE_BM * MR_PITCH * (int)sizeof(bf16);
+  const int block_cols = gated ? 64 : 128;
+  dim3 grid((N + block_cols - 1) / block_cols, max_tiles);
+#define KVB_MOE_STREAM_ROWS(G_)                                                                               \
   do {                                                                                                        \
-    if (smem > 48 * 1024)                                                                                     \
-      KVB_CHECK_CUDA(cudaFuncSetAttribute(moe_gemv_rows_kernel<G_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-    KVB_CHECK_CUDA(kvb_launch((moe_gemv_rows_kernel<G_>), grid, dim3(256), smem, stream, true, (bf16*)out,     \
-                              (const bf16*)a, a_stride, a_row_div, pair_weight, (const bf16*)w, sorted,        \
-                              tile_expert, meta, N, K, join));                                                 \
+    static bool allowed = false;                    /* more than 48 KB a block is asked for once */           \
+    if (!allowed) {                                                                                           \
+      KVB_CHECK_CUDA(cudaFuncSetAttribute(moe_stream_rows_kernel<G_>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)); \
+      allowed = true;                                                                                         \
+    }                                                                                                         \
+    KVB_CHECK_CUDA(kvb_launch((moe_stream_rows_kernel<G_>), grid, dim3(256), smem, stream, true, (bf16*)out,  \
+                              (const bf16*)a, a_stride, a_row_div, pair_weight, (const bf16*)w, sorted,       \
+                              tile_expert, meta, N, K, join));                                                \
   } while (0)
-  if (gated) KVB_MOE_GEMV_ROWS(true); else KVB_MOE_GEMV_ROWS(false);
-#undef KVB_MOE_GEMV_ROWS
+  if (gated) KVB_MOE_STREAM_ROWS(true); else KVB_MOE_STREAM_ROWS(false);
+#undef KVB_MOE_STREAM_ROWS
   KVB_CHECK_LAUNCH();
   return 0;
 }

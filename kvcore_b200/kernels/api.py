@@ -55,8 +55,8 @@ def ensure_built(verbose: bool = False) -> str:
                           _float, _vp, _int, _vp],
         "kvb_moe_align": [_vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _vp],
         "kvb_moe_gemv": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _int, _int, _int, _int, _int, _float, _float, _float, _vp],
-        "kvb_moe_gemv_rows": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _float, _float,
-                              _float, _vp],
+        "kvb_moe_stream_rows": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _float, _float,
+                                _float, _vp],
         "kvb_moe_gather": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _int, _int, _vp, _int, _int, _vp],
         "kvb_moe_gemm": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _float, _float, _float,
                          _int, _vp],
@@ -1887,8 +1887,7 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, top: int, *, score: str = "
 # bf16 batches of at most this many (token, expert) pairs take the kernel that streams each chosen expert's
 # matrices once; larger ones take library products over each expert's run of rows
 MOE_GEMV_MAX_PAIRS = int(os.environ.get("KVCORE_B200_MOE_GEMV_PAIRS", "512"))
-# up to this many pairs, or fewer than four pairs an expert, each pair streams its expert alone; otherwise
-# the pairs are grouped by expert first
+# up to this many pairs, each pair streams its expert alone; otherwise the pairs are grouped by expert first
 MOE_GEMV_SINGLE_PAIRS = int(os.environ.get("KVCORE_B200_MOE_GEMV_SINGLE_PAIRS", "16"))
 
 
@@ -1993,15 +1992,15 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
 
     if path is None:
         path = moe_path(x, pairs, ff)
-    if path == "stream" and pairs > MOE_GEMV_SINGLE_PAIRS and pairs >= 4 * experts:
-        # enough pairs that experts are shared: the pairs of an expert take one pass over its matrices together
+    if path == "stream" and pairs > MOE_GEMV_SINGLE_PAIRS:
+        # some experts are shared: the pairs of an expert take one pass over its matrices together
         g = grouping if grouping is not None else moe_group(ids, experts, for_library=False)
         hidden = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
-        _call("kvb_moe_gemv_rows", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,
+        _call("kvb_moe_stream_rows", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,
               weights.data_ptr() if weight_on_input else None, gate_up.data_ptr(), g.sorted_pairs.data_ptr(),
               g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, ff, k, 1, *joined, _stream())
         out = torch.empty((pairs, n), dtype=x.dtype, device=x.device)
-        _call("kvb_moe_gemv_rows", out.data_ptr(), hidden.data_ptr(), hidden.stride(0), 1,
+        _call("kvb_moe_stream_rows", out.data_ptr(), hidden.data_ptr(), hidden.stride(0), 1,
               None if weight_on_input else weights.data_ptr(), down.data_ptr(), g.sorted_pairs.data_ptr(),
               g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, n, ff, 0, *joined, _stream())
         return ExpertRows(out, top=top)

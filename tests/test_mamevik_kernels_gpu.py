@@ -295,6 +295,9 @@ def test_router_logits_far_below_the_largest():
     (torch.bfloat16, "tiles", 40, 5, 2, 48, 24),
     (torch.bfloat16, "stream", 3, 8, 2, 64, 48),            # each pair streams its expert alone
     (torch.bfloat16, "stream", 40, 4, 2, 64, 32),           # pairs grouped by expert
+    (torch.bfloat16, "stream", 60, 3, 2, 72, 40),           # more than a tile of pairs an expert, ragged widths
+    (torch.bfloat16, "stream", 30, 4, 1, 2120, 24),         # an input wider than a staged slab
+    (torch.bfloat16, "stream", 25, 7, 2, 136, 2056),        # a hidden row wider than one, experts with few pairs
     (torch.bfloat16, "library", 300, 4, 2, 72, 40),
 ])
 @pytest.mark.parametrize("limit", [0.7, 3.0])
