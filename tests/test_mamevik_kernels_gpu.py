@@ -316,12 +316,12 @@ def test_experts_with_bounded_branches(limit, dtype, path, tokens, experts, top,
             g, u = both[:ff].clamp(max=limit), both[ff:].clamp(min=-limit, max=limit)
             want[t] += a * (down[e].cpu().double() @ (g * torch.sigmoid(1.702 * g) * (u + 1.0)))
     torch.testing.assert_close(got.cpu().double(), want, **(dict(rtol=2e-5, atol=2e-5) if dtype == torch.float32
-                                                            else dict(rtol=3e-2, atol=3e-2)))
+                                                            else dict(rtol=3e-2, atol=6e-2)))
     # the sum into the stream takes the same rows
     stream = torch.zeros(tokens, width, dtype=torch.float32, device=DEV)
     K().stream_add_rows(stream, pairs)
     torch.testing.assert_close(stream.cpu().double(), want, **(dict(rtol=2e-5, atol=2e-5) if dtype == torch.float32
-                                                               else dict(rtol=3e-2, atol=3e-2)))
+                                                               else dict(rtol=3e-2, atol=6e-2)))
 
 
 def test_wrappers_refuse_what_does_not_fit():
