@@ -712,8 +712,8 @@ def mamevik_config(size: dict, kinds: str, loop: tuple[int, int, int]) -> dict:
                      "scale": size["dim"] ** -0.5, "mask": {"size": 1024}}
         layers.append({"type": "mamba2" if kind == "s" else "latent_attention", "mixer": mixer, "mlp": moe})
     return {"architecture": "Mamevik", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5},
-            "embedding": {"bigram": {"buckets": size["vocab"] - 1, "mul_prev": 31, "mul_cur": 17}}, "layers": layers,
-            "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]}, "logit_scale": 0.25, "logit_softcap": 30.0}
+            "embedding": {"bigram": {"buckets": size["vocab"] - 1, "mul_prev": 7, "mul_cur": 13}}, "layers": layers,
+            "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]}, "logit_scale": 0.5, "logit_softcap": 20.0}
 
 
 def llama_config(size: dict) -> dict:

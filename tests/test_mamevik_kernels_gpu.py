@@ -237,8 +237,8 @@ def test_embedding_of_pairs(normed, width, buckets, factors, dtype):
 
 def test_logits_cap():
     logits = randn(3, 1001, dtype=torch.float32, seed=81, scale=40.0)
-    want = 30.0 * torch.tanh(logits.double() * 0.25 / 30.0)
-    got = K().softcap(logits, 0.25, 30.0)
+    want = 22.0 * torch.tanh(logits.double() * 0.4 / 22.0)
+    got = K().softcap(logits, 0.4, 22.0)
     assert got.data_ptr() == logits.data_ptr()
     torch.testing.assert_close(got.double(), want, rtol=1e-5, atol=1e-5)
 
