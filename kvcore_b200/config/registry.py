@@ -127,6 +127,9 @@ def _register_stock_architectures() -> None:
     from .mamevik import ARCHITECTURE as MAMEVIK, MamevikConfig
 
     register_architecture(MAMEVIK, lambda raw: MamevikConfig.from_dict(raw).to_model_spec())
+    from .tabopel import ARCHITECTURE as TABOPEL, TabopelConfig
+
+    register_architecture(TABOPEL, lambda raw: TabopelConfig.from_dict(raw).to_model_spec())
 
 
 _register_stock_architectures()

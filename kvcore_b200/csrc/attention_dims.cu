@@ -13,6 +13,7 @@
 //     with no key and no value;
 //   * an optional slope per query head: slope * (query position - key position) is taken off the scaled
 //     score (a linear bias by distance);
+//   * an optional cap on the scaled scores, cap * tanh(score / cap), ahead of the slope (the sink is not capped);
 //   * the output is 32-bit or of the cache's type, with token and head strides of its own.
 //
 // One warp owns one (token, query head) row and walks the keys from the first visible position to the
@@ -34,7 +35,7 @@ struct DimsParams {
   const float* sink;
   const float* slopes;
   int num_rows, HQ, per_value_head, maps, DK, DV, page_size, num_pages, window;
-  float scale;
+  float scale, cap;          // cap 0: none
   int* status;
 };
 
@@ -83,7 +84,9 @@ attention_dims_rows_kernel(const DimsParams p) {
         const T* krow = kbase + (size_t)page * p.k_page_stride + (size_t)(key % p.page_size) * p.k_row_stride;
         float dot = 0.0f;
         for (int d = 0; d < DK; ++d) dot = fmaf(to_float(krow[d]), qv[d], dot);
-        score = dot * p.scale - slope * (float)(pos - key);
+        score = dot * p.scale;
+        if (p.cap > 0.0f) score = p.cap * tanhf(score / p.cap);
+        score -= slope * (float)(pos - key);
       }
     }
     const float new_max = fmaxf(running_max, warp_max(score));
@@ -126,7 +129,8 @@ extern "C" int kvb_attention_dims_rows(void* out, long long out_token_stride, lo
                                        int table_stride, const int* positions, const int* req_index,
                                        const float* sink, const float* slopes, int tokens, int HQ, int per_value_head,
                                        int maps, int DK,
-                                       int DV, int page_size, int num_pages, float scale, int window, int dtype,
+                                       int DV, int page_size, int num_pages, float scale, float cap, int window,
+                                       int dtype,
                                        cudaStream_t stream) {
   if (tokens == 0) return 0;
   KVB_REQUIRE(DK > 0 && DK <= 2048, "attention_dims: the key width must be in [1, 2048]");
@@ -146,6 +150,7 @@ extern "C" int kvb_attention_dims_rows(void* out, long long out_token_stride, lo
   p.table = table; p.table_stride = table_stride; p.positions = positions; p.req_index = req_index;
   p.sink = sink; p.slopes = slopes; p.num_rows = (int)rows; p.HQ = HQ; p.per_value_head = per_value_head; p.maps = maps;
   p.DK = DK; p.DV = DV; p.page_size = page_size; p.num_pages = num_pages; p.window = window; p.scale = scale;
+  p.cap = cap;
   p.status = status;
   const int blocks = (int)((rows + AD_WARPS - 1) / AD_WARPS);
   const size_t smem = (size_t)AD_WARPS * DK * sizeof(float);

@@ -2,7 +2,7 @@
 // a query/key (DK) and the width of a value (DV) differ: the tensor-core form of attention_dims.cu, with the
 // same parameters (strides of keys and values given apart, several score maps a value head, values that
 // may be the first entries of the key rows, a sink per query head, a slope per query head times the distance
-// between query and key taken off the score, 32-bit or bf16 output).
+// between query and key taken off the score, a smooth cap on the scores, 32-bit or bf16 output).
 //
 // A block of 4 warps works on one (request, key head, slice of the value width) and one tile of query
 // rows; a row is a (token, query head of the key head's group) pair, so the heads that share a key head
@@ -38,6 +38,7 @@ struct FlashDimsParams {
   const float* slopes;
   int num_reqs, KH, G, maps, DK, DV, page_size, num_pages, window, v_in_k, vsplit, tiles;
   float scale_log2;
+  float cap_in, cap_out;   // capped scores: cap_out * tanh(dot * scale / cap) with cap_in = 2 log2(e) scale / cap, cap_out = cap log2(e); 0: none
   int num_splits;
   float* partial_o;   // [slot][TILE_M][DVB]
   float* partial_ml;  // [slot][TILE_M][2]
@@ -70,6 +71,15 @@ __device__ __forceinline__ void fd_mma(float (&c)[4], const unsigned (&a)[4], un
 __device__ __forceinline__ unsigned fd_pack(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<const unsigned*>(&v);
+}
+
+// cap_out * tanh(x) for y = 2 log2(e) x, by tanh(x) = 1 - 2 / (1 + exp(2 x)): two approximate instructions (base-2
+// exponential, reciprocal), within a few units of 1e-7 of cap_out; both ends saturate without a special case.
+__device__ __forceinline__ float fd_capped(float y, float cap_out) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(y));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return fmaf(-2.0f * cap_out, r, cap_out);
 }
 
 // Element offsets of every key row (and value row) of a tile inside the cache, or -1: zero-fill.
@@ -254,6 +264,14 @@ flash_dims_kernel(const FlashDimsParams p) {
         fd_mma(s[j + 1], qf, kb[2], kb[3]);
       }
     }
+    // (capped scores are in units of the base-2 exponent already)
+    const float multiplier = p.cap_out > 0.0f ? 1.0f : p.scale_log2;
+    if (p.cap_out > 0.0f) {
+#pragma unroll
+      for (int j = 0; j < NB; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[j][e] = fd_capped(s[j][e] * p.cap_in, p.cap_out);
+    }
     // mask and online softmax (base-2 exponent)
     float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -264,7 +282,7 @@ flash_dims_kernel(const FlashDimsParams p) {
         const int key = t * KEYS + wkey + j * 8 + (lane & 3) * 2 + (e & 1);
         const bool seen = row_valid[h] && key >= key_lo && key < key_hi && key <= row_pos[h] &&
                           (p.window <= 0 || key > row_pos[h] - p.window);
-        const float v = seen ? fmaf(s[j][e], p.scale_log2, -row_slope[h] * (float)(row_pos[h] - key)) : -INFINITY;
+        const float v = seen ? fmaf(s[j][e], multiplier, -row_slope[h] * (float)(row_pos[h] - key)) : -INFINITY;
         s[j][e] = v;
         tile_max[h] = fmaxf(tile_max[h], v);
       }
@@ -521,7 +539,7 @@ extern "C" int kvb_flash_dims_attention(void* out, long long out_token_stride, l
                                         const float* sink, const float* slopes, int num_reqs, int max_query_len,
                                         int value_heads,
                                         int group, int maps, int DK, int DV, int page_size, int num_pages,
-                                        float scale, int window, int num_splits, float* scratch,
+                                        float scale, float cap, int window, int num_splits, float* scratch,
                                         cudaStream_t stream) {
   if (num_reqs == 0) return 0;
   KVB_REQUIRE(DK >= 16 && DK % 16 == 0 && DK <= 1024, "flash_dims: the key width must be a multiple of 16 up to 1024");
@@ -550,6 +568,8 @@ extern "C" int kvb_flash_dims_attention(void* out, long long out_token_stride, l
               k_row_stride == v_row_stride && slices * dvb <= DK) ? 1 : 0;
   p.vsplit = slices;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.cap_in = cap > 0.0f ? 2.0f * 1.4426950408889634f * scale / cap : 0.0f;
+  p.cap_out = cap > 0.0f ? cap * 1.4426950408889634f : 0.0f;
   p.status = kvb_status_word();
   KVB_REQUIRE(p.status != nullptr, "flash_dims: no status word");
   const int max_rows = max_query_len * group;

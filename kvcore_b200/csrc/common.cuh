@@ -179,6 +179,9 @@ struct KvbTrace {
 #define KVB_TAG_ADD_ROWS 51
 #define KVB_TAG_EMBED_PAIRS 52
 #define KVB_TAG_SOFTCAP 53
+#define KVB_TAG_ATTN_PREPARE 54
+#define KVB_TAG_RETENTION_PREPARE 55
+#define KVB_TAG_RELU_SQUARED 56
 
 // 1 when launches should carry the programmatic-serialization attribute (set by the host side).
 extern "C" int kvb_pdl_enabled();

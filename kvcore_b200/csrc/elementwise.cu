@@ -284,6 +284,43 @@ extern "C" int kvb_silu_mul(void* out, const void* gate_up, int rows, int inter,
 }
 
 // ------------------------------------------------------------------------------------------
+// max(x, 0)^2 in place: the activation between the two products of an ungated feed-forward.
+// ------------------------------------------------------------------------------------------
+template <typename T, bool VEC>
+__global__ void relu_squared_kernel(T* __restrict__ x, long long vecs) {
+  KVB_KERNEL_PROLOGUE(KVB_TAG_RELU_SQUARED);
+  const long long step = (long long)gridDim.x * blockDim.x;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < vecs; i += step) {
+    if (VEC) {
+      Vec16<T> v;
+      v.load(x + i * Vec16<T>::N);
+#pragma unroll
+      for (int j = 0; j < Vec16<T>::N; ++j) { const float p = fmaxf(v.get(j), 0.0f); v.set(j, p * p); }
+      v.store(x + i * Vec16<T>::N);
+    } else {
+      const float p = fmaxf(to_float(x[i]), 0.0f);
+      x[i] = from_float<T>(p * p);
+    }
+  }
+}
+
+extern "C" int kvb_relu_squared(void* x, long long count, int dtype, cudaStream_t stream) {
+  if (count == 0) return 0;
+  const int n = dtype == KVB_F32 ? 4 : 8;
+  const bool vec = count % n == 0 && aligned16(x);
+  const long long vecs = vec ? count / n : count;
+  const long long wanted = (vecs + 255) / 256;
+  const long long resident = (long long)(kvb_sm_count() > 0 ? kvb_sm_count() : 1) * 16;
+  const dim3 grid((unsigned)(wanted < resident ? wanted : resident));
+#define KVB_RS(T_, V_) KVB_CHECK_CUDA(kvb_launch((relu_squared_kernel<T_, V_>), grid, dim3(256), 0, stream, true, (T_*)x, vecs))
+  if (dtype == KVB_F32) { if (vec) KVB_RS(float, true); else KVB_RS(float, false); }
+  else { if (vec) KVB_RS(bf16, true); else KVB_RS(bf16, false); }
+#undef KVB_RS
+  KVB_CHECK_LAUNCH();
+  return 0;
+}
+
+// ------------------------------------------------------------------------------------------
 // cos/sin of every (token, frequency) of the step: table[t, j] = (cos, sin)(float(pos_t) * inv_freq[j]).
 // Computed once per step and shared by all layers with the same frequency table.
 // ------------------------------------------------------------------------------------------

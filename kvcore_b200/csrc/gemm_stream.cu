@@ -63,6 +63,7 @@ struct StreamParams {
   // written over residual (every tile its own columns), and the sum of its squares over the tile's
   // 64 columns to sumsq_out[m * n_tiles + tile].  out itself is not written.
   bf16* residual; float* sumsq_out;
+  int square_relu;                   // 1: out = max(x . W, 0)^2, formed from the 32-bit sums
   int silu_pairs;                    // 1: rows n and n+8 of every 16 are a (gate, up) pair: out[m, .] = silu(gate) * up
   unsigned spin_limit;               // polls after which a wait gives up
   // Test of the give-up path (kvb_gemm_stream_test_give_up): block test_skip_block never asks for the
@@ -435,6 +436,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
                   const int n = n_tile * GS_NT + r;
                   float v = acc[0][j][e];
                   if (p.bias && n < p.N) v += __bfloat162float(p.bias[n]);
+                  if (p.square_relu) { v = fmaxf(v, 0.0f); v *= v; }
                   if (p.out_f32) reinterpret_cast<float*>(out_tile)[m * GS_NT + r] = v;
                   else reinterpret_cast<bf16*>(out_tile)[m * GS_NT + r] = __float2bfloat16_rn(v);
                 }
@@ -578,7 +580,8 @@ extern "C" int kvb_gemm_stream_norm_max_k() { return GS_NORM_W_BYTES / 4; }
 // out[M, N] = x[M, K] . w[N, K]^T (+ bias), 1 <= M <= 16, K a multiple of 64.
 //   scratch: kvb_gemm_stream_scratch_floats(sms) words, each holding kvb_gemm_stream_scratch_marker()
 //   before the first launch.  Launches that share scratch must be ordered in one stream.
-//   silu_pairs: the rows of w come in runs of 8 gate rows, 8 up rows, ...; out is [M, N / 2] with
+//   activation 2: out = max(x . w^T + bias, 0)^2.
+//   activation 1: the rows of w come in runs of 8 gate rows, 8 up rows, ...; out is [M, N / 2] with
 //   out[m, c] = silu(gate_c(m)) * up_c(m) (the feed-forward's activation fused into the epilogue).
 //   norm_weight != null: the rows of x are sums that still need their RMS norm; sumsq_in holds
 //   every token's sum of squares in sumsq_pieces pieces ([M, sumsq_pieces]); the kernel uses
@@ -587,17 +590,19 @@ extern "C" int kvb_gemm_stream_norm_max_k() { return GS_NORM_W_BYTES / 4; }
 //   stream: residual = bf16(bf16(out) + residual) in place, and sumsq_out[m, tile] (M x ceil(N / 64)
 //   floats) gets the squares of the new sums, 64 columns a piece; out is not written.
 extern "C" int kvb_gemm_stream_bf16(void* out, int out_f32, long long ldo, const void* x, long long ldx,
-                                    const void* w, const void* bias, int M, int N, int K, int silu_pairs,
+                                    const void* w, const void* bias, int M, int N, int K, int activation,
                                     const void* norm_weight, int norm_weight_f32, float eps, const float* sumsq_in,
                                     int sumsq_pieces, void* residual, float* sumsq_out, float* scratch, int sms,
                                     cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
+  KVB_REQUIRE(activation >= 0 && activation <= 2, "stream gemm: unknown activation");
+  const int silu_pairs = activation == 1;
   KVB_REQUIRE(M > 0 && M <= 16, "stream gemm: takes 1 to 16 rows of x");
   KVB_REQUIRE(K > 0 && K % 64 == 0 && ldx % 8 == 0, "stream gemm: K must be a multiple of 64 and the row stride of x of 8");
   KVB_REQUIRE(aligned16(x) && aligned16(w), "stream gemm: x and w must be 16-byte aligned");
   KVB_REQUIRE(scratch != nullptr && sms > 0, "stream gemm: needs scratch");
   KVB_REQUIRE(!silu_pairs || (N % 16 == 0 && !out_f32), "stream gemm: gated pairs need N a multiple of 16 and a bf16 result");
-  KVB_REQUIRE(residual == nullptr || (!silu_pairs && !out_f32 && N % 8 == 0 && sumsq_out != nullptr && aligned16(residual)),
+  KVB_REQUIRE(residual == nullptr || (!activation && !out_f32 && N % 8 == 0 && sumsq_out != nullptr && aligned16(residual)),
               "stream gemm: the residual epilogue needs a plain bf16 product, N a multiple of 8 and a place for the squares");
   KVB_REQUIRE(norm_weight == nullptr || (sumsq_in != nullptr && sumsq_pieces > 0 && aligned16(norm_weight) &&
                                          (size_t)K * (norm_weight_f32 ? 4 : 2) <= GS_NORM_W_BYTES),
@@ -608,6 +613,7 @@ extern "C" int kvb_gemm_stream_bf16(void* out, int out_f32, long long ldo, const
   p.bias = (const bf16*)bias;
   p.M = M; p.N = N; p.K = K;
   p.silu_pairs = silu_pairs;
+  p.square_relu = activation == 2;
   p.norm_weight = norm_weight; p.norm_weight_f32 = norm_weight_f32; p.eps = eps;
   p.sumsq_in = sumsq_in; p.sumsq_pieces = sumsq_pieces;
   p.residual = (bf16*)residual; p.sumsq_out = sumsq_out;

@@ -18,7 +18,9 @@
 //            a(p, k) = A[p / a_row_div, k] (* pair weight, rounded to the storage type): the weight
 //            multiplies the expert's INPUT.  GATED: w holds gate rows [0, N) and up rows [N, 2N) and
 //            out = silu(gate) * up, or with g = min(gate, limit), u = clamp(up, -limit, limit):
-//            out = g * sigmoid(alpha g) * (u + shift).
+//            out = g * sigmoid(alpha g) * (u + shift).  Ungated with SQUARE: out = max(sum, 0)^2.
+//   Experts without tensors (the ids from E on) hand their input on: align leaves their pairs out, no product sees
+//   them, and the sum over a token's slots adds weight * the token's own input row for them.
 //   gemv:    the same two products for a handful of pairs in bf16, bound by the bytes of the chosen
 //            experts' matrices (no padded tiles); for more pairs, a tile's pairs share one pass (stream_rows).
 //   gather:  the pairs' input rows expert by expert at a common stride, for one batched library product
@@ -219,7 +221,7 @@ extern "C" int kvb_moe_route(int* ids_out, float* weights_out, float* gate_out, 
 __global__ void __launch_bounds__(1024)
 moe_align_kernel(int* __restrict__ sorted, int* __restrict__ tile_expert, int* __restrict__ meta,
                  int* __restrict__ row_of_pair, int* __restrict__ expert_begin,
-                 const int* __restrict__ ids, int pairs, int E, int capacity, int* status) {
+                 const int* __restrict__ ids, int pairs, int E, int known, int capacity, int* status) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_MOE_ALIGN);
   extern __shared__ int ismem[];
   int* counts = ismem;        // [E]
@@ -230,7 +232,7 @@ moe_align_kernel(int* __restrict__ sorted, int* __restrict__ tile_expert, int* _
   for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
     const int e = ids[p];
     if (e >= 0 && e < E) atomicAdd(&counts[e], 1);
-    else atomicOr(status, KVB_STATUS_BAD_TOKEN);
+    else if (e < 0 || e >= known) atomicOr(status, KVB_STATUS_BAD_TOKEN);
   }
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -262,9 +264,9 @@ moe_align_kernel(int* __restrict__ sorted, int* __restrict__ tile_expert, int* _
 }
 
 extern "C" int kvb_moe_align(int* sorted, int* tile_expert, int* meta, int* row_of_pair, int* expert_begin,
-                             const int* ids, int pairs, int E, int capacity, cudaStream_t stream) {
+                             const int* ids, int pairs, int E, int known, int capacity, cudaStream_t stream) {
   if (pairs == 0) return 0;
-  KVB_REQUIRE(E > 0 && E <= 8192, "moe_align: between 1 and 8192 experts");
+  KVB_REQUIRE(E > 0 && E <= 8192 && known >= E, "moe_align: between 1 and 8192 experts");
   // tiles used: one per started run of MOE_BM pairs of an expert, so at most one per pair
   const long long padded = (pairs + (long long)E * (MOE_BM - 1) + MOE_BM - 1) / MOE_BM;
   KVB_REQUIRE(capacity % MOE_BM == 0 && capacity / MOE_BM >= (padded < pairs ? padded : pairs),
@@ -272,7 +274,7 @@ extern "C" int kvb_moe_align(int* sorted, int* tile_expert, int* meta, int* row_
   int* status = kvb_status_word();
   KVB_REQUIRE(status != nullptr, "moe_align: no status word");
   KVB_CHECK_CUDA(kvb_launch((moe_align_kernel), dim3(1), dim3(1024), (size_t)2 * E * sizeof(int), stream, true,
-                            sorted, tile_expert, meta, row_of_pair, expert_begin, ids, pairs, E, capacity, status));
+                            sorted, tile_expert, meta, row_of_pair, expert_begin, ids, pairs, E, known, capacity, status));
   KVB_CHECK_LAUNCH();
   return 0;
 }
@@ -287,7 +289,14 @@ template <>
 __device__ __forceinline__ float moe_silu<bf16>(float x) { return kvb_silu_for_bf16(x); }
 
 // How an expert joins its two branches: silu(gate) * up, or (limit > 0) the bounded form.
-struct MoeJoin { float alpha, limit, shift; };
+// `square`: an ungated product is max(sum, 0)^2.
+struct MoeJoin { float alpha, limit, shift; int square; };
+
+__device__ __forceinline__ float moe_plain(float v, const MoeJoin& join) {
+  if (!join.square) return v;
+  v = fmaxf(v, 0.0f);
+  return v * v;
+}
 
 // As the separate kernels would: both products rounded, then (silu) the activation rounded and the product taken.
 template <typename T>
@@ -360,8 +369,7 @@ moe_gemm_kernel(T* __restrict__ out, const T* __restrict__ a, long long a_stride
   for (int j = 0; j < 4; ++j) {
     const int n = n0 + c0 + j;
     if (n >= N) continue;
-    float v = acc[j];
-    if (GATED) v = moe_join<T>(acc[j], acc_up[j], join);
+    const float v = GATED ? moe_join<T>(acc[j], acc_up[j], join) : moe_plain(acc[j], join);
     out[(size_t)pair * N + n] = from_float<T>(v);
   }
 }
@@ -370,7 +378,7 @@ extern "C" int kvb_moe_gemm(void* out, const void* a, long long a_stride, int a_
                             const void* w, const int* sorted, const int* tile_expert, const int* meta, int max_tiles,
                             int N, int K, int gated, float alpha, float limit, float shift, int dtype,
                             cudaStream_t stream) {
-  const MoeJoin join = {alpha, limit, shift};
+  const MoeJoin join = {alpha, limit, shift, gated == 2};
   if (max_tiles == 0) return 0;
   KVB_REQUIRE(N > 0 && K > 0 && a_row_div > 0, "moe_gemm: empty product");
   dim3 grid(max_tiles, (N + MOE_BN - 1) / MOE_BN);
@@ -378,8 +386,8 @@ extern "C" int kvb_moe_gemm(void* out, const void* a, long long a_stride, int a_
 #define KVB_MOE_GEMM(T_, G_)                                                                                  \
   KVB_CHECK_CUDA(kvb_launch((moe_gemm_kernel<T_, G_>), grid, dim3(256), 0, stream, true, (T_*)out, (const T_*)a, \
                             a_stride, a_row_div, pair_weight, (const T_*)w, sorted, tile_expert, meta, N, K, join))
-  if (dtype == KVB_F32) { if (gated) KVB_MOE_GEMM(float, true); else KVB_MOE_GEMM(float, false); }
-  else { if (gated) KVB_MOE_GEMM(bf16, true); else KVB_MOE_GEMM(bf16, false); }
+  if (dtype == KVB_F32) { if (gated == 1) KVB_MOE_GEMM(float, true); else KVB_MOE_GEMM(float, false); }
+  else { if (gated == 1) KVB_MOE_GEMM(bf16, true); else KVB_MOE_GEMM(bf16, false); }
 #undef KVB_MOE_GEMM
   KVB_CHECK_LAUNCH();
   return 0;
@@ -395,14 +403,14 @@ template <bool GATED>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long long a_stride, int a_row_div,
                 const float* __restrict__ pair_weight, const bf16* __restrict__ w, const int* __restrict__ ids,
-                int E, int N, int K, int* status, MoeJoin join) {
+                int E, int known, int N, int K, int* status, MoeJoin join) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_MOE_GEMM);
   extern __shared__ __align__(16) unsigned char gemv_smem[];
   bf16* xs = reinterpret_cast<bf16*>(gemv_smem);
   const int pair = blockIdx.y;
   const int expert = ids[pair];
-  if (expert < 0 || expert >= E) {
-    if (threadIdx.x == 0) atomicOr(status, KVB_STATUS_BAD_TOKEN);
+  if (expert < 0 || expert >= E) {                   // none, or one without tensors
+    if (threadIdx.x == 0 && (expert < 0 || expert >= known)) atomicOr(status, KVB_STATUS_BAD_TOKEN);
     return;
   }
   const bf16* row = a + (size_t)(pair / a_row_div) * a_stride;
@@ -448,15 +456,17 @@ moe_gemv_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long long a_
     if (GATED) {
       const float u = lane == 0 ? acc[4 % ROWS] : lane == 1 ? acc[5 % ROWS] : lane == 2 ? acc[6 % ROWS] : acc[7 % ROWS];
       v = moe_join<bf16>(v, u, join);
+    } else {
+      v = moe_plain(v, join);
     }
     out[(size_t)pair * N + n0 + lane] = from_float<bf16>(v);
   }
 }
 
 extern "C" int kvb_moe_gemv(void* out, const void* a, long long a_stride, int a_row_div, const float* pair_weight,
-                            const void* w, const int* ids, int pairs, int E, int N, int K, int gated, float alpha,
+                            const void* w, const int* ids, int pairs, int E, int known, int N, int K, int gated, float alpha,
                             float limit, float shift, cudaStream_t stream) {
-  const MoeJoin join = {alpha, limit, shift};
+  const MoeJoin join = {alpha, limit, shift, gated == 2};
   if (pairs == 0) return 0;
   KVB_REQUIRE(N > 0 && K > 0 && K % 8 == 0 && a_stride % 8 == 0 && a_row_div > 0, "moe_gemv: K and the row stride must be multiples of 8");
   KVB_REQUIRE(aligned16(a) && aligned16(w), "moe_gemv: operands must be 16-byte aligned");
@@ -471,9 +481,9 @@ extern "C" int kvb_moe_gemv(void* out, const void* a, long long a_stride, int a_
     if (smem > 48 * 1024)                                                                                      \
       KVB_CHECK_CUDA(cudaFuncSetAttribute(moe_gemv_kernel<G_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
     KVB_CHECK_CUDA(kvb_launch((moe_gemv_kernel<G_>), grid, dim3(256), smem, stream, true, (bf16*)out, (const bf16*)a, \
-                              a_stride, a_row_div, pair_weight, (const bf16*)w, ids, E, N, K, status, join));  \
+                              a_stride, a_row_div, pair_weight, (const bf16*)w, ids, E, known, N, K, status, join));  \
   } while (0)
-  if (gated) KVB_MOE_GEMV(true); else KVB_MOE_GEMV(false);
+  if (gated == 1) KVB_MOE_GEMV(true); else KVB_MOE_GEMV(false);
 #undef KVB_MOE_GEMV
   KVB_CHECK_LAUNCH();
   return 0;
@@ -585,7 +595,7 @@ moe_stream_rows_kernel(bf16* __restrict__ out, const bf16* __restrict__ a, long 
       for (int j = 0; j < 2; ++j) {
         const int n = n0 + c * 8 + 2 * q + j;
         const float v = acc[c][2 * half + j];
-        if (n < N) out[(size_t)pair * N + n] = from_float<bf16>(GATED ? moe_join<bf16>(v, acc[1][2 * half + j], join) : v);
+        if (n < N) out[(size_t)pair * N + n] = from_float<bf16>(GATED ? moe_join<bf16>(v, acc[1][2 * half + j], join) : moe_plain(v, join));
       }
   }
 }
@@ -594,13 +604,13 @@ extern "C" int kvb_moe_stream_rows(void* out, const void* a, long long a_stride,
                                    const void* w, const int* sorted, const int* tile_expert, const int* meta,
                                    int max_tiles, int N, int K, int gated, float alpha, float limit, float shift,
                                    cudaStream_t stream) {
-  const MoeJoin join = {alpha, limit, shift};
+  const MoeJoin join = {alpha, limit, shift, gated == 2};
   if (max_tiles == 0) return 0;
   KVB_REQUIRE(N > 0 && K > 0 && K % 8 == 0 && a_stride % 8 == 0 && a_row_div > 0, "moe_stream_rows: K and the row stride must be multiples of 8");
   KVB_REQUIRE(aligned16(a) && aligned16(w), "moe_stream_rows: operands must be 16-byte aligned");
   KVB_REQUIRE(max_tiles <= 65535, "moe_stream_rows: too many tiles for one launch");
   const int smem = MOE_BM * MR_PITCH * (int)sizeof(bf16);
-  const int block_cols = gated ? 64 : 128;
+  const int block_cols = gated == 1 ? 64 : 128;
   dim3 grid((N + block_cols - 1) / block_cols, max_tiles);
 #define KVB_MOE_STREAM_ROWS(G_)                                                                               \
   do {                                                                                                        \
@@ -613,7 +623,7 @@ extern "C" int kvb_moe_stream_rows(void* out, const void* a, long long a_stride,
                               (const bf16*)a, a_stride, a_row_div, pair_weight, (const bf16*)w, sorted,       \
                               tile_expert, meta, N, K, join));                                                \
   } while (0)
-  if (gated) KVB_MOE_STREAM_ROWS(true); else KVB_MOE_STREAM_ROWS(false);
+  if (gated == 1) KVB_MOE_STREAM_ROWS(true); else KVB_MOE_STREAM_ROWS(false);
 #undef KVB_MOE_STREAM_ROWS
   KVB_CHECK_LAUNCH();
   return 0;
@@ -680,7 +690,8 @@ template <typename T, bool VEC>
 __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ expert_out, int top,
                                    const int* __restrict__ row_of_pair, const float* __restrict__ pair_weight,
                                    const T* __restrict__ shared, const float* __restrict__ gate, int gate_stride,
-                                   int width, long long total_vecs) {
+                                   int width, long long total_vecs, const int* __restrict__ ids, int identity_from,
+                                   const float* __restrict__ all_weight, const T* __restrict__ input) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_MOE_COMBINE);
   constexpr int N = VEC ? Vec16<T>::N : 1;
   const int per_row = width / N;
@@ -693,17 +704,19 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ ex
     for (int j = 0; j < N; ++j) acc[j] = 0.0f;
     for (int slot = 0; slot < top; ++slot) {
       const long long pair = token * top + slot;
+      const bool own = ids != nullptr && ids[pair] >= identity_from;     // the token's input row itself
       const long long row = row_of_pair != nullptr ? row_of_pair[pair] : pair;
-      if (row < 0) continue;
-      const float w = pair_weight != nullptr ? pair_weight[pair] : 1.0f;
-      const T* src = expert_out + (size_t)row * width + col;
+      if (row < 0 && !own) continue;
+      const float w = own ? all_weight[pair] : pair_weight != nullptr ? pair_weight[pair] : 1.0f;
+      const bool weighted = own || pair_weight != nullptr;
+      const T* src = (own ? input + (size_t)token * width : expert_out + (size_t)row * width) + col;
       if (VEC) {
         Vec16<T> x;
         x.load(src);
 #pragma unroll
-        for (int j = 0; j < N; ++j) acc[j] += pair_weight != nullptr ? w * x.get(j) : x.get(j);
+        for (int j = 0; j < N; ++j) acc[j] += weighted ? w * x.get(j) : x.get(j);
       } else {
-        acc[0] += pair_weight != nullptr ? w * to_float(src[0]) : to_float(src[0]);
+        acc[0] += weighted ? w * to_float(src[0]) : to_float(src[0]);
       }
     }
     if (shared != nullptr) {
@@ -732,12 +745,14 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ ex
 
 extern "C" int kvb_moe_combine(void* out, const void* expert_out, int tokens, int top, const int* row_of_pair,
                                const float* pair_weight, const void* shared, const float* gate, int gate_stride,
-                               int width, int dtype, cudaStream_t stream) {
+                               int width, const int* ids, int identity_from, const float* all_weight,
+                               const void* input, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   KVB_REQUIRE(width > 0 && top >= 0, "moe_combine: empty rows");
+  KVB_REQUIRE(ids == nullptr || (all_weight != nullptr && input != nullptr), "moe_combine: identity experts need the weights and the input");
   const int esize = dtype == KVB_F32 ? 4 : 2;
   const bool vec = ((size_t)width * esize) % 16 == 0 && aligned16(out) && aligned16(expert_out) &&
-                   (shared == nullptr || aligned16(shared));
+                   (shared == nullptr || aligned16(shared)) && (ids == nullptr || aligned16(input));
   const long long total = (long long)tokens * (width / (vec ? 16 / esize : 1));
   const int threads = 256;
   const long long wanted = (total + threads - 1) / threads;
@@ -746,7 +761,7 @@ extern "C" int kvb_moe_combine(void* out, const void* expert_out, int tokens, in
 #define KVB_COMBINE(T_, V_)                                                                                   \
   KVB_CHECK_CUDA(kvb_launch((moe_combine_kernel<T_, V_>), dim3(blocks), dim3(threads), 0, stream, true, (T_*)out, \
                             (const T_*)expert_out, top, row_of_pair, pair_weight, (const T_*)shared, gate,     \
-                            gate_stride, width, total))
+                            gate_stride, width, total, ids, identity_from, all_weight, (const T_*)input))
   if (dtype == KVB_F32) { if (vec) KVB_COMBINE(float, true); else KVB_COMBINE(float, false); }
   else { if (vec) KVB_COMBINE(bf16, true); else KVB_COMBINE(bf16, false); }
 #undef KVB_COMBINE

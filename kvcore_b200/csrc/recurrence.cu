@@ -13,7 +13,7 @@
 //   moves the last C - 1 inputs of every request into its state row.
 //
 //   gated_rms_norm: out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * weight * silu(gate[t, h, :]) * scale
-//   (or sigmoid(gate) in place of silu(gate)).
+//   (or sigmoid(gate) in place of silu(gate); without a weight where none is given).
 #include "state_scan.cuh"
 
 // What the decay-per-channel scan reads, 32-bit [T, 3 * H * D]: q times q_scale, k, and the decays
@@ -64,73 +64,6 @@ extern "C" int kvb_gla_scan(float* out, float* prepared, const void* q, const vo
   p.heads = heads; p.kv_share = 1; p.D = D; p.V = V;
   return dtype == KVB_F32 ? launch_state_scan<float, 0>(p, num_reqs, tokens, stream)
                           : launch_state_scan<bf16, 0>(p, num_reqs, tokens, stream);
-}
-
-// What the fixed-decay scan reads, 32-bit [T, 2 * H * D + H * V]: silu(q) times q_scale, silu(k), silu(v).
-// QUADS: four neighbouring entries a thread, loaded and stored as one piece (widths that are multiples of four,
-// rows and pointers on the boundaries of such pieces).
-template <typename T>
-struct __align__(4 * sizeof(T)) ScanQuad { T v[4]; };
-
-__device__ __forceinline__ float scan_silu(float x) { return __fdividef(x, 1.0f + expf(-x)); }
-
-template <typename T, bool QUADS>
-__global__ void __launch_bounds__(256)
-lightning_prepare_kernel(float* __restrict__ out, const T* __restrict__ q, const T* __restrict__ k,
-                         const T* __restrict__ v, long long row_stride, long long tokens, int width, int vwidth,
-                         float q_scale) {
-  KVB_KERNEL_PROLOGUE(KVB_TAG_LIGHTNING_PREPARE);
-  constexpr int N = QUADS ? 4 : 1;
-  const int per_token = (2 * width + vwidth) / N;
-  const long long total = tokens * per_token;
-  for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (long long)gridDim.x * blockDim.x) {
-    const long long t = e / per_token;
-    const int i = (int)(e - t * per_token) * N;
-    const T* src = (i < width ? q + i : i < 2 * width ? k + (i - width) : v + (i - 2 * width)) + t * row_stride;
-    const float factor = i < width ? q_scale : 1.0f;
-    if (QUADS) {
-      const ScanQuad<T> in = *reinterpret_cast<const ScanQuad<T>*>(src);
-      ScanQuad<float> y;
-#pragma unroll
-      for (int j = 0; j < 4; ++j) y.v[j] = scan_silu(to_float(in.v[j])) * factor;
-      *reinterpret_cast<ScanQuad<float>*>(out + e * 4) = y;
-    } else {
-      out[e] = scan_silu(to_float(src[0])) * factor;
-    }
-  }
-}
-
-// One fixed decay a head.  q, k, v: columns of the projected rows (row stride `row_stride`, heads side by side),
-// all three passed through SiLU; decay [H] 32-bit; prepared: scratch, 32-bit [T, 2 * H * D + H * V].
-extern "C" int kvb_lightning_scan(float* out, float* prepared, const void* q, const void* k, const void* v,
-                                  long long row_stride, const float* decay, float* state, long long state_stride,
-                                  long long state_offset, const int* query_start, const int* state_slots, int tokens,
-                                  int num_reqs, int heads, int D, int V, float q_scale, int dtype,
-                                  cudaStream_t stream) {
-  if (num_reqs == 0 || tokens == 0) return 0;
-  KVB_REQUIRE(heads > 0 && D > 0 && V > 0 && decay != nullptr, "lightning_scan: bad sizes");
-  KVB_REQUIRE(heads <= 65535, "lightning_scan: too many heads");
-  const int width = heads * D, vwidth = heads * V;
-  const long long per_token = 2LL * width + vwidth;
-  const size_t piece = 4 * (dtype == KVB_F32 ? sizeof(float) : sizeof(bf16));
-  const bool quads = width % 4 == 0 && vwidth % 4 == 0 && row_stride % 4 == 0 && aligned16(prepared) &&
-                     ((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) % piece == 0;
-  const long long wanted = ((long long)tokens * per_token / (quads ? 4 : 1) + 255) / 256;
-  const long long resident = (long long)(kvb_sm_count() > 0 ? kvb_sm_count() : 1) * 16;
-  const dim3 grid((unsigned)(wanted < resident ? wanted : resident));
-#define KVB_LP_LAUNCH(T_, Q_)                                                                                  \
-  KVB_CHECK_CUDA(kvb_launch((lightning_prepare_kernel<T_, Q_>), grid, dim3(256), 0, stream, true, prepared,    \
-      (const T_*)q, (const T_*)k, (const T_*)v, row_stride, (long long)tokens, width, vwidth, q_scale))
-  if (dtype == KVB_F32) { if (quads) KVB_LP_LAUNCH(float, true); else KVB_LP_LAUNCH(float, false); }
-  else { if (quads) KVB_LP_LAUNCH(bf16, true); else KVB_LP_LAUNCH(bf16, false); }
-#undef KVB_LP_LAUNCH
-  ScanParams p = {};
-  p.q = prepared; p.k = prepared + width; p.a = decay; p.vec_token = per_token;
-  p.v = prepared + 2 * width; p.v_token = per_token;
-  p.out = out; p.state = state; p.state_stride = state_stride; p.state_offset = state_offset;
-  p.query_start = query_start; p.state_slots = state_slots;
-  p.heads = heads; p.kv_share = 1; p.D = D; p.V = V;
-  return launch_state_scan<float, 2>(p, num_reqs, tokens, stream);
 }
 
 // Delta rule.  prepared [T, 2 * G * D + H * V + 2 * H] 32-bit as conv_prepare leaves it: q, k (G heads), v, beta, gate.
@@ -293,7 +226,7 @@ gated_rms_norm_kernel(T* __restrict__ out, long long out_stride, const float* __
     for (int i = lane; i < V; i += 32) {
       const float gv = to_float(g[i]);
       const float sig = 1.0f / (1.0f + expf(-gv));
-      dst[i] = from_float<T>(src[i] * inv * to_float(weight[i]) * (sigmoid_gate ? sig : gv * sig));
+      dst[i] = from_float<T>(src[i] * inv * (weight != nullptr ? to_float(weight[i]) : 1.0f) * (sigmoid_gate ? sig : gv * sig));
     }
   }
 }
@@ -318,7 +251,7 @@ gated_rms_norm_wide_kernel(T* __restrict__ out, long long out_stride, const floa
   for (int i = threadIdx.x; i < V; i += blockDim.x) {
     const float gv = to_float(g[i]);
     const float sig = 1.0f / (1.0f + expf(-gv));
-    dst[i] = from_float<T>(src[i] * inv * to_float(weight[i]) * (sigmoid_gate ? sig : gv * sig));
+    dst[i] = from_float<T>(src[i] * inv * (weight != nullptr ? to_float(weight[i]) : 1.0f) * (sigmoid_gate ? sig : gv * sig));
   }
 }
 

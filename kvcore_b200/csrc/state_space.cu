@@ -143,6 +143,23 @@ ssm_keep_inputs_kernel(float* state, long long state_stride, long long state_off
   }
 }
 
+// The same for any mixer whose state holds the last `keep` inputs of a convolution as [keep, channels].
+extern "C" int kvb_keep_inputs(float* state, long long state_stride, long long state_offset, const void* rows,
+                               long long row_stride, int channels, int keep, const int* query_start,
+                               const int* state_slots, int num_reqs, int dtype, cudaStream_t stream) {
+  if (num_reqs == 0 || keep == 0) return 0;
+  KVB_REQUIRE(num_reqs <= 65535, "keep_inputs: too many requests for one launch");
+  const dim3 grid((channels + SSM_THREADS - 1) / SSM_THREADS, num_reqs);
+  if (dtype == KVB_F32)
+    KVB_CHECK_CUDA(kvb_launch((ssm_keep_inputs_kernel<float>), grid, dim3(SSM_THREADS), 0, stream, true, state, state_stride,
+        state_offset, (const float*)rows, row_stride, channels, keep, query_start, state_slots));
+  else
+    KVB_CHECK_CUDA(kvb_launch((ssm_keep_inputs_kernel<bf16>), grid, dim3(SSM_THREADS), 0, stream, true, state, state_stride,
+        state_offset, (const bf16*)rows, row_stride, channels, keep, query_start, state_slots));
+  KVB_CHECK_LAUNCH();
+  return 0;
+}
+
 template <typename T>
 static int launch_ssm_prepare(float* out, long long out_stride, const T* rows, long long row_stride, const float* taps,
                               int num_taps, const float* bias, float* state, long long state_stride,

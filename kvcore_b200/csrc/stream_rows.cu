@@ -4,7 +4,9 @@
 //   token's chosen experts left (ascending slot), one row for all tokens, or nothing.  From X, as asked: X itself (the new stream), its RMS norm
 //   y = X * rsqrt(mean(X^2) + eps) * w in the activation type, and the row [X | x0] in the activation type (the
 //   input of a product that reads the stream together with what it was at the start).  With a list of token rows
-//   only those are worked on and the outputs are compact.
+//   only those are worked on and the outputs are compact.  With a norm behind the sub-layer (`after`) it is
+//   X = x + a * rsqrt(mean(a^2) + eps) * w_after (+ one row for all tokens, `step`); experts without tensors then add
+//   their weight times the token's own input row.
 //
 //   embed_pairs: the first value of the stream, table[id] + pairs[row], with an RMS norm over the sum: row =
 //   (id in front * mul_prev + id * mul_cur) mod buckets, or `buckets` (the row behind the last bucket) for a
@@ -27,6 +29,10 @@ struct AddRowsParams {
   const void* rows; int top;                         // row of pair (token, slot): row_of_pair[pair], or pair itself
   const int* row_of_pair; const float* pair_weight;  // weights 1 without a list
   int one_row;                                       // every token's row is row 0
+  // experts without tensors: a pair whose id is `identity_from` or more adds all_weight[pair] * input[token]
+  const int* ids; int identity_from; const float* all_weight; const void* input;
+  const void* after; float after_eps;                // AFTER: the weight of the norm that the sum of the rows gets
+  const void* step;                                  // [width] or null: one row for all tokens, added behind that
   const int* token_rows;                             // tokens to work on, or null: all
   float* stream;                                     // [tokens, width] or null
   void* normed; const void* weight; float eps;       // [count, width] or null
@@ -34,7 +40,7 @@ struct AddRowsParams {
   int width;
 };
 
-template <typename T, typename OUT, typename W, int N>
+template <typename T, typename OUT, typename W, int N, bool AFTER>
 __global__ void __launch_bounds__(SR_THREADS)
 stream_add_rows_kernel(const AddRowsParams p) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_ADD_ROWS);
@@ -42,31 +48,52 @@ stream_add_rows_kernel(const AddRowsParams p) {
   const int n = blockIdx.x, t = p.token_rows != nullptr ? p.token_rows[n] : n;
   const int width = p.width;
   const float* x = p.x + (size_t)t * width;
-  const T* rows = (const T*)p.rows;
-  // the row and the weight of a slot of this token (row < 0: none)
-  auto slot_row = [&](int slot, float& w) {
+  // the row and the weight of a slot of this token (null: none)
+  auto slot_row = [&](int slot, float& w) -> const T* {
     const long long pair = (long long)t * p.top + slot;
+    if (AFTER && p.ids != nullptr && p.ids[pair] >= p.identity_from) {
+      w = p.all_weight[pair];
+      return (const T*)p.input + (size_t)t * width;
+    }
     w = p.pair_weight != nullptr ? p.pair_weight[pair] : 1.0f;
-    return p.row_of_pair != nullptr ? (long long)p.row_of_pair[pair] : p.one_row ? 0ll : pair;
+    const long long row = p.row_of_pair != nullptr ? (long long)p.row_of_pair[pair] : p.one_row ? 0ll : pair;
+    return row < 0 ? nullptr : (const T*)p.rows + (size_t)row * width;
   };
-  auto summed = [&](int i, float (&v)[N]) {          // one piece of the sum: what the registers do not hold
-    float a[N];
+  auto added = [&](int i, float (&a)[N]) {           // one piece of what is added: what the registers do not hold
 #pragma unroll
     for (int j = 0; j < N; ++j) a[j] = 0.0f;
     for (int slot = 0; slot < p.top; ++slot) {
       float w;
-      const long long row = slot_row(slot, w);
-      if (row < 0) continue;
-      const RowPiece<T, N> r = *reinterpret_cast<const RowPiece<T, N>*>(rows + (size_t)row * width + i);
+      const T* row = slot_row(slot, w);
+      if (row == nullptr) continue;
+      const RowPiece<T, N> r = *reinterpret_cast<const RowPiece<T, N>*>(row + i);
 #pragma unroll
       for (int j = 0; j < N; ++j) a[j] = fmaf(w, to_float(r.v[j]), a[j]);
     }
-    const RowPiece<float, N> s = *reinterpret_cast<const RowPiece<float, N>*>(x + i);
-#pragma unroll
-    for (int j = 0; j < N; ++j) v[j] = s.v[j] + a[j];
   };
   float kept[SR_PIECES][N];
-  float ss = 0.0f;
+  float ss = 0.0f, inv_a = 1.0f;
+  // the new stream from what is added
+  auto join = [&](int i, const RowPiece<float, N>& s, const RowPiece<W, N>& g, float (&v)[N]) {
+    if (AFTER) {
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] = s.v[j] + v[j] * inv_a * to_float(g.v[j]);
+      if (p.step != nullptr) {
+        const RowPiece<T, N> r = *reinterpret_cast<const RowPiece<T, N>*>((const T*)p.step + i);
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[j] += to_float(r.v[j]);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] = s.v[j] + v[j];
+    }
+  };
+  auto summed = [&](int i, float (&v)[N]) {          // one piece of the new stream, from the beginning
+    added(i, v);
+    RowPiece<W, N> g;
+    if (AFTER) g = *reinterpret_cast<const RowPiece<W, N>*>((const W*)p.after + i);
+    join(i, *reinterpret_cast<const RowPiece<float, N>*>(x + i), g, v);
+  };
   auto first_pass = [&](int i, const float (&v)[N]) {
     if (p.stream != nullptr) {
       RowPiece<float, N> s;
@@ -88,7 +115,7 @@ stream_add_rows_kernel(const AddRowsParams p) {
   };
   // the kept pieces: the stream's, the weights' and a slot's loads are each in flight together
   RowPiece<float, N> xs[SR_PIECES];
-  RowPiece<W, N> ws[SR_PIECES];
+  RowPiece<W, N> ws[SR_PIECES], gs[AFTER ? SR_PIECES : 1];
 #pragma unroll
   for (int s = 0; s < SR_PIECES; ++s) {
     const int i = (threadIdx.x + s * SR_THREADS) * N;
@@ -97,18 +124,19 @@ stream_add_rows_kernel(const AddRowsParams p) {
     if (i < width) {
       xs[s] = *reinterpret_cast<const RowPiece<float, N>*>(x + i);
       if (p.normed != nullptr) ws[s] = *reinterpret_cast<const RowPiece<W, N>*>((const W*)p.weight + i);
+      if (AFTER) gs[s] = *reinterpret_cast<const RowPiece<W, N>*>((const W*)p.after + i);
     }
   }
 #pragma unroll 2
   for (int slot = 0; slot < p.top; ++slot) {
     float w;
-    const long long row = slot_row(slot, w);
-    if (row < 0) continue;
+    const T* row = slot_row(slot, w);
+    if (row == nullptr) continue;
     RowPiece<T, N> r[SR_PIECES];
 #pragma unroll
     for (int s = 0; s < SR_PIECES; ++s) {
       const int i = (threadIdx.x + s * SR_THREADS) * N;
-      if (i < width) r[s] = *reinterpret_cast<const RowPiece<T, N>*>(rows + (size_t)row * width + i);
+      if (i < width) r[s] = *reinterpret_cast<const RowPiece<T, N>*>(row + i);
     }
 #pragma unroll
     for (int s = 0; s < SR_PIECES; ++s) {
@@ -119,17 +147,30 @@ stream_add_rows_kernel(const AddRowsParams p) {
       }
     }
   }
+  const int rest = (threadIdx.x + SR_PIECES * SR_THREADS) * N;
+  if (AFTER) {                                       // the root mean square of what is added
+    float sa = 0.0f;
+#pragma unroll
+    for (int s = 0; s < SR_PIECES; ++s)              // (pieces beyond the width are zeros)
+#pragma unroll
+      for (int j = 0; j < N; ++j) sa = fmaf(kept[s][j], kept[s][j], sa);
+    for (int i = rest; i < width; i += SR_THREADS * N) {
+      float a[N];
+      added(i, a);
+#pragma unroll
+      for (int j = 0; j < N; ++j) sa = fmaf(a[j], a[j], sa);
+    }
+    inv_a = 1.0f / sqrtf(block_sum(sa, scratch) / (float)width + p.after_eps);
+  }
 #pragma unroll
   for (int s = 0; s < SR_PIECES; ++s) {
     const int i = (threadIdx.x + s * SR_THREADS) * N;
     if (i < width) {
-#pragma unroll
-      for (int j = 0; j < N; ++j) kept[s][j] = xs[s].v[j] + kept[s][j];
+      join(i, xs[s], gs[AFTER ? s : 0], kept[s]);
       first_pass(i, kept[s]);
     }
   }
   // rows wider than the registers hold: the sum goes through `stream`, which the same thread reads again
-  const int rest = (threadIdx.x + SR_PIECES * SR_THREADS) * N;
   for (int i = rest; i < width; i += SR_THREADS * N) {
     float v[N];
     summed(i, v);
@@ -167,23 +208,33 @@ stream_add_rows_kernel(const AddRowsParams p) {
 extern "C" int kvb_stream_add_rows(const float* x, const void* rows, int top, const int* row_of_pair,
                                    const float* pair_weight, int one_row, const int* token_rows, int count, float* stream,
                                    void* normed, const void* weight, float eps, void* packed, const float* origin,
-                                   int width, int dtype, int out_dtype, int weight_dtype, cudaStream_t cuda_stream) {
+                                   const void* after, float after_eps, const void* step, const int* ids,
+                                   int identity_from, const float* all_weight, const void* input, int width, int dtype, int out_dtype, int weight_dtype, cudaStream_t cuda_stream) {
   if (count == 0) return 0;
   KVB_REQUIRE(width > 0 && top >= 0 && x != nullptr && (rows != nullptr || top == 0), "stream_add_rows: empty rows");
   KVB_REQUIRE(normed == nullptr || weight != nullptr, "stream_add_rows: the norm needs its weight");
   KVB_REQUIRE(packed == nullptr || origin != nullptr, "stream_add_rows: the packed rows need what the stream started as");
   KVB_REQUIRE(token_rows == nullptr || stream == nullptr, "stream_add_rows: a list of tokens leaves the stream alone");
+  KVB_REQUIRE(after != nullptr || (step == nullptr && ids == nullptr),
+              "stream_add_rows: a step row and identity experts come with the norm behind the sub-layer");
+  KVB_REQUIRE(ids == nullptr || (all_weight != nullptr && input != nullptr),
+              "stream_add_rows: identity experts need the weights and the input rows");
   AddRowsParams p;
+  p.after = after; p.after_eps = after_eps; p.step = step; p.ids = ids; p.identity_from = identity_from;
+  p.all_weight = all_weight; p.input = input;
   p.x = x; p.rows = rows; p.top = top; p.row_of_pair = row_of_pair; p.pair_weight = pair_weight;
   p.one_row = one_row; p.token_rows = token_rows; p.stream = stream; p.normed = normed; p.weight = weight; p.eps = eps; p.packed = packed;
   p.origin = origin; p.width = width;
   const bool quads = width % 4 == 0 && aligned16(x) && aligned16(rows) && (stream == nullptr || aligned16(stream)) &&
                      (normed == nullptr || (aligned16(normed) && aligned16(weight))) &&
-                     (packed == nullptr || (aligned16(packed) && aligned16(origin)));
+                     (packed == nullptr || (aligned16(packed) && aligned16(origin))) && aligned16(after) &&
+                     aligned16(step) && aligned16(input);
   cudaError_t err;
-#define KVB_AR(T, OUT, W)                                                                                              \
-  err = quads ? kvb_launch((stream_add_rows_kernel<T, OUT, W, 4>), dim3(count), dim3(SR_THREADS), 0, cuda_stream, true, p) \
-              : kvb_launch((stream_add_rows_kernel<T, OUT, W, 1>), dim3(count), dim3(SR_THREADS), 0, cuda_stream, true, p)
+#define KVB_AR_SHAPE(T, OUT, W, N, A) \
+  kvb_launch((stream_add_rows_kernel<T, OUT, W, N, A>), dim3(count), dim3(SR_THREADS), 0, cuda_stream, true, p)
+#define KVB_AR(T, OUT, W)                                                                              \
+  err = after != nullptr ? (quads ? KVB_AR_SHAPE(T, OUT, W, 4, true) : KVB_AR_SHAPE(T, OUT, W, 1, true)) \
+                         : (quads ? KVB_AR_SHAPE(T, OUT, W, 4, false) : KVB_AR_SHAPE(T, OUT, W, 1, false))
   const int code = (dtype == KVB_BF16 ? 4 : 0) | (out_dtype == KVB_BF16 ? 2 : 0) | (weight_dtype == KVB_BF16 ? 1 : 0);
   switch (code) {
     case 0: KVB_AR(float, float, float); break;
@@ -196,6 +247,7 @@ extern "C" int kvb_stream_add_rows(const float* x, const void* rows, int top, co
     default: KVB_AR(bf16, bf16, bf16); break;
   }
 #undef KVB_AR
+#undef KVB_AR_SHAPE
   KVB_CHECK_CUDA(err);
   KVB_CHECK_LAUNCH();
   return 0;

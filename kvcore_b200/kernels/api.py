@@ -53,14 +53,14 @@ def ensure_built(verbose: bool = False) -> str:
         "kvb_glu_clamped": [_vp, _vp, _int, _int, _float, _float, _float, _int, _vp],
         "kvb_moe_route": [_vp, _vp, _vp, _vp, _ll, _vp, _vp, _int, _int, _int, _int, _int, _int, _int, _vp, _int, _int,
                           _float, _vp, _int, _vp],
-        "kvb_moe_align": [_vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _vp],
-        "kvb_moe_gemv": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _int, _int, _int, _int, _int, _float, _float, _float, _vp],
+        "kvb_moe_align": [_vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _vp],
+        "kvb_moe_gemv": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _int, _int, _int, _int, _int, _int, _float, _float, _float, _vp],
         "kvb_moe_stream_rows": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _float, _float,
                                 _float, _vp],
         "kvb_moe_gather": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _int, _int, _vp, _int, _int, _vp],
         "kvb_moe_gemm": [_vp, _vp, _ll, _int, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _float, _float, _float,
                          _int, _vp],
-        "kvb_moe_combine": [_vp, _vp, _int, _int, _vp, _vp, _vp, _vp, _int, _int, _int, _vp],
+        "kvb_moe_combine": [_vp, _vp, _int, _int, _vp, _vp, _vp, _vp, _int, _int, _vp, _int, _vp, _vp, _int, _vp],
         "kvb_flash_paged_attention": [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _int, _vp, _vp, _int, _int, _int,
                                       _int, _int, _int, _int, _float, _int, _int, _vp, _vp, _vp],
         "kvb_kept_first_merge": [_vp, _int, _vp, _vp, _int, _vp, _vp, _vp, _int, _vp, _vp, _int, _int, _int, _int,
@@ -75,11 +75,11 @@ def ensure_built(verbose: bool = False) -> str:
         "kvb_rms_norm_shift": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _float, _int, _int, _int, _vp],
         "kvb_stream_add_norm": [_vp, _vp, _vp, _vp, _int, _int, _float, _vp, _vp, _ll, _vp, _int, _vp, _int, _int, _vp],
         "kvb_attention_dims_rows": [_vp, _ll, _ll, _int, _vp, _ll, _ll, _vp, _ll, _ll, _ll, _vp, _ll, _ll, _ll, _vp,
-                                    _int, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _int, _int, _int, _int, _float,
+                                    _int, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _int, _int, _int, _int, _float, _float,
                                     _int, _int, _vp],
         "kvb_flash_dims_attention": [_vp, _ll, _ll, _int, _vp, _ll, _ll, _vp, _ll, _ll, _ll, _vp, _ll, _ll, _ll, _vp,
                                      _int, _vp, _vp, _vp, _vp, _int, _int, _int, _int, _int, _int, _int, _int, _int,
-                                     _float, _int, _int, _vp, _vp],
+                                     _float, _float, _int, _int, _vp, _vp],
         "kvb_latent_prepare": [_vp, _ll, _vp, _float, _vp, _int, _vp, _vp, _vp, _int, _vp, _int, _int, _int, _vp,
                                _ll, _ll, _int, _vp, _ll, _ll, _vp, _int, _int, _int, _int, _int, _int, _vp],
         "kvb_gather_cached_rows": [_vp, _ll, _ll, _int, _vp, _int, _int, _int, _vp, _vp, _int, _vp, _int, _int,
@@ -102,8 +102,13 @@ def ensure_built(verbose: bool = False) -> str:
                             _int, _int, _int, _vp],
         "kvb_ssm_scan": [_vp, _vp, _ll, _vp, _vp, _ll, _ll, _vp, _vp, _int, _int, _int, _int, _int, _int, _vp],
         "kvb_gated_group_norm": [_vp, _ll, _vp, _vp, _ll, _vp, _int, _int, _int, _float, _int, _vp],
-        "kvb_stream_add_rows": [_vp, _vp, _int, _vp, _vp, _int, _vp, _int, _vp, _vp, _vp, _float, _vp, _vp, _int, _int, _int,
-                                _int, _vp],
+        "kvb_stream_add_rows": [_vp, _vp, _int, _vp, _vp, _int, _vp, _int, _vp, _vp, _vp, _float, _vp, _vp, _vp, _float, _vp,
+                                _vp, _int, _vp, _vp, _int, _int, _int, _int, _vp],
+        "kvb_attention_prepare": [_vp, _ll, _vp, _ll, _vp, _int, _vp, _vp, _vp, _vp, _vp, _int, _vp, _int, _int, _int, _int,
+                                  _int, _int, _int, _int, _int, _vp, _int, _vp, _ll, _ll, _vp, _vp, _float, _int, _vp],
+        "kvb_retention_scan": [_vp, _vp, _vp, _vp, _vp, _ll, _vp, _int, _vp, _vp, _ll, _ll, _vp, _vp, _int, _int, _int, _int,
+                               _int, _float, _int, _vp],
+        "kvb_relu_squared": [_vp, _ll, _int, _vp],
         "kvb_embed_pairs": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _int, _ll, _ll, _ll, _float,
                             _int, _vp],
         "kvb_softcap": [_vp, _ll, _float, _float, _vp],
@@ -685,14 +690,15 @@ TRACE_TAGS = {27: "rms_norm_shift", 28: "stream_add_norm", 29: "attention_dims_r
               31: "head_norm_kv_write", 32: "maps_combine", 33: "sigmoid_gate_mul", 34: "flash_dims",
               35: "flash_dims_combine", 36: "gather_cached_rows", 37: "gla_scan", 38: "delta_scan", 39: "conv_prepare",
               40: "gated_rms_norm", 41: "turn_norm_kv_write", 42: "head_gate", 43: "embed_scaled", 44: "gla_prepare", 45: "gelu_mul", 46: "lightning_prepare", 47: "lightning_scan", 48: "ssm_scan",
-              49: "ssm_prepare", 50: "gated_group_norm", 51: "stream_add_rows", 52: "embed_pairs", 53: "softcap", 25: "kept_first_merge", 26: "moe_gather", 17: "layer_norm", 18: "stream_add", 19: "qk_prepare", 20: "glu_clamped", 21: "moe_route",
+              49: "ssm_prepare", 50: "gated_group_norm", 51: "stream_add_rows", 52: "embed_pairs", 53: "softcap", 54: "attention_prepare", 55: "retention_prepare",
+              56: "relu_squared", 25: "kept_first_merge", 26: "moe_gather", 17: "layer_norm", 18: "stream_add", 19: "qk_prepare", 20: "glu_clamped", 21: "moe_route",
               22: "moe_align", 23: "moe_gemm", 24: "moe_combine", 1: "gather_rows", 2: "rmsnorm", 3: "silu_mul", 4: "rope_table", 5: "rope_kv_write", 6: "attention_rows",
               7: "flash_paged", 8: "flash_combine", 9: "flash_decode_tma", 10: "flash_decode_combine",
               11: "flash_prefill_tc5", 12: "gemm_f32", 13: "gemm_stream", 14: "sample", 16: "feed_tokens"}
 _TRACE_UNITS = ("elementwise", "attention_decode_tma", "attention_flash", "attention_generic",
                 "attention_prefill_tc5", "gemm_f32", "sampling", "gemm_stream", "layer_norm", "qk_prepare", "moe", "attention_kept_first",
                 "stream_norm", "attention_dims", "mixer_prepare", "attention_flash_dims", "recurrence", "turn_norm",
-                "state_space", "stream_rows")
+                "state_space", "stream_rows", "fixed_decay", "attention_prepare")
 _trace_buffer: torch.Tensor | None = None
 
 
@@ -749,12 +755,14 @@ def set_overlapped_launch(enabled: bool) -> None:
 
 
 def linear_stream(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None, *,
-                  out_dtype: torch.dtype | None = None, silu_pairs: bool = False) -> torch.Tensor:
+                  out_dtype: torch.dtype | None = None, silu_pairs: bool = False,
+                  square_relu: bool = False) -> torch.Tensor:
     """``x @ weight.T`` for a decode-sized batch of bf16 ``x`` (at most 16 rows), K a multiple of 64: a
     balanced weight-streaming kernel (one block per SM, every block the same number of bytes).
 
     ``silu_pairs``: the rows of ``weight`` alternate in runs of 8 gate rows and 8 up rows; the
-    result is ``[M, N/2]``, ``silu(gate) * up``, with the roundings of the unfused path."""
+    result is ``[M, N/2]``, ``silu(gate) * up``, with the roundings of the unfused path.
+    ``square_relu``: the result is ``max(x @ weight.T + bias, 0)^2``, formed from the 32-bit sums."""
     _check(x, "x", dtype=torch.bfloat16, contiguous=False)
     _check(weight, "weight", dtype=torch.bfloat16)
     m, k = x.shape
@@ -765,10 +773,12 @@ def linear_stream(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | No
         _check(bias, "bias", dtype=torch.bfloat16)
     if silu_pairs and (n % 16 or out_dtype not in (None, torch.bfloat16)):
         raise KernelError("linear_stream: gated pairs need an output width that is a multiple of 16 and a bf16 result")
+    if silu_pairs and square_relu:
+        raise KernelError("linear_stream: one activation at a time")
     out = torch.empty((m, n // 2 if silu_pairs else n), dtype=out_dtype or torch.bfloat16, device=x.device)
     _stream_call(x.device, out.data_ptr(), int(out.dtype == torch.float32), out.stride(0),
                  x.data_ptr(), x.stride(0), weight.data_ptr(), None if bias is None else bias.data_ptr(),
-                 m, n, k, int(silu_pairs), None, 0, 0.0, None, 0, None, None)
+                 m, n, k, 1 if silu_pairs else 2 if square_relu else 0, None, 0, 0.0, None, 0, None, None)
     return out
 
 
@@ -863,6 +873,23 @@ def linear_silu_mul(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | 
     if group == 8 and x.dim() == 2 and _stream_ok(x, weight) and weight.shape[0] % 16 == 0:
         return linear_stream(x, weight, bias, silu_pairs=True)
     return silu_mul(linear(x, weight, bias), group)
+
+
+def relu_squared(x: torch.Tensor) -> torch.Tensor:
+    """``max(x, 0)^2`` in place."""
+    _check(x, "x")
+    _call("kvb_relu_squared", x.data_ptr(), x.numel(), _dtype_code(x), _stream())
+    return x
+
+
+def linear_relu_squared(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """The first half of an ungated feed-forward: ``max(x @ weight.T, 0)^2``.  Decode-sized bf16 batches take the
+    streaming kernel with the activation in its epilogue; everything else is the product and then the activation."""
+    _check(x, "x", contiguous=False)
+    _check(weight, "weight", dtype=x.dtype)
+    if x.dim() == 2 and x.shape[1] == weight.shape[1] and _stream_ok(x, weight):
+        return linear_stream(x, weight, square_relu=True)
+    return relu_squared(linear(x, weight))
 
 
 def norm_linear(h: torch.Tensor | None, residual: torch.Tensor | None, norm_weight: torch.Tensor, eps: float,
@@ -1052,14 +1079,17 @@ def stream_add_norm(x: torch.Tensor, a: torch.Tensor, weight: torch.Tensor, eps:
 
 def stream_add_rows(x: torch.Tensor, a, *, weight: torch.Tensor | None = None, eps: float = 0.0,
                     out_dtype: torch.dtype | None = None, token_rows: torch.Tensor | None = None,
-                    origin: torch.Tensor | None = None, keep: bool = True) -> tuple:
+                    origin: torch.Tensor | None = None, keep: bool = True, after: tuple | None = None,
+                    step: torch.Tensor | None = None) -> tuple:
     """``X = x + a`` on the 32-bit stream ``x [T, width]``, ``a`` a sub-layer's output ``[T, width]``, one row for all
     tokens ``[1, width]``, the rows a sub-layer's experts left (``ExpertRows``: summed per token in ascending slot,
     weights still pending included), or None.  Returns
     ``(X, y, packed)``: ``X`` is ``x`` updated in place (``keep`` False or ``token_rows`` given: ``x`` stays and
     ``X`` is None); ``y = X * rsqrt(mean(X^2) + eps) * weight`` in ``out_dtype`` (with ``weight``, else None);
     ``packed [T, 2 * width]`` = ``[X | origin]`` in ``out_dtype`` (with ``origin``, a stream of the same shape, else
-    None).  ``token_rows`` (int32): only those tokens, the outputs compact and in their order."""
+    None).  ``token_rows`` (int32): only those tokens, the outputs compact and in their order.  ``after = (weight,
+    eps)``: what is added gets an RMS norm first, ``X = x + a * rsqrt(mean(a^2) + eps) * weight``, and then ``step``
+    (``[1, width]``, one row for all tokens) is added too."""
     experts = a if isinstance(a, ExpertRows) else None
     rows = a if experts is None else experts.rows
     _check(x, "x", dtype=torch.float32)
@@ -1101,12 +1131,37 @@ def stream_add_rows(x: torch.Tensor, a, *, weight: torch.Tensor | None = None, e
             raise KernelError("stream_add_rows: origin does not match the stream")
         packed = torch.empty((count, 2 * width), dtype=dtype, device=x.device)
     code = _BF16 if dtype == torch.bfloat16 else _F32
+    behind, identity = (None, 0.0, None), (None, 0, None, None)
+    if after is not None:
+        after_weight = after[0]
+        _check(after_weight, "after weight")
+        if rows is None or after_weight.numel() != width or (weight is not None and after_weight.dtype != weight.dtype):
+            raise KernelError(f"stream_add_rows: the norm behind the sub-layer ({after_weight.numel()} weights of "
+                              f"{after_weight.dtype}) does not fit rows of width {width}")
+        weight_code = _dtype_code(after_weight)
+        if step is not None:
+            _check(step, "step", dtype=rows.dtype)
+            if step.numel() != width:
+                raise KernelError(f"stream_add_rows: a step row of {step.numel()} entries for rows of width {width}")
+        behind = (after_weight.data_ptr(), float(after[1]), None if step is None else step.data_ptr())
+    elif step is not None:
+        raise KernelError("stream_add_rows: a step row comes with the norm behind the sub-layer")
+    if experts is not None and experts.identity is not None:
+        ids, all_weights, own, first = experts.identity
+        if after is None:
+            raise KernelError("stream_add_rows: identity experts are summed together with the norm behind them")
+        _check(ids, "ids", dtype=torch.int32)
+        _check(all_weights, "weights", dtype=torch.float32)
+        _check(own, "input rows", dtype=rows.dtype)
+        if tuple(own.shape) != (tokens, width) or ids.numel() != tokens * top or all_weights.numel() != tokens * top:
+            raise KernelError(f"stream_add_rows: input rows {tuple(own.shape)} of identity experts do not fit")
+        identity = (ids.data_ptr(), int(first), all_weights.data_ptr(), own.data_ptr())
     _call("kvb_stream_add_rows", x.data_ptr(), None if rows is None else rows.data_ptr(), int(top),
           None if row_of_pair is None else row_of_pair.data_ptr(), None if pair_weight is None else pair_weight.data_ptr(),
           int(experts is None and rows is not None and rows.shape[0] == 1), None if token_rows is None else token_rows.data_ptr(), count, x.data_ptr() if keep else None,
           None if normed is None else normed.data_ptr(), None if weight is None else weight.data_ptr(), float(eps),
-          None if packed is None else packed.data_ptr(), None if origin is None else origin.data_ptr(), width,
-          code if rows is None else _dtype_code(rows), code, weight_code, _stream())
+          None if packed is None else packed.data_ptr(), None if origin is None else origin.data_ptr(), *behind,
+          *identity, width, code if rows is None else _dtype_code(rows), code, weight_code, _stream())
     return (x if keep else None), normed, packed
 
 
@@ -1116,7 +1171,7 @@ def attention_dims(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, ta
                    sink: torch.Tensor | None = None, window: int | None = None,
                    out: torch.Tensor | None = None, out_dtype: torch.dtype | None = None,
                    force_general: bool = False, num_splits: int | None = None,
-                   slopes: torch.Tensor | None = None) -> torch.Tensor:
+                   slopes: torch.Tensor | None = None, softcap: float | None = None) -> torch.Tensor:
     """Paged attention with a key width and a value width of their own.
 
     ``q [T, HQ, key_width]`` (a view; last stride 1) with ``HQ = value_heads * group * maps``: query head
@@ -1125,7 +1180,8 @@ def attention_dims(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, ta
     view of ``keys``); ``key_strides`` / ``value_strides`` give their (page, head, row) strides in elements;
     page ``p`` slot ``s`` head ``h`` starts at ``p * page + h * head + s * row``.  ``sink [HQ]`` (32-bit):
     a logit per query head that joins the softmax's denominator.  ``slopes [HQ]`` (32-bit): query head ``hq``'s
-    score of the key at position ``j`` for the query at position ``i`` is lowered by ``slopes[hq] * (i - j)``.  Returns ``[T, HQ, value_width]`` in
+    score of the key at position ``j`` for the query at position ``i`` is lowered by ``slopes[hq] * (i - j)``.
+    ``softcap``: the scaled score first becomes ``softcap * tanh(score / softcap)``.  Returns ``[T, HQ, value_width]`` in
     ``out_dtype`` (32-bit or the cache's type; default the cache's) or fills ``out`` (a view with last
     stride 1).  bfloat16 shapes the tensor-core kernel takes run there; everything else, and all of float32,
     on the general kernel."""
@@ -1149,19 +1205,21 @@ def attention_dims(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, ta
         _check(slopes, "slopes", dtype=torch.float32)
         if slopes.numel() != hq:
             raise KernelError(f"attention_dims: {slopes.numel()} slopes for {hq} query heads")
+    if softcap is not None and not softcap > 0:
+        raise KernelError(f"attention_dims: the scores' cap must be positive, got {softcap}")
     if tokens == 0:
         return out
     if (not force_general and flash_dims_supported(q, out, key_width, value_width, page_size, key_strides,
                                                     value_strides, keys, values, maps)):
         _flash_dims(out, q, keys, values, table, ctx, value_heads, group, maps, key_width, value_width, page_size,
-                    num_pages, key_strides, value_strides, scale, sink, window, num_splits, slopes)
+                    num_pages, key_strides, value_strides, scale, sink, window, num_splits, slopes, softcap)
         return out
     _call("kvb_attention_dims_rows", out.data_ptr(), out.stride(0), out.stride(1), int(out.dtype == torch.float32),
           q.data_ptr(), q.stride(0), q.stride(1), keys.data_ptr(), *key_strides, values.data_ptr(), *value_strides,
           table.data_ptr(), table.stride(0), ctx.positions.data_ptr(), ctx.req_index.data_ptr(),
           None if sink is None else sink.data_ptr(), None if slopes is None else slopes.data_ptr(), tokens, hq,
-          group * maps, maps, key_width, value_width, page_size, num_pages, float(scale), int(window or 0),
-          _dtype_code(q), _stream())
+          group * maps, maps, key_width, value_width, page_size, num_pages, float(scale), float(softcap or 0.0),
+          int(window or 0), _dtype_code(q), _stream())
     return out
 
 
@@ -1208,7 +1266,7 @@ def flash_dims_supported(q, out, key_width, value_width, page_size, key_strides,
 
 
 def _flash_dims(out, q, keys, values, table, ctx, value_heads, group, maps, key_width, value_width, page_size,
-                num_pages, key_strides, value_strides, scale, sink, window, num_splits, slopes=None) -> None:
+                num_pages, key_strides, value_strides, scale, sink, window, num_splits, slopes=None, softcap=None) -> None:
     """The tensor-core kernel on the step's batch.  A mixed step (portions of prompts beside single decoded
     tokens, longest first as the step function packs them) goes as two runs of requests, so that the
     decoded tokens take the shape made for few rows and have their keys cut into chunks."""
@@ -1251,8 +1309,8 @@ def _flash_dims(out, q, keys, values, table, ctx, value_heads, group, maps, key_
               values.data_ptr(), *value_strides, run_table.data_ptr(), run_table.stride(0),
               run.query_start.data_ptr(), run.context_lens.data_ptr(), None if sink is None else sink.data_ptr(),
               None if slopes is None else slopes.data_ptr(), run.num_reqs, run.max_query_len, value_heads, group, maps, key_width, value_width, page_size,
-              num_pages, float(scale), int(window or 0), splits, None if scratch is None else scratch.data_ptr(),
-              _stream(), kernels=2 if splits > 1 else 1)
+              num_pages, float(scale), float(softcap or 0.0), int(window or 0), splits,
+              None if scratch is None else scratch.data_ptr(), _stream(), kernels=2 if splits > 1 else 1)
 
 
 def latent_prepare(kv_rows: torch.Tensor, norm_weight: torch.Tensor, eps: float, inv_freq: torch.Tensor, dims: int,
@@ -1377,14 +1435,19 @@ def maps_combine(a: torch.Tensor, lam: float, eps: float, out_scale: float, out_
     return out
 
 
-def sigmoid_gate_mul(o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
-    """``o [T, H, width]`` (a view) times ``sigmoid(gate [T, H * width])`` (a view of rows) -> ``[T, H * width]``."""
+def sigmoid_gate_mul(o: torch.Tensor, gate: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``o [T, H, width]`` (a view) times ``sigmoid(gate [T, H * width])`` (a view of rows) -> ``[T, H * width]``
+    (into ``out``, contiguous, when given)."""
     _check(o, "o", contiguous=False)
     _check(gate, "gate", dtype=o.dtype, contiguous=False)
     tokens, heads, width = o.shape
     if o.stride(2) != 1 or gate.stride(1) != 1 or tuple(gate.shape) != (tokens, heads * width):
         raise KernelError(f"sigmoid_gate_mul: o {tuple(o.shape)} and gate {tuple(gate.shape)} do not fit")
-    out = torch.empty((tokens, heads * width), dtype=o.dtype, device=o.device)
+    if out is None:
+        out = torch.empty((tokens, heads * width), dtype=o.dtype, device=o.device)
+    _check(out, "out", dtype=o.dtype)
+    if tuple(out.shape) != (tokens, heads * width):
+        raise KernelError(f"sigmoid_gate_mul: out {tuple(out.shape)} does not fit o {tuple(o.shape)}")
     _call("kvb_sigmoid_gate_mul", out.data_ptr(), o.data_ptr(), o.stride(0), o.stride(1), gate.data_ptr(),
           gate.stride(0), tokens, heads, width, _dtype_code(o), _stream())
     return out
@@ -1626,10 +1689,10 @@ def delta_scan(prepared: torch.Tensor, state: torch.Tensor, ctx, *, heads: int, 
     return out
 
 
-def gated_rms_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+def gated_rms_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor | None, eps: float, out: torch.Tensor,
                    scale: float = 1.0, *, gate_act: str = "silu") -> torch.Tensor:
     """``out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight * silu(gate[t, h, :]) * scale``:
-    ``o [T, H, V]`` 32-bit, ``gate`` and ``out [T, H * V]`` views of the activation type, ``weight [V]``.
+    ``o [T, H, V]`` 32-bit, ``gate`` and ``out [T, H * V]`` views of the activation type, ``weight [V]`` (or None: no factor).
     ``gate_act="sigmoid"``: ``sigmoid(gate)`` in place of ``silu(gate)``.  (A norm over all heads together is
     the case ``H = 1``.)"""
     if gate_act not in ("silu", "sigmoid"):
@@ -1637,14 +1700,17 @@ def gated_rms_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, ep
     _check(o, "o", dtype=torch.float32)
     _check(gate, "gate", contiguous=False)
     _check(out, "out", dtype=gate.dtype, contiguous=False)
-    _check(weight, "weight", dtype=gate.dtype)
+    if weight is not None:
+        _check(weight, "weight", dtype=gate.dtype)
     tokens, heads, width = o.shape
     if (tuple(gate.shape) != (tokens, heads * width) or tuple(out.shape) != (tokens, heads * width)
-            or weight.numel() != width or (tokens and (gate.stride(1) != 1 or out.stride(1) != 1))):
+            or (weight is not None and weight.numel() != width)
+            or (tokens and (gate.stride(1) != 1 or out.stride(1) != 1))):
         raise KernelError(f"gated_rms_norm: gate {tuple(gate.shape)} / out {tuple(out.shape)} / weight do not fit "
                           f"o {tuple(o.shape)}")
     _call("kvb_gated_rms_norm", out.data_ptr(), out.stride(0), o.data_ptr(), gate.data_ptr(), gate.stride(0),
-          weight.data_ptr(), tokens, heads, width, float(eps), float(scale), int(gate_act == "sigmoid"),
+          None if weight is None else weight.data_ptr(), tokens, heads, width, float(eps), float(scale),
+          int(gate_act == "sigmoid"),
           _dtype_code(out), _stream())
     return out
 
@@ -1677,6 +1743,101 @@ def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
           ctx.state_slots.data_ptr(), q.shape[0], ctx.num_reqs, heads, dim, value_dim, float(q_scale),
           _dtype_code(q), _stream(), kernels=2)
     return out
+
+
+def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cos_sin: torch.Tensor | None, decay: torch.Tensor,
+                   state: torch.Tensor, ctx, *, heads: int, dim: int, value_dim: int, k_scale: float,
+                   state_offset: int = 0) -> torch.Tensor:
+    """Linear attention with one fixed decay a head on turned projections, request by request in order:
+    ``S <- decay[h] S + k_t v_t^T``, ``o_t = S^T q_t``.  ``q, k [T, heads * dim]`` and ``v [T, heads * value_dim]`` are
+    views of one tensor of projected rows; the first ``2 * cos_sin.shape[1]`` entries of every q and k head turn in
+    halves with the ``[T, rot / 2, 2]`` 32-bit table ``cos_sin`` (None: nothing turns), k is then multiplied by
+    ``k_scale``.  ``decay [heads]`` 32-bit; ``state [slots, n]`` (32-bit) holds each request's ``S`` column by column
+    (``[heads, value_dim, dim]``) at ``state_offset`` of its slot's row and is brought up to date.  Returns
+    ``o [T, heads, value_dim]`` 32-bit."""
+    for name, t in (("q", q), ("k", k), ("v", v)):
+        _check(t, name, dtype=q.dtype, contiguous=False)
+        if t.stride(1) != 1 or t.shape[0] != q.shape[0]:
+            raise KernelError(f"retention_scan: {name} {tuple(t.shape)} is not a view of the step's rows")
+    if q.stride(0) != k.stride(0) or q.stride(0) != v.stride(0):
+        raise KernelError("retention_scan: q, k and v must be views of one tensor of rows")
+    if q.shape[1] != heads * dim or k.shape[1] != heads * dim or v.shape[1] != heads * value_dim:
+        raise KernelError("retention_scan: widths do not match the head layout")
+    _check(decay, "decay", dtype=torch.float32)
+    if decay.numel() != heads:
+        raise KernelError(f"retention_scan: {decay.numel()} decays for {heads} heads")
+    rot = _turned_entries(cos_sin, q.shape[0], dim, "retention_scan")
+    _state_row(state, state_offset, heads * dim * value_dim)
+    out = torch.empty((q.shape[0], heads, value_dim), dtype=torch.float32, device=q.device)
+    # what the scan reads a token, 32-bit: the turned q and k
+    prepared = torch.empty((q.shape[0], 2 * heads * dim), dtype=torch.float32, device=q.device)
+    _call("kvb_retention_scan", out.data_ptr(), prepared.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(),
+          q.stride(0), None if cos_sin is None else cos_sin.data_ptr(), rot, decay.data_ptr(), state.data_ptr(),
+          state.stride(0), state_offset, ctx.query_start.data_ptr(), ctx.state_slots.data_ptr(), q.shape[0],
+          ctx.num_reqs, heads, dim, value_dim, float(k_scale), _dtype_code(q), _stream(), kernels=2)
+    return out
+
+
+def _turned_entries(cos_sin: torch.Tensor | None, tokens: int, dim: int, who: str) -> int:
+    """Entries of a head that turn with the table ``cos_sin [tokens, rot / 2, 2]`` (None: 0)."""
+    if cos_sin is None:
+        return 0
+    _check(cos_sin, "cos_sin", dtype=torch.float32)
+    if cos_sin.dim() != 3 or cos_sin.shape[0] != tokens or cos_sin.shape[2] != 2 or 2 * cos_sin.shape[1] > dim:
+        raise KernelError(f"{who}: cos_sin has shape {tuple(cos_sin.shape)} for {tokens} tokens and heads of {dim}")
+    return 2 * cos_sin.shape[1]
+
+
+def attention_prepare(rows: torch.Tensor, q_out: torch.Tensor, cos_sin: torch.Tensor | None, ctx, table: torch.Tensor,
+                      cache: torch.Tensor, *, q_heads: int, k_heads: int, dim: int, value_width: int,
+                      taps: torch.Tensor | None = None, state: torch.Tensor | None = None, state_offset: int = 0,
+                      q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None, eps: float = 0.0,
+                      write: bool = True) -> None:
+    """Between the projections and the attention: ``rows [T, >= (q_heads + k_heads) * dim + value_width]`` (a view) hold a
+    token's q, k and v.  In order, each where given: ``taps [K, channels]``, a causal convolution over time on every
+    channel (the last tap on the current token; the ``K - 1`` inputs in front of a portion are the request's
+    ``state[slot, state_offset:]`` as ``[K - 1, channels]``, brought up to date by this call); ``q_weight`` /
+    ``k_weight``, one RMS norm over all of q and one over all of k; ``cos_sin [T, rot / 2, 2]``, a turn of the first
+    ``rot`` entries of every q and k head in halves.  q goes to ``q_out [T, q_heads * dim]`` (a view; without taps it may
+    be q's own columns); with ``write`` k and v go side by side into the token's row of
+    ``cache [pages, 1, page, k_heads * dim + value_width]``."""
+    _check(rows, "rows", contiguous=False)
+    _check(q_out, "q_out", dtype=rows.dtype, contiguous=False)
+    _check(cache, "cache", dtype=rows.dtype)
+    _check(table, "block table", dtype=torch.int32, contiguous=False)
+    tokens = rows.shape[0]
+    q_len, k_len = q_heads * dim, k_heads * dim
+    channels = q_len + k_len + value_width
+    if rows.shape[1] < channels or tuple(q_out.shape) != (tokens, q_len) or (tokens and (rows.stride(1) != 1 or q_out.stride(1) != 1)):
+        raise KernelError(f"attention_prepare: rows {tuple(rows.shape)} / q_out {tuple(q_out.shape)} do not hold the heads")
+    rot = _turned_entries(cos_sin, tokens, dim, "attention_prepare")
+    num_pages, one, page_size, width = cache.shape
+    if one != 1 or width != k_len + value_width or table.stride(1) != 1:
+        raise KernelError(f"attention_prepare: cache {tuple(cache.shape)} does not hold rows of {k_len} + {value_width}")
+    kept = (None, 0, None, 0, 0)
+    if taps is not None:
+        _check(taps, "taps", dtype=rows.dtype)
+        if taps.dim() != 2 or taps.shape[0] < 1 or taps.shape[1] != channels:
+            raise KernelError(f"attention_prepare: taps {tuple(taps.shape)} for {channels} channels")
+        kept = (taps.data_ptr(), taps.shape[0], None, 0, 0)
+        if taps.shape[0] > 1:
+            if state is None:
+                raise KernelError("attention_prepare: a convolution needs the state rows")
+            _state_row(state, state_offset, channels * (taps.shape[0] - 1))
+            kept = (taps.data_ptr(), taps.shape[0], state.data_ptr(), state.stride(0), state_offset)
+    for name, w, n in (("q_weight", q_weight, q_len), ("k_weight", k_weight, k_len)):
+        if w is not None:
+            _check(w, name, dtype=rows.dtype)
+            if w.numel() != n:
+                raise KernelError(f"attention_prepare: {name} has {w.numel()} entries, not {n}")
+    slots = getattr(ctx, "state_slots", None) if kept[2] is not None else None
+    _call("kvb_attention_prepare", rows.data_ptr(), rows.stride(0), q_out.data_ptr(), q_out.stride(0),
+          None if cos_sin is None else cos_sin.data_ptr(), rot, ctx.positions.data_ptr(), ctx.req_index.data_ptr(),
+          ctx.query_start.data_ptr(), None if slots is None else slots.data_ptr(), table.data_ptr(), table.stride(0),
+          cache.data_ptr(), page_size, num_pages, int(bool(write)), tokens, ctx.num_reqs, q_heads, k_heads, dim,
+          value_width, *kept, None if q_weight is None else q_weight.data_ptr(),
+          None if k_weight is None else k_weight.data_ptr(), float(eps), _dtype_code(rows), _stream(),
+          kernels=2 if kept[2] is not None and tokens != ctx.num_reqs else 1)
 
 
 def ssm_row_width(heads: int, groups: int, dim: int, value_dim: int) -> int:
@@ -1894,12 +2055,15 @@ MOE_GEMV_SINGLE_PAIRS = int(os.environ.get("KVCORE_B200_MOE_GEMV_SINGLE_PAIRS", 
 class ExpertRows:
     """What ``moe_experts`` leaves for ``moe_combine``: the experts' outputs ``rows [R, N]``, where the row of
     pair ``t * top + s`` is that index itself (``row_of_pair`` None) or ``row_of_pair[t * top + s]``, and
-    weights still to be applied (``pending_weights`` [T * top], or None).  ``top``: pairs of a token."""
+    weights still to be applied (``pending_weights`` [T * top], or None).  ``top``: pairs of a token.  ``identity``:
+    ``(ids [T, top], weights [T, top], x [T, N], E)`` where some pairs chose an expert without tensors (an id of ``E`` or
+    more): such a pair has no row; it adds its weight times the token's row of ``x``."""
 
-    __slots__ = ("rows", "row_of_pair", "pending_weights", "top")
+    __slots__ = ("rows", "row_of_pair", "pending_weights", "top", "identity")
 
-    def __init__(self, rows, row_of_pair=None, pending_weights=None, top=None):
+    def __init__(self, rows, row_of_pair=None, pending_weights=None, top=None, identity=None):
         self.rows, self.row_of_pair, self.pending_weights, self.top = rows, row_of_pair, pending_weights, top
+        self.identity = identity
 
 
 class ExpertGrouping:
@@ -1914,8 +2078,8 @@ class ExpertGrouping:
         return self._host.tolist()
 
 
-def moe_group(ids: torch.Tensor, experts: int, *, for_library: bool) -> ExpertGrouping:
-    """Group the pairs ``t * top + s`` of ``ids [T, top]`` by expert.  ``for_library``: also the row of every
+def moe_group(ids: torch.Tensor, experts: int, *, for_library: bool, identity: int = 0) -> ExpertGrouping:
+    """Group the pairs ``t * top + s`` of ``ids [T, top]`` by expert (the ``identity`` ids behind ``experts`` are left out).  ``for_library``: also the row of every
     pair and where each expert's run begins, the latter copied to pinned host memory behind an event, so that
     a caller who has other work to launch first (a layer whose mixer runs beside its feed-forward) finds the
     counts there when it comes back, without draining the stream."""
@@ -1933,7 +2097,8 @@ def moe_group(ids: torch.Tensor, experts: int, *, for_library: bool) -> ExpertGr
     g._host = g._ready = None
     _call("kvb_moe_align", g.sorted_pairs.data_ptr(), g.tile_expert.data_ptr(), g.meta.data_ptr(),
           None if g.row_of_pair is None else g.row_of_pair.data_ptr(),
-          None if g.expert_begin is None else g.expert_begin.data_ptr(), ids.data_ptr(), pairs, experts, g.capacity,
+          None if g.expert_begin is None else g.expert_begin.data_ptr(), ids.data_ptr(), pairs, experts,
+          experts + int(identity), g.capacity,
           _stream())
     if for_library:
         g._host = torch.empty(experts + 1, dtype=torch.int32, pin_memory=True)
@@ -1954,13 +2119,16 @@ def moe_path(x: torch.Tensor, pairs: int, ff: int) -> str:
 
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_up: torch.Tensor,
                 down: torch.Tensor, *, weight_on_input: bool, path: str | None = None,
-                grouping: ExpertGrouping | None = None, join: tuple | None = None) -> ExpertRows:
+                grouping: ExpertGrouping | None = None, join: tuple | None = None, activation: str | None = None,
+                identity: int = 0) -> ExpertRows:
     """The chosen experts of every token: for pair ``t * top + s`` with ``e = ids[t, s]``,
     ``down[e] @ (silu(gate[e] @ a) * (up[e] @ a))``.  ``weight_on_input``: ``a = weights[t, s] * x[t]``
     (rounded to the storage type).  Otherwise ``a = x[t]`` and the weight multiplies the output (the rows
     that enter the last product, or the sum in ``moe_combine``: that product is linear).
     ``gate_up [E, 2F, K]`` (gate rows first), ``down [E, N, F]``.  ``join = (alpha, limit, shift)``: the branches
-    join as in ``glu_clamped`` instead of ``silu(gate) * up``.
+    join as in ``glu_clamped`` instead of ``silu(gate) * up``.  ``activation="squared_relu"``: no gate, ``gate_up
+    [E, F, K]`` and ``down[e] @ max(up[e] @ a, 0)^2``.  ``identity``: that many ids behind ``E`` stand for experts whose
+    output is their input; no product sees their pairs (see ``ExpertRows``).
 
     Three ways, by ``path`` (default: by type and size).  "tiles": grouped products of this library, one
     accumulator per output in ascending k (all of float32: bit-equal under any batching).  "stream": bf16,
@@ -1975,7 +2143,10 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
     tokens, k = x.shape
     top = ids.shape[1]
     experts, two_ff, _ = gate_up.shape
-    ff = two_ff // 2
+    if activation not in (None, "squared_relu") or (activation and join is not None):
+        raise KernelError(f"moe_experts: an expert's activation is None or 'squared_relu', got {activation!r}")
+    ff = two_ff if activation else two_ff // 2
+    first = 2 if activation else 1               # what the first product does with its sums: square, or join two branches
     n = down.shape[1]
     if gate_up.shape[2] != k or down.shape != (experts, n, ff) or x.stride(1) != 1:
         raise KernelError("moe_experts: the experts' matrices do not match the input")
@@ -1985,7 +2156,15 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
         raise KernelError(f"moe_experts: the branches' limit must be positive, got {join[1]}")
     joined = (0.0, 0.0, 0.0) if join is None else tuple(float(v) for v in join)
 
+    own = None
+    if identity:
+        if n != k or not x.is_contiguous():
+            raise KernelError("moe_experts: an expert that hands its input on needs contiguous rows of the output's width")
+        own = (ids, weights, x, experts)
+
     def activate(both: torch.Tensor) -> torch.Tensor:
+        if activation:
+            return relu_squared(both)
         if join is None:
             return silu_mul(both, 0)
         return glu_clamped(both, alpha=joined[0], limit=joined[1], shift=joined[2])
@@ -1994,29 +2173,29 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
         path = moe_path(x, pairs, ff)
     if path == "stream" and pairs > MOE_GEMV_SINGLE_PAIRS:
         # some experts are shared: the pairs of an expert take one pass over its matrices together
-        g = grouping if grouping is not None else moe_group(ids, experts, for_library=False)
+        g = grouping if grouping is not None else moe_group(ids, experts, for_library=False, identity=identity)
         hidden = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
         _call("kvb_moe_stream_rows", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,
               weights.data_ptr() if weight_on_input else None, gate_up.data_ptr(), g.sorted_pairs.data_ptr(),
-              g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, ff, k, 1, *joined, _stream())
+              g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, ff, k, first, *joined, _stream())
         out = torch.empty((pairs, n), dtype=x.dtype, device=x.device)
         _call("kvb_moe_stream_rows", out.data_ptr(), hidden.data_ptr(), hidden.stride(0), 1,
               None if weight_on_input else weights.data_ptr(), down.data_ptr(), g.sorted_pairs.data_ptr(),
               g.tile_expert.data_ptr(), g.meta.data_ptr(), g.max_tiles, n, ff, 0, *joined, _stream())
-        return ExpertRows(out, top=top)
+        return ExpertRows(out, top=top, identity=own)
     if path == "stream":
         hidden = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
         _call("kvb_moe_gemv", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,
               weights.data_ptr() if weight_on_input else None, gate_up.data_ptr(), ids.data_ptr(), pairs, experts,
-              ff, k, 1, *joined, _stream())
+              experts + identity, ff, k, first, *joined, _stream())
         out = torch.empty((pairs, n), dtype=x.dtype, device=x.device)
         _call("kvb_moe_gemv", out.data_ptr(), hidden.data_ptr(), hidden.stride(0), 1,
               None if weight_on_input else weights.data_ptr(), down.data_ptr(), ids.data_ptr(), pairs, experts,
-              n, ff, 0, *joined, _stream())
-        return ExpertRows(out, top=top)
+              experts + identity, n, ff, 0, *joined, _stream())
+        return ExpertRows(out, top=top, identity=own)
     library = path == "library"
     if grouping is None or (library and grouping.expert_begin is None):
-        grouping = moe_group(ids, experts, for_library=library)
+        grouping = moe_group(ids, experts, for_library=library, identity=identity)
     tile = int(_lib.kvb_moe_tile_rows())
     sorted_pairs, tile_expert, meta = grouping.sorted_pairs, grouping.tile_expert, grouping.meta
     row_of_pair, expert_begin = grouping.row_of_pair, grouping.expert_begin
@@ -2049,16 +2228,16 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
                 if counts[e]:
                     torch.mm(hidden[e, : counts[e]], down[e].t(), out=out[e, : counts[e]])
             out = out.view(experts * stride, n)
-        return ExpertRows(out, row_of_pair, None if weight_on_input else weights.reshape(-1), top)
+        return ExpertRows(out, row_of_pair, None if weight_on_input else weights.reshape(-1), top, own)
     hidden = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
     _call("kvb_moe_gemm", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,
           weights.data_ptr() if weight_on_input else None, gate_up.data_ptr(), sorted_pairs.data_ptr(),
-          tile_expert.data_ptr(), meta.data_ptr(), max_tiles, ff, k, 1, *joined, code, _stream())
+          tile_expert.data_ptr(), meta.data_ptr(), max_tiles, ff, k, first, *joined, code, _stream())
     out = torch.empty((pairs, n), dtype=x.dtype, device=x.device)
     _call("kvb_moe_gemm", out.data_ptr(), hidden.data_ptr(), hidden.stride(0), 1,
           None if weight_on_input else weights.data_ptr(), down.data_ptr(), sorted_pairs.data_ptr(),
           tile_expert.data_ptr(), meta.data_ptr(), max_tiles, n, ff, 0, *joined, code, _stream())
-    return ExpertRows(out, top=top)
+    return ExpertRows(out, top=top, identity=own)
 
 
 def moe_combine(expert_out, tokens: int, top: int, shared: torch.Tensor | None = None,
@@ -2080,12 +2259,19 @@ def moe_combine(expert_out, tokens: int, top: int, shared: torch.Tensor | None =
         _check(gates, "gates", dtype=torch.float32)
         if shared is None or gates.shape[0] != tokens:
             raise KernelError("moe_combine: gates need the shared rows they multiply")
+    identity = (None, 0, None, None)
+    if expert_out.identity is not None:
+        ids, all_weights, own, first = expert_out.identity
+        _check(own, "input rows", dtype=rows.dtype)
+        if tuple(own.shape) != (tokens, width):
+            raise KernelError("moe_combine: the input rows of identity experts do not match")
+        identity = (ids.data_ptr(), int(first), all_weights.data_ptr(), own.data_ptr())
     out = torch.empty((tokens, width), dtype=rows.dtype, device=rows.device)
     _call("kvb_moe_combine", out.data_ptr(), rows.data_ptr(), tokens, top,
           None if expert_out.row_of_pair is None else expert_out.row_of_pair.data_ptr(),
           None if expert_out.pending_weights is None else expert_out.pending_weights.data_ptr(),
           None if shared is None else shared.data_ptr(), None if gates is None else gates.data_ptr(),
-          0 if gates is None else gates.stride(0), width, _dtype_code(rows), _stream())
+          0 if gates is None else gates.stride(0), width, *identity, _dtype_code(rows), _stream())
     return out
 
 

@@ -137,6 +137,17 @@ class Summed:
         self.sumsq = sumsq
 
 
+class PendingNorm:
+    """A sub-layer's output that still has to be normed and added to the stream: what stands where it would stand in
+    the ``(h, residual)`` pair, ``x <- x + rows * rsqrt(mean(rows^2) + eps) * weight`` (``rows``: a tensor, or the rows
+    its experts left), then ``x <- x + step`` (``step``: one row for all tokens, or None)."""
+
+    __slots__ = ("rows", "weight", "eps", "step")
+
+    def __init__(self, rows: Any, weight: torch.Tensor, eps: float, step: torch.Tensor | None = None) -> None:
+        self.rows, self.weight, self.eps, self.step = rows, weight, float(eps), step
+
+
 class Norm(Part):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
@@ -196,6 +207,9 @@ class Block(Part):
 
 
 class StreamStep(Part):
+    # whether the step reads (and does not keep) what the stream started as; the model keeps that apart only then
+    reads_origin = True
+
     def forward(self, h: Any, residual: torch.Tensor | None, origin: torch.Tensor, number: int,
                 ctx: Any) -> tuple[Any, torch.Tensor]:
         raise NotImplementedError
@@ -271,6 +285,7 @@ __all__ = [
     "POSITION_ENCODINGS",
     "Part",
     "PartRegistry",
+    "PendingNorm",
     "PositionEncoding",
     "STREAM_STEPS",
     "StateSpec",

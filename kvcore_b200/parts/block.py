@@ -1,5 +1,6 @@
 """Arrangements of one layer: pre-norm mixer and feed-forward in sequence on a deferred residual (of the
-activation type, or a 32-bit stream), side by side on a 32-bit stream, or in sequence on a 32-bit stream with a norm on both sides of each.
+activation type, or a 32-bit stream), side by side on a 32-bit stream, or in sequence on a 32-bit stream with a norm on
+both sides of each.
 
 As the reference's decoder layer (kvcore/model/models/llama3.py:124-142): the running
 ``residual`` and the last sub-layer output ``h`` stay separate and are summed inside the
@@ -11,7 +12,7 @@ import torch
 
 from .. import kernels as K
 from ..config.model_spec import LayerSpec
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, StateSpec, Summed, WeightSlot
+from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, PendingNorm, StateSpec, Summed, WeightSlot
 
 
 class PreNormResidualBlock(Block):
@@ -110,10 +111,45 @@ class PreNormStreamBlock(PreNormResidualBlock):
         h = self.mixer.forward(x, ctx, cache)
         if self.feed_forward is None:
             return h, residual
-        x, residual = self.feed_forward_norm.forward_residual(h, residual)
+        x, residual = self.feed_forward_norm.forward_residual(self._behind_mixer(h), residual)
         unsummed = getattr(self.feed_forward, "forward_rows", None)
         h = None if unsummed is None else unsummed(x, ctx)
         return (self.feed_forward.forward(x, ctx) if h is None else h), residual
+
+    def _behind_mixer(self, a):
+        """What of the mixer's output is left to the norm in front of the feed-forward."""
+        return a
+
+
+class SandwichStreamBlock(PreNormStreamBlock):
+    """``x <- x + norm_b(mixer(norm_a(x)))``, then ``x <- x + norm_d(ff(norm_c(x)))`` on one 32-bit stream (a layer may
+    have no feed-forward).  What stands between two sub-layers is one kernel: the norm behind the first, its sum into
+    the stream and the norm in front of the second.  It also weights and sums the rows of a mixture's experts, and adds
+    the row of a stream step that stands between two layers.
+
+    In the ``(h, residual)`` pair that runs through the blocks this block returns ``(PendingNorm, stream)``."""
+
+    def __init__(self, *, layer: LayerSpec, unused_tensors: tuple = (), dtype: torch.dtype, device: torch.device) -> None:
+        super().__init__(layer=layer, unused_tensors=unused_tensors, dtype=dtype, device=device)
+        self.mixer_out_norm = NORMS.build(layer.norms["mixer_out_norm"], dtype=dtype, device=device)
+        self.feed_forward_out_norm = None
+        if self.feed_forward is not None:
+            self.feed_forward_out_norm = NORMS.build(layer.norms["feed_forward_out_norm"], dtype=dtype, device=device)
+        for norm in (self.mixer_out_norm, self.feed_forward_out_norm):
+            if norm is not None and norm.as_rms_scale() is None:
+                raise ValueError("the norms behind the sub-layers are left to the kernel behind them: they must be RMS scales")
+
+    def parts(self):
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.mixer_out_norm, self.feed_forward_norm,
+                                 self.feed_forward, self.feed_forward_out_norm) if p is not None)
+
+    def forward(self, h, residual, ctx, cache):
+        h, residual = super().forward(h, residual, ctx, cache)
+        out_norm = self.mixer_out_norm if self.feed_forward is None else self.feed_forward_out_norm
+        return PendingNorm(h, *out_norm.as_rms_scale()), residual
+
+    def _behind_mixer(self, a):
+        return PendingNorm(a, *self.mixer_out_norm.as_rms_scale())
 
 
 class ParallelResidualBlock(Block):
@@ -325,6 +361,8 @@ class SandwichResidualBlock(Block):
 BLOCKS.register("prenorm_residual", PreNormResidualBlock)
 BLOCKS.register("prenorm_stream", PreNormStreamBlock)
 BLOCKS.register("sandwich_residual", SandwichResidualBlock)
+BLOCKS.register("sandwich_stream", SandwichStreamBlock)
 BLOCKS.register("parallel_residual", ParallelResidualBlock)
 
-__all__ = ["ParallelResidualBlock", "PreNormResidualBlock", "PreNormStreamBlock", "SandwichResidualBlock"]
+__all__ = ["ParallelResidualBlock", "PreNormResidualBlock", "PreNormStreamBlock", "SandwichResidualBlock",
+           "SandwichStreamBlock"]

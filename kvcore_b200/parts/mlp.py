@@ -1,4 +1,4 @@
-"""Gated feed-forward: ``down(silu(gate(x)) * up(x))`` with gate and up in one matrix.
+"""Gated feed-forward: ``down(silu(gate(x)) * up(x))`` with gate and up in one matrix; bounded and ungated forms.
 
 The arithmetic is the reference's (kvcore/model/models/llama3.py:25-45;
 kvcore/model/layer/activation.py:8-17).  The packing differs: when the intermediate size is a
@@ -123,7 +123,29 @@ class ClampedGLU(FeedForward):
         return K.linear(hidden, self.down_weight)
 
 
+class SquaredReLU(FeedForward):
+    """``down(max(up(x), 0)^2)``: two products with the squared positive part between them; no gate, no biases."""
+
+    graph_safe = True
+
+    def __init__(self, *, hidden_size: int, intermediate_size: int, name: str, tensor_names: dict | None = None,
+                 dtype: torch.dtype, device: torch.device) -> None:
+        self.hidden_size, self.intermediate_size, self.name = int(hidden_size), int(intermediate_size), name
+        self.tensor_names = dict(GATED_TENSOR_NAMES)
+        self.tensor_names.update(tensor_names or {})
+        self.up_weight = torch.empty(self.intermediate_size, self.hidden_size, dtype=dtype, device=device)
+        self.down_weight = torch.empty(self.hidden_size, self.intermediate_size, dtype=dtype, device=device)
+
+    def weight_slots(self) -> list[WeightSlot]:
+        return [WeightSlot(f"{self.name}.{self.tensor_names['up']}", self.up_weight),
+                WeightSlot(f"{self.name}.{self.tensor_names['down']}", self.down_weight)]
+
+    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+        return K.linear(K.linear_relu_squared(x, self.up_weight), self.down_weight)
+
+
 FEED_FORWARDS.register("swiglu", SwiGLU)
+FEED_FORWARDS.register("squared_relu", SquaredReLU)
 FEED_FORWARDS.register("clamped_glu", ClampedGLU)
 
-__all__ = ["ClampedGLU", "GATED_TENSOR_NAMES", "SwiGLU"]
+__all__ = ["ClampedGLU", "GATED_TENSOR_NAMES", "SquaredReLU", "SwiGLU"]

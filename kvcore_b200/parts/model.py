@@ -13,10 +13,11 @@ import torch
 
 from .. import kernels as K
 from ..config.model_spec import ModelSpec
-from . import (attention, attention_maps, block, embedding, mlp, moe, norm, recurrent, rope,  # noqa: F401
+from . import (attention, attention_maps, block, embedding, grouped_attention, mlp, moe, norm, recurrent, rope,  # noqa: F401
                side_by_side, stream_steps)                                                   # (register the stock parts)
-from .base import (BLOCKS, EMBEDDINGS, LM_HEADS, NORMS, STREAM_STEPS, CacheSpec, StateSpec, Summed,
+from .base import (BLOCKS, EMBEDDINGS, LM_HEADS, NORMS, STREAM_STEPS, CacheSpec, PendingNorm, StateSpec, Summed,
                    WeightSlot)
+from .norm import add_pending
 
 
 @dataclass(frozen=True)
@@ -118,11 +119,12 @@ class DecoderModel:
         embed_step = getattr(self.embedding, "forward_step", None)
         h = self.embedding.forward(ctx.token_ids) if embed_step is None else embed_step(ctx)
         residual = origin = None
-        if self.stream_steps:
+        if any(step.reads_origin for step in self.stream_steps.values()):
             # what the stream started as: the blocks add to the stream in place, so it is kept apart from it
             # (unless a step replaces the stream ahead of the first block)
             origin = h if h.dtype == torch.float32 else K.stream_add(h)
-            if self.schedule[0].ahead is None:
+            first = self.schedule[0].ahead
+            if first is None or not self.stream_steps[first[0]].reads_origin:
                 h = origin.clone()
         # per-token inputs of the layers themselves: gathered once, every block reads its own columns
         side_rows = getattr(self.embedding, "side_rows", None)
@@ -134,9 +136,10 @@ class DecoderModel:
                 name, number = entry.ahead
                 h, residual = self.stream_steps[name].forward(h, residual, origin, number, ctx)
             if residual is not None and not isinstance(h, Summed) and not getattr(block, "takes_rows", False):
-                # rows that only the norm behind them knows how to add: experts' rows, one row for all tokens
-                if isinstance(h, K.ExpertRows) or h.shape != residual.shape:
-                    residual, h = K.stream_add_rows(residual, h)[0], Summed(None)
+                # rows that only the norm behind them knows how to add: experts' rows, one row for all tokens, an
+                # output with a norm of its own ahead of the sum
+                if isinstance(h, (K.ExpertRows, PendingNorm)) or h.shape != residual.shape:
+                    residual, h = add_pending(residual, h)[0], Summed(None)
             h, residual = block.forward(h, residual, ctx, caches[index])
         return h, residual
 
@@ -145,8 +148,8 @@ class DecoderModel:
         forward_rows = getattr(self.final_norm, "forward_rows", None)
         if forward_rows is not None and residual.dtype == torch.float32 and not isinstance(h, Summed):
             return self.lm_head.forward(forward_rows(h, residual, rows))
-        if isinstance(h, K.ExpertRows):
-            residual, h = K.stream_add_rows(residual, h)[0], Summed(None)
+        if isinstance(h, (K.ExpertRows, PendingNorm)):
+            residual, h = add_pending(residual, h)[0], Summed(None)
         residual_rows = K.gather_rows(residual, rows)
         if isinstance(h, Summed):      # the last sub-layer has added its output into the residual itself
             normed = self.final_norm.forward(residual_rows)

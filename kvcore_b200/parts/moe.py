@@ -14,7 +14,12 @@ feed-forwards per token; an optional shared expert runs for every token.
     y += sigmoid(g . x) * shared(x)   (``shared`` given; ``shared_gate`` False: plain sum)
 
     expert(a) = down(silu(gate a) * (up a)), no biases; or with ``join = (alpha, limit, shift)``
-                down(g * sigmoid(alpha g) * (u + shift)), g = min(gate a, limit), u = clamp(up a, -limit, limit)
+                down(g * sigmoid(alpha g) * (u + shift)), g = min(gate a, limit), u = clamp(up a, -limit, limit);
+                or with ``activation="squared_relu"``  down(max(up a, 0)^2)  (no gate)
+
+``identity_experts``: that many experts without tensors stand behind the others in the router (whose rows, bias and
+correction then count both kinds); their output is their input ``a`` itself.  They take no part in the products: the
+kernel that sums a token's experts adds the token's own row for them.
 
 The experts' matrices are stacked ``[E, 2F, K]`` (gate rows, then up rows) and ``[E, K, F]``; the
 (token, expert) pairs are grouped by expert on the device and the two products run as grouped
@@ -42,32 +47,41 @@ class RoutedExperts(FeedForward):
                  score: str = "sigmoid", renormalize: bool = False, weight_on: str = "input",
                  shared: PartSpec | None = None, shared_gate: bool = False, weight_scale: float = 1.0,
                  choice_correction: bool = False, group_count: int = 1, group_keep: int = 1,
-                 router_bias: bool = False, join: tuple | None = None,
+                 router_bias: bool = False, join: tuple | None = None, activation: str | None = None,
+                 identity_experts: int = 0,
                  tensor_names: dict | None = None, dtype: torch.dtype, device: torch.device) -> None:
         self.hidden_size, self.num_experts = int(hidden_size), int(num_experts)
         self.top_k, self.expert_size = int(top_k), int(expert_size)
-        if not 0 < self.top_k <= self.num_experts:
-            raise ValueError(f"top_k {top_k} must lie in [1, num_experts {num_experts}]")
+        self.identity_experts = int(identity_experts)
+        if self.num_experts <= 0 or self.identity_experts < 0:
+            raise ValueError(f"a mixture has experts, got {num_experts} and {identity_experts} identity experts")
+        self.routed = self.num_experts + self.identity_experts         # what the router chooses among
+        if not 0 < self.top_k <= self.routed:
+            raise ValueError(f"top_k {top_k} must lie in [1, {self.routed}] (num_experts + identity_experts)")
         if score not in ("sigmoid", "softmax", "softmax_chosen"):
             raise ValueError(f"unknown router score {score!r}")
         if weight_on not in ("input", "output"):
             raise ValueError(f"weight_on must be 'input' or 'output', got {weight_on!r}")
         self.score, self.renormalize, self.weight_on = score, bool(renormalize), weight_on
         self.weight_scale, self.group_count, self.group_keep = float(weight_scale), int(group_count), int(group_keep)
-        if (self.group_count <= 0 or self.num_experts % self.group_count or not 0 < self.group_keep <= self.group_count
-                or self.group_keep * (self.num_experts // self.group_count) < self.top_k):
-            raise ValueError(f"{group_keep} of {group_count} equal groups of {num_experts} experts must hold top_k {top_k}")
+        if (self.group_count <= 0 or self.routed % self.group_count or not 0 < self.group_keep <= self.group_count
+                or self.group_keep * (self.routed // self.group_count) < self.top_k):
+            raise ValueError(f"{group_keep} of {group_count} equal groups of {self.routed} experts must hold top_k {top_k}")
         if join is not None and (len(join) != 3 or not join[1] > 0):
             raise ValueError(f"join is (alpha, limit, shift) with a positive limit, got {join!r}")
         self.join = None if join is None else tuple(float(v) for v in join)
+        if activation not in (None, "squared_relu") or (activation and join is not None):
+            raise ValueError(f"an expert's activation is None (gated units) or 'squared_relu' (no gate), got {activation!r}")
+        self.activation = activation
         self.name = name
         self.tensor_names = dict(self.DEFAULT_TENSOR_NAMES)
         self.tensor_names.update(tensor_names or {})
         experts, ff, hidden = self.num_experts, self.expert_size, self.hidden_size
-        self.router_weight = torch.empty(experts, hidden, dtype=torch.float32, device=device)
-        self.correction = torch.empty(experts, dtype=torch.float32, device=device) if choice_correction else None
-        self.router_bias = torch.empty(experts, dtype=torch.float32, device=device) if router_bias else None
-        self.gate_up_weight = torch.empty(experts, 2 * ff, hidden, dtype=dtype, device=device)
+        self.router_weight = torch.empty(self.routed, hidden, dtype=torch.float32, device=device)
+        self.correction = torch.empty(self.routed, dtype=torch.float32, device=device) if choice_correction else None
+        self.router_bias = torch.empty(self.routed, dtype=torch.float32, device=device) if router_bias else None
+        # gate rows, then up rows; without a gate the up rows alone
+        self.gate_up_weight = torch.empty(experts, (1 if self.activation else 2) * ff, hidden, dtype=dtype, device=device)
         self.down_weight = torch.empty(experts, hidden, ff, dtype=dtype, device=device)
         self.shared = None if shared is None else FEED_FORWARDS.build(shared, dtype=dtype, device=device)
         if shared_gate and self.shared is None:
@@ -90,9 +104,10 @@ class RoutedExperts(FeedForward):
         if self.correction is not None:
             slots.append(WeightSlot(self._tensor("correction"), self.correction, init="zeros"))
         for e in range(self.num_experts):
+            if self.activation is None:
+                slots.append(WeightSlot(self._tensor("gate", e), self.gate_up_weight[e, :ff]))
             slots += [
-                WeightSlot(self._tensor("gate", e), self.gate_up_weight[e, :ff]),
-                WeightSlot(self._tensor("up", e), self.gate_up_weight[e, ff:]),
+                WeightSlot(self._tensor("up", e), self.gate_up_weight[e, -ff:]),
                 WeightSlot(self._tensor("down", e), self.down_weight[e]),
             ]
         if self.shared is not None:
@@ -118,13 +133,14 @@ class RoutedExperts(FeedForward):
                              weight_scale=self.weight_scale, bias=self.router_bias)
         grouping = None
         if K.moe_path(x, x.shape[0] * self.top_k, self.expert_size) == "library":
-            grouping = K.moe_group(routed[0], self.num_experts, for_library=True)
+            grouping = K.moe_group(routed[0], self.num_experts, for_library=True, identity=self.identity_experts)
         return routed, grouping
 
     def _expert_rows(self, x: torch.Tensor, ctx, prepared):
         (ids, weights, gates), grouping = prepared if prepared is not None else self.prepare(x, ctx)
         return gates, K.moe_experts(x, ids, weights, self.gate_up_weight, self.down_weight,
-                                    weight_on_input=self.weight_on == "input", grouping=grouping, join=self.join)
+                                    weight_on_input=self.weight_on == "input", grouping=grouping, join=self.join,
+                                    activation=self.activation, identity=self.identity_experts)
 
     def forward_rows(self, x: torch.Tensor, ctx):
         """The chosen experts' rows, for a block whose next norm weights and sums them into the stream (None: a

@@ -9,7 +9,15 @@ from __future__ import annotations
 import torch
 
 from .. import kernels as K
-from .base import NORMS, Norm, WeightSlot
+from .base import NORMS, Norm, PendingNorm, WeightSlot
+
+
+def add_pending(residual: torch.Tensor, h, **kwargs) -> tuple:
+    """``K.stream_add_rows`` of a 32-bit stream and whatever a block has left to add: a sub-layer's output, one row for
+    all tokens, the rows of its experts, or any of these with a norm of its own ahead of the sum (``PendingNorm``)."""
+    if isinstance(h, PendingNorm):
+        return K.stream_add_rows(residual, h.rows, after=(h.weight, h.eps), step=h.step, **kwargs)
+    return K.stream_add_rows(residual, h, **kwargs)
 
 
 class RMSNorm(Norm):
@@ -108,17 +116,18 @@ class RMSNormStream(Norm):
         return K.rms_norm_shift(x, self.weight, self.eps, self.dtype)
 
     def forward_residual(self, h, residual: torch.Tensor):
-        """``h``: a sub-layer's output, or the rows its experts left (``ExpertRows``, a 32-bit stream only)."""
+        """``h``: a sub-layer's output, the rows its experts left (``ExpertRows``), or either with a norm ahead of the
+        sum (``PendingNorm``); the latter two on a 32-bit stream only."""
         if residual.dtype != torch.float32:
             residual = residual.add_(h)
             return self.forward(residual), residual
-        residual, y, _ = K.stream_add_rows(residual, h, weight=self.weight, eps=self.eps, out_dtype=self.dtype)
+        residual, y, _ = add_pending(residual, h, weight=self.weight, eps=self.eps, out_dtype=self.dtype)
         return y, residual
 
     def forward_rows(self, h, residual: torch.Tensor, token_rows: torch.Tensor) -> torch.Tensor:
         """``norm(residual + h)`` of some tokens of a 32-bit stream, which stays as it is."""
-        return K.stream_add_rows(residual, h, weight=self.weight, eps=self.eps, out_dtype=self.dtype,
-                                 token_rows=token_rows)[1]
+        return add_pending(residual, h, weight=self.weight, eps=self.eps, out_dtype=self.dtype,
+                           token_rows=token_rows)[1]
 
     def as_rms_scale(self):
         return self.weight, self.eps
@@ -128,4 +137,4 @@ NORMS.register("rmsnorm", RMSNorm)
 NORMS.register("rmsnorm_stream", RMSNormStream)
 NORMS.register("layernorm", LayerNorm)
 
-__all__ = ["LayerNorm", "RMSNorm", "RMSNormStream"]
+__all__ = ["LayerNorm", "RMSNorm", "RMSNormStream", "add_pending"]

@@ -27,6 +27,10 @@ shares B and C) ``S <- exp(-exp(A_log) dt) S + dt B x^T``, ``y = S^T C + D x``; 
 ``norm_groups`` equal parts of all heads' values.  The state of a request is ``S`` and the last ``taps - 1`` inputs of
 the convolution.
 
+``Retention``: ``LightningAttention``'s recurrence on plain projections: q and k turn by the token's position (an
+encoding that offers its cos/sin table), k is multiplied by ``dim^(-1/2)``; each head's read-out is divided by its root
+mean square (no weight) and multiplied by ``silu(W_g x)``.
+
 Decays, step sizes, unit norms, the state, the read-out and the norm behind it are 32-bit whatever the
 activation type.
 """
@@ -35,7 +39,8 @@ from __future__ import annotations
 import torch
 
 from .. import kernels as K
-from .base import MIXERS, Mixer, StateSpec, WeightSlot
+from ..config.model_spec import PartSpec
+from .base import MIXERS, POSITION_ENCODINGS, Mixer, StateSpec, WeightSlot
 
 
 def _round8(n: int) -> int:
@@ -255,6 +260,67 @@ class LightningAttention(ProjectedMixer):
                          out, scale, gate_act="sigmoid")
 
 
+class Retention(ProjectedMixer):
+    DEFAULT_TENSOR_NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o"}
+
+    def __init__(self, *, hidden_size: int, num_heads: int, head_dim: int, value_dim: int, decay: tuple, eps: float,
+                 name: str, position: PartSpec | None = None, k_scale: float | None = None,
+                 tensor_names: dict | None = None, dtype: torch.dtype, device: torch.device) -> None:
+        if min(num_heads, head_dim, value_dim) <= 0 or len(decay) != num_heads:
+            raise ValueError("retention needs positive heads and sizes and one decay a head")
+        if head_dim > 512:
+            raise ValueError(f"head_dim {head_dim} exceeds the state kernel's 512 key channels")
+        self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
+        self.head_dim, self.value_dim = int(head_dim), int(value_dim)
+        self.eps, self.name = float(eps), name
+        self.k_scale = self.head_dim ** -0.5 if k_scale is None else float(k_scale)
+        self.tensor_names = dict(self.DEFAULT_TENSOR_NAMES)
+        self.tensor_names.update(tensor_names or {})
+        self.qk_cols, self.v_cols = self.num_heads * self.head_dim, self.num_heads * self.value_dim
+        # one packed projection: q, k, v, the gate
+        self.in_rows = _round8(2 * self.qk_cols + 2 * self.v_cols)
+        self.out_cols = self.v_cols
+        self._allocate(dtype, device)
+        self.position = None if position is None else POSITION_ENCODINGS.build(position, dtype=dtype, device=device)
+        if self.position is not None and getattr(self.position, "rotary_dim", 0) > self.head_dim:
+            raise ValueError(f"{self.name}: the encoding turns more than a head's {self.head_dim} entries")
+        table = torch.tensor([float(a) for a in decay], dtype=torch.float32)
+        self.decay = table if torch.device(device).type == "meta" else table.to(device)
+
+    @property
+    def graph_safe(self) -> bool:
+        return self.position is None or self.position.graph_safe
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec((_round4(self.num_heads * self.head_dim * self.value_dim),), torch.float32)
+
+    def _tensor(self, key: str) -> str:
+        return f"{self.name}.{self.tensor_names[key]}"
+
+    def weight_slots(self) -> list[WeightSlot]:
+        qk, v, w = self.qk_cols, self.v_cols, self.in_weight
+        return [
+            WeightSlot(self._tensor("q"), w[:qk]), WeightSlot(self._tensor("k"), w[qk:2 * qk]),
+            WeightSlot(self._tensor("v"), w[2 * qk:2 * qk + v]), WeightSlot(self._tensor("g"), w[2 * qk + v:2 * qk + 2 * v]),
+            WeightSlot(self._tensor("o"), self.o_weight),
+        ]
+
+    def ignorable_tensor_names(self) -> list[str]:
+        return [] if self.position is None else self.position.ignorable_tensor_names()
+
+    def mix_rows(self, rows, ctx, cache, out, scale: float = 1.0) -> None:
+        qk, v = self.qk_cols, self.v_cols
+        cos_sin = None
+        if self.position is not None:
+            cos_sin = self.position.cos_sin(ctx)
+            if cos_sin is None:
+                raise NotImplementedError(f"{self.name}: the position encoding must offer its cos/sin table")
+        o = K.retention_scan(rows[:, :qk], rows[:, qk:2 * qk], rows[:, 2 * qk:2 * qk + v], cos_sin, self.decay,
+                             cache.state, ctx, heads=self.num_heads, dim=self.head_dim, value_dim=self.value_dim,
+                             k_scale=self.k_scale, state_offset=self.state_offset)
+        K.gated_rms_norm(o, rows[:, 2 * qk + v:2 * qk + 2 * v], None, self.eps, out, scale)
+
+
 class SelectiveStateSpace(ProjectedMixer):
     graph_safe = True
 
@@ -322,5 +388,7 @@ MIXERS.register("selective_state_space", SelectiveStateSpace)
 MIXERS.register("gated_linear_attention", GatedLinearAttention)
 MIXERS.register("lightning_attention", LightningAttention)
 MIXERS.register("gated_delta_rule", GatedDeltaRule)
+MIXERS.register("retention", Retention)
 
-__all__ = ["GatedDeltaRule", "GatedLinearAttention", "LightningAttention", "ProjectedMixer", "SelectiveStateSpace"]
+__all__ = ["GatedDeltaRule", "GatedLinearAttention", "LightningAttention", "ProjectedMixer", "Retention",
+           "SelectiveStateSpace"]

@@ -84,7 +84,7 @@ class RotaryEncoding(PositionEncoding):
             raise ValueError("a rotary encoding that turns nothing: leave the position encoding out instead")
         # layers with the same frequency parameters share one cos/sin table per step
         self.table_key = ("rope", int(head_dim), float(theta), str(rope_type), float(factor),
-                          float(low_freq_factor), float(high_freq_factor), int(original_max_position_embeddings))
+                          float(low_freq_factor), float(high_freq_factor), float(original_max_position_embeddings))
         table = rope_inverse_frequencies(
             head_dim, theta, rope_type, factor, low_freq_factor, high_freq_factor,
             original_max_position_embeddings,

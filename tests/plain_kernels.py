@@ -207,21 +207,31 @@ def stream_add_norm(x, a, weight, eps, *, out=None, stack=None, depth=0, coeffs=
     return out, avg
 
 
-def stream_add_rows(x, a, *, weight=None, eps=0.0, out_dtype=None, token_rows=None, origin=None, keep=True):
+def stream_add_rows(x, a, *, weight=None, eps=0.0, out_dtype=None, token_rows=None, origin=None, keep=True, after=None,
+                    step=None):
     tokens, width = x.shape
     total = x
     if a is not None:
         if hasattr(a, "rows"):                      # the rows of the chosen experts, as the product hands them on
             pairs = a.rows.float()
             if a.row_of_pair is not None:
-                pairs = pairs[a.row_of_pair.long()]
+                pairs = pairs[a.row_of_pair.long().clamp(min=0)]
             if a.pending_weights is not None:
                 pairs = pairs * a.pending_weights.reshape(-1, 1)
+            if a.identity is not None:              # pairs without a row: their weight times the token's own row
+                ids, weights, own, first = a.identity
+                given = weights.reshape(-1, 1) * own.float().repeat_interleave(ids.shape[1], 0)
+                pairs = torch.where(ids.reshape(-1, 1) >= first, given, pairs)
         else:
             pairs = a.float()
             if a.shape[0] == 1:                     # one row for all tokens
                 pairs = pairs.expand(tokens, width)
-        total = x + pairs.reshape(tokens, -1, width).sum(1)
+        added = pairs.reshape(tokens, -1, width).sum(1)
+        if after is not None:                       # the sum gets a norm of its own first
+            added = _rms(added, after[1]) * after[0].float()
+            if step is not None:
+                added = added + step.float().reshape(1, width)
+        total = x + added
     dtype = out_dtype or (a.rows if hasattr(a, "rows") else a).dtype
     keep = keep and token_rows is None and a is not None
     if keep:
@@ -269,7 +279,7 @@ def _strided(tensor, page, slot, head, strides, width):
 
 def attention_dims(q, keys, values, table, ctx, *, value_heads, group, maps, key_width, value_width, page_size,
                    num_pages, key_strides, value_strides, scale, sink=None, window=None, out=None, out_dtype=None,
-                   force_general=False, num_splits=None, slopes=None):
+                   force_general=False, num_splits=None, slopes=None, softcap=None):
     tokens, hq, _ = q.shape
     if out is None:
         out = torch.empty((tokens, hq, value_width), dtype=out_dtype or q.dtype, device=q.device)
@@ -292,6 +302,8 @@ def attention_dims(q, keys, values, table, ctx, *, value_heads, group, maps, key
             k = flat_k[k_begin[:, None] + torch.arange(key_width)[None]].float()
             v = flat_v[v_begin[:, None] + torch.arange(value_width)[None]].float()
             scores = (k @ q[t, h].float()) * scale
+            if softcap is not None:
+                scores = softcap * torch.tanh(scores / softcap)
             if slopes is not None:
                 scores = scores - slopes[h] * (pos - positions).float()
             top = scores.max() if sink is None else torch.maximum(scores.max(), sink[h])
@@ -375,9 +387,18 @@ def maps_combine(a, lam, eps, out_scale, out_dtype):
     return (_rms(o, eps) * out_scale).to(out_dtype).reshape(tokens, heads * width)
 
 
-def sigmoid_gate_mul(o, gate):
+def sigmoid_gate_mul(o, gate, out=None):
     tokens, heads, width = o.shape
-    return (o.float().reshape(tokens, heads * width) * torch.sigmoid(gate.float())).to(o.dtype)
+    y = (o.float().reshape(tokens, heads * width) * torch.sigmoid(gate.float())).to(o.dtype)
+    return y if out is None else out.copy_(y)
+
+
+def relu_squared(x):
+    return x.copy_((x.float().clamp(min=0.0) ** 2).to(x.dtype))
+
+
+def linear_relu_squared(x, weight):
+    return ((x.float() @ weight.float().T).clamp(min=0.0) ** 2).to(x.dtype)
 
 
 def heads_linear(x, weight, out=None):
@@ -473,14 +494,26 @@ def moe_path(x, pairs, ff):
     return "tiles"
 
 
-def moe_experts(x, ids, weights, gate_up, down, *, weight_on_input, path=None, grouping=None, join=None):
+def moe_experts(x, ids, weights, gate_up, down, *, weight_on_input, path=None, grouping=None, join=None, activation=None,
+                identity=0):
     tokens, top = ids.shape
-    ff = gate_up.shape[1] // 2
+    experts = gate_up.shape[0]
+    ff = gate_up.shape[1] // (1 if activation else 2)
     out = torch.empty(tokens * top, down.shape[1], dtype=x.dtype, device=x.device)
     for t in range(tokens):
         for s in range(top):
             e, w = int(ids[t, s]), weights[t, s]
+            assert 0 <= e < experts + identity
+            if e >= experts:                        # hands its input on (as the weighted row that a sum takes)
+                out[t * top + s] = (w * x[t].float()).to(x.dtype)
+                continue
             a = (w * x[t].float()).to(x.dtype).float() if weight_on_input else x[t].float()
+            if activation:
+                hidden = ((gate_up[e].float() @ a).clamp(min=0.0) ** 2).to(x.dtype).float()
+                if not weight_on_input:
+                    hidden = (w * hidden).to(x.dtype).float()
+                out[t * top + s] = (down[e].float() @ hidden).to(x.dtype)
+                continue
             g = (gate_up[e, :ff].float() @ a).to(x.dtype).float()
             u = (gate_up[e, ff:].float() @ a).to(x.dtype).float()
             if join is None:
@@ -664,11 +697,71 @@ def lightning_scan(q, k, v, decay, state, ctx, *, heads, dim, value_dim, q_scale
     return out
 
 
+def _turn_halves(x, cos_sin):
+    """x [T, heads, D] float: entries i and i + rot / 2 of the first rot = 2 * cos_sin.shape[1] turn together."""
+    if cos_sin is None:
+        return x
+    half = cos_sin.shape[1]
+    c, s = cos_sin[:, None, :, 0], cos_sin[:, None, :, 1]
+    u, v = x[..., :half], x[..., half:2 * half]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1)
+
+
+def retention_scan(q, k, v, cos_sin, decay, state, ctx, *, heads, dim, value_dim, k_scale, state_offset=0):
+    tokens, n = q.shape[0], heads * dim * value_dim
+    out = torch.empty((tokens, heads, value_dim), dtype=torch.float32, device=q.device)
+    qf = _turn_halves(q.float().reshape(tokens, heads, dim), cos_sin)
+    kf = _turn_halves(k.float().reshape(tokens, heads, dim), cos_sin) * k_scale
+    vf = v.float().reshape(tokens, heads, value_dim)
+    for _, begin, end, slot in _request_ranges(ctx):
+        S = state[slot, state_offset:state_offset + n].reshape(heads, value_dim, dim).transpose(1, 2).clone()   # kept column by column
+        for t in range(begin, end):
+            S = S * decay.float()[:, None, None] + kf[t][:, :, None] * vf[t][:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S, qf[t])
+        state[slot, state_offset:state_offset + n] = S.transpose(1, 2).reshape(n)
+    return out
+
+
+def attention_prepare(rows, q_out, cos_sin, ctx, table, cache, *, q_heads, k_heads, dim, value_width, taps=None, state=None,
+                      state_offset=0, q_weight=None, k_weight=None, eps=0.0, write=True):
+    tokens, page_size = rows.shape[0], cache.shape[2]
+    q_len, k_len = q_heads * dim, k_heads * dim
+    channels = q_len + k_len + value_width
+    x = rows[:, :channels].float()
+    if taps is not None:
+        keep = taps.shape[0] - 1
+        convolved = torch.empty_like(x)
+        if keep:
+            for _, begin, end, slot in _request_ranges(ctx):
+                held = state[slot, state_offset:state_offset + channels * keep].reshape(keep, channels)
+                history = torch.cat([held.clone(), x[begin:end]])
+                convolved[begin:end] = sum(history[j:j + end - begin] * taps[j].float() for j in range(keep + 1))
+                state[slot, state_offset:state_offset + channels * keep] = history[-keep:].reshape(-1)
+        else:
+            convolved = x * taps[0].float()
+        x = convolved
+    q, k, v = x[:, :q_len], x[:, q_len:q_len + k_len], x[:, q_len + k_len:]
+    if q_weight is not None:
+        q, k = _rms(q, eps) * q_weight.float(), _rms(k, eps) * k_weight.float()
+    q = _turn_halves(q.reshape(tokens, q_heads, dim), cos_sin).reshape(tokens, q_len).to(rows.dtype)
+    k = _turn_halves(k.reshape(tokens, k_heads, dim), cos_sin).reshape(tokens, k_len).to(rows.dtype)
+    v = v.to(rows.dtype)
+    q_out.copy_(q)
+    if not write:
+        return
+    for t in range(tokens):
+        pos = int(ctx.positions[t])
+        page = int(table[int(ctx.req_index[t]), pos // page_size])
+        assert page > 0, "write through the null page"
+        cache[page, 0, pos % page_size, :k_len] = k[t]
+        cache[page, 0, pos % page_size, k_len:] = v[t]
+
+
 def gated_rms_norm(o, gate, weight, eps, out, scale=1.0, *, gate_act="silu"):
     tokens, heads, width = o.shape
     g = gate.float().reshape(tokens, heads, width)
     factor = g * torch.sigmoid(g) if gate_act == "silu" else torch.sigmoid(g)
-    y = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight.float() * factor * scale
+    y = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * (1.0 if weight is None else weight.float()) * factor * scale
     out.copy_(y.reshape(tokens, heads * width).to(out.dtype))
     return out
 
@@ -780,6 +873,7 @@ _NAMES = [
     "sigmoid_gate_mul", "heads_linear", "gather_cached_rows",
     "embed_scaled", "turn_norm_kv_write", "head_gate", "gla_scan", "conv_prepare", "delta_scan", "gated_rms_norm",
     "latent_cache_write", "stream_add_rows", "embed_pairs", "softcap", "ssm_prepare", "ssm_scan", "gated_group_norm",
+    "retention_scan", "attention_prepare", "relu_squared", "linear_relu_squared",
     "lightning_scan", "gelu_mul", "layer_norm", "stream_add", "qk_prepare", "glu_clamped", "moe_route", "moe_experts", "moe_combine", "moe_path",
 ]
 
