@@ -669,12 +669,13 @@ def dutivik_config(size: dict, kinds: str) -> dict:
             "embedding": {"scale": 24.0}, "layers": layers}
 
 
-def rubuvik_config(size: dict, kinds: str) -> dict:
+def rubuvik_config(size: dict, kinds: str, window: int | None = 1024) -> dict:
     """A Rubuvik config.json of ``DESIGN_LAYERS`` layers.  ``kinds``: a letter per layer, "l" lightning attention
     (half of Llama's heads, values twice as wide as the keys) with a dense feed-forward, "a" the plain window
     attention (Llama's heads, a window of 1,024, a query temperature, value mixing) with a dense feed-forward,
     "m" the same with a mixture of experts (four groups of which two are kept), "b" the attention with biases,
-    unit q and k, a sink and a gate a head.  Every layer adds a token side input of 256 entries."""
+    unit q and k, a sink and a gate a head.  Every layer adds a token side input of 256 entries.  ``window`` None: the
+    attentions see every earlier token."""
     half, dim = size["heads"] // 2, size["dim"]
     dense = {"kind": "dense", "ff": size["ff"]}
     moe = {"kind": "moe", "expert": {"ff": size["expert_ff"]}, "shared": {"ff": size["shared_ff"]},
@@ -687,7 +688,9 @@ def rubuvik_config(size: dict, kinds: str) -> dict:
                            "mixer": {"heads": half, "dim": dim, "vdim": 2 * dim, "decay": decay}})
             continue
         mixer = {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": dim, "vdim": dim, "scale": dim ** -0.5,
-                 "mask": {"size": 1024}, "v_mix": True}
+                 "v_mix": True}
+        if window is not None:
+            mixer["mask"] = {"size": window}
         if kind != "b":
             mixer["q_temp"] = {"coef": 0.1, "every": 1024}
         layers.append({"type": "attention_2" if kind == "b" else "attention", "mixer": mixer,
@@ -714,6 +717,38 @@ def mamevik_config(size: dict, kinds: str, loop: tuple[int, int, int]) -> dict:
     return {"architecture": "Mamevik", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5},
             "embedding": {"bigram": {"buckets": size["vocab"] - 1, "mul_prev": 7, "mul_cur": 13}}, "layers": layers,
             "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]}, "logit_scale": 0.5, "logit_softcap": 20.0}
+
+
+def tabopel_config(size: dict, kinds: str, loop: tuple[int, int, int] | None = None) -> dict:
+    """A Tabopel config.json.  ``kinds``: a letter per layer, "r" retention (half of Llama's heads, values twice as wide
+    as the keys), "c" the attention with a short convolution and a gate (Llama's heads, four taps, half of each head
+    turned), "n" the attention with capped scores (Llama's heads, all of each head turned), each with a dense feed-forward
+    of Llama's weight (two matrices in place of three); "e" the capped attention with a mixture of experts whose chosen
+    ones together are as wide, and one expert in sixteen handing its input on.  ``loop``: start, stop, times."""
+    half, dim, ff = size["heads"] // 2, size["dim"], size["ff"] * 3 // 2
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // size["top"]},
+           "router": {"experts": size["experts"], "top": size["top"], "identity": size["experts"] // 16}}
+    heads = {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+    layers = []
+    for kind in kinds:
+        if kind == "r":
+            decay = [1.0 - 2.0 ** (-5.0 - 5.0 * h / max(1, half - 1)) for h in range(half)]
+            layers.append({"type": "retention", "mlp": dense,
+                           "mixer": {"heads": half, "dim": dim, "vdim": 2 * dim, "decay": decay,
+                                     "rot": {"base": 10000.0, "dims": dim}}})
+        elif kind == "c":
+            scaling = {"factor": 4.0, "low": 1.0, "high": 2.0, "original": 4096}
+            layers.append({"type": "attention", "mlp": dense,
+                           "mixer": dict(heads, conv=4, rot={"base": 10000.0, "dims": dim // 2, "scaling": scaling})})
+        else:
+            layers.append({"type": "attention_2", "mlp": moe if kind == "e" else dense,
+                           "mixer": dict(heads, softcap=50.0, rot={"base": 10000.0, "dims": dim})})
+    config = {"architecture": "Tabopel", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5},
+              "embedding": {"scale": 24.0}, "layers": layers}
+    if loop is not None:
+        config["loop"] = {"start": loop[0], "stop": loop[1], "times": loop[2]}
+    return config
 
 
 def llama_config(size: dict) -> dict:
@@ -783,6 +818,17 @@ def compare_designs(args) -> int:
                 "mamevik_state": mamevik_config(size, "ssss", (0, 4, 1)),
                 "mamevik_latent": mamevik_config(size, "llll", (0, 4, 1)),
                 "mamevik_mixed": mamevik_config(size, "sll", (1, 2, 2)),      # one layer twice: four runs
+            })
+        elif args.designs_of == "tabopel":
+            models.update({
+                "rubuvik_lightning": rubuvik_config(size, "l"),
+                "rubuvik_sink_full": rubuvik_config(size, "b", window=None),
+                "mamevik_latent": mamevik_config(size, "llll", (0, 4, 1)),
+                "tabopel_retention": tabopel_config(size, "rrrr"),
+                "tabopel_conv": tabopel_config(size, "cccc"),
+                "tabopel_capped": tabopel_config(size, "nnnn"),
+                "tabopel_moe": tabopel_config(size, "eeee"),
+                "tabopel_mixed": tabopel_config(size, "rce", (0, 1, 2)),      # one layer twice: four runs
             })
         elif args.designs_of == "dutivik":
             models.update({
@@ -866,7 +912,7 @@ def main() -> int:
     parser.add_argument("--designs", action="store_true",
                         help="instead: Toposun (dense and mixture feed-forward) beside a Llama of equal layer sizes, "
                              "prefill and decode throughput and each kernel's share of a step; prints a line of its own")
-    parser.add_argument("--designs-of", default="toposun", choices=["toposun", "pipesun", "dutivik", "rubuvik", "mamevik"],
+    parser.add_argument("--designs-of", default="toposun", choices=["toposun", "pipesun", "dutivik", "rubuvik", "mamevik", "tabopel"],
                         help="which design --designs sets beside Llama")
     parser.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES), help="one size of --designs")
     args = parser.parse_args()

@@ -40,10 +40,13 @@ struct AddRowsParams {
   int width;
 };
 
-template <typename T, typename OUT, typename W, int N, bool AFTER>
-__global__ void __launch_bounds__(SR_THREADS)
+// THREADS a block, by the width alone (so are the sums): a wide row with a norm behind the sub-layer has two sums in a
+// chain, which more threads with fewer pieces each shorten
+template <typename T, typename OUT, typename W, int N, bool AFTER, int THREADS>
+__global__ void __launch_bounds__(THREADS)
 stream_add_rows_kernel(const AddRowsParams p) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_ADD_ROWS);
+  constexpr int PIECES = THREADS > SR_THREADS ? 1 : SR_PIECES;
   __shared__ float scratch[32];
   const int n = blockIdx.x, t = p.token_rows != nullptr ? p.token_rows[n] : n;
   const int width = p.width;
@@ -71,7 +74,7 @@ stream_add_rows_kernel(const AddRowsParams p) {
       for (int j = 0; j < N; ++j) a[j] = fmaf(w, to_float(r.v[j]), a[j]);
     }
   };
-  float kept[SR_PIECES][N];
+  float kept[PIECES][N];
   float ss = 0.0f, inv_a = 1.0f;
   // the new stream from what is added
   auto join = [&](int i, const RowPiece<float, N>& s, const RowPiece<W, N>& g, float (&v)[N]) {
@@ -114,11 +117,11 @@ stream_add_rows_kernel(const AddRowsParams p) {
     for (int j = 0; j < N; ++j) ss = fmaf(v[j], v[j], ss);
   };
   // the kept pieces: the stream's, the weights' and a slot's loads are each in flight together
-  RowPiece<float, N> xs[SR_PIECES];
-  RowPiece<W, N> ws[SR_PIECES], gs[AFTER ? SR_PIECES : 1];
+  RowPiece<float, N> xs[PIECES];
+  RowPiece<W, N> ws[PIECES], gs[AFTER ? PIECES : 1];
 #pragma unroll
-  for (int s = 0; s < SR_PIECES; ++s) {
-    const int i = (threadIdx.x + s * SR_THREADS) * N;
+  for (int s = 0; s < PIECES; ++s) {
+    const int i = (threadIdx.x + s * THREADS) * N;
 #pragma unroll
     for (int j = 0; j < N; ++j) kept[s][j] = 0.0f;
     if (i < width) {
@@ -132,29 +135,29 @@ stream_add_rows_kernel(const AddRowsParams p) {
     float w;
     const T* row = slot_row(slot, w);
     if (row == nullptr) continue;
-    RowPiece<T, N> r[SR_PIECES];
+    RowPiece<T, N> r[PIECES];
 #pragma unroll
-    for (int s = 0; s < SR_PIECES; ++s) {
-      const int i = (threadIdx.x + s * SR_THREADS) * N;
+    for (int s = 0; s < PIECES; ++s) {
+      const int i = (threadIdx.x + s * THREADS) * N;
       if (i < width) r[s] = *reinterpret_cast<const RowPiece<T, N>*>(row + i);
     }
 #pragma unroll
-    for (int s = 0; s < SR_PIECES; ++s) {
-      const int i = (threadIdx.x + s * SR_THREADS) * N;
+    for (int s = 0; s < PIECES; ++s) {
+      const int i = (threadIdx.x + s * THREADS) * N;
       if (i < width) {
 #pragma unroll
         for (int j = 0; j < N; ++j) kept[s][j] = fmaf(w, to_float(r[s].v[j]), kept[s][j]);
       }
     }
   }
-  const int rest = (threadIdx.x + SR_PIECES * SR_THREADS) * N;
+  const int rest = (threadIdx.x + PIECES * THREADS) * N;
   if (AFTER) {                                       // the root mean square of what is added
     float sa = 0.0f;
 #pragma unroll
-    for (int s = 0; s < SR_PIECES; ++s)              // (pieces beyond the width are zeros)
+    for (int s = 0; s < PIECES; ++s)              // (pieces beyond the width are zeros)
 #pragma unroll
       for (int j = 0; j < N; ++j) sa = fmaf(kept[s][j], kept[s][j], sa);
-    for (int i = rest; i < width; i += SR_THREADS * N) {
+    for (int i = rest; i < width; i += THREADS * N) {
       float a[N];
       added(i, a);
 #pragma unroll
@@ -163,15 +166,15 @@ stream_add_rows_kernel(const AddRowsParams p) {
     inv_a = 1.0f / sqrtf(block_sum(sa, scratch) / (float)width + p.after_eps);
   }
 #pragma unroll
-  for (int s = 0; s < SR_PIECES; ++s) {
-    const int i = (threadIdx.x + s * SR_THREADS) * N;
+  for (int s = 0; s < PIECES; ++s) {
+    const int i = (threadIdx.x + s * THREADS) * N;
     if (i < width) {
       join(i, xs[s], gs[AFTER ? s : 0], kept[s]);
       first_pass(i, kept[s]);
     }
   }
   // rows wider than the registers hold: the sum goes through `stream`, which the same thread reads again
-  for (int i = rest; i < width; i += SR_THREADS * N) {
+  for (int i = rest; i < width; i += THREADS * N) {
     float v[N];
     summed(i, v);
     first_pass(i, v);
@@ -187,11 +190,11 @@ stream_add_rows_kernel(const AddRowsParams p) {
     *reinterpret_cast<RowPiece<OUT, N>*>(dst + i) = r;
   };
 #pragma unroll
-  for (int s = 0; s < SR_PIECES; ++s) {
-    const int i = (threadIdx.x + s * SR_THREADS) * N;
+  for (int s = 0; s < PIECES; ++s) {
+    const int i = (threadIdx.x + s * THREADS) * N;
     if (i < width) put(i, kept[s], ws[s]);
   }
-  for (int i = rest; i < width; i += SR_THREADS * N) {
+  for (int i = rest; i < width; i += THREADS * N) {
     float v[N];
     if (p.stream != nullptr) {
       const RowPiece<float, N> s = *reinterpret_cast<const RowPiece<float, N>*>(p.stream + (size_t)t * width + i);
@@ -230,11 +233,14 @@ extern "C" int kvb_stream_add_rows(const float* x, const void* rows, int top, co
                      (packed == nullptr || (aligned16(packed) && aligned16(origin))) && aligned16(after) &&
                      aligned16(step) && aligned16(input);
   cudaError_t err;
-#define KVB_AR_SHAPE(T, OUT, W, N, A) \
-  kvb_launch((stream_add_rows_kernel<T, OUT, W, N, A>), dim3(count), dim3(SR_THREADS), 0, cuda_stream, true, p)
-#define KVB_AR(T, OUT, W)                                                                              \
-  err = after != nullptr ? (quads ? KVB_AR_SHAPE(T, OUT, W, 4, true) : KVB_AR_SHAPE(T, OUT, W, 1, true)) \
-                         : (quads ? KVB_AR_SHAPE(T, OUT, W, 4, false) : KVB_AR_SHAPE(T, OUT, W, 1, false))
+#define KVB_AR_SHAPE(T, OUT, W, N, A, TH) \
+  kvb_launch((stream_add_rows_kernel<T, OUT, W, N, A, TH>), dim3(count), dim3(TH), 0, cuda_stream, true, p)
+#define KVB_AR(T, OUT, W)                                                                                        \
+  err = after == nullptr ? (quads ? KVB_AR_SHAPE(T, OUT, W, 4, false, 256) : KVB_AR_SHAPE(T, OUT, W, 1, false, 256)) \
+        : !quads         ? KVB_AR_SHAPE(T, OUT, W, 1, true, 256)                                                  \
+        : width <= 1024  ? KVB_AR_SHAPE(T, OUT, W, 4, true, 256)                                                  \
+        : width <= 2048  ? KVB_AR_SHAPE(T, OUT, W, 4, true, 512)                                                  \
+                         : KVB_AR_SHAPE(T, OUT, W, 4, true, 1024)
   const int code = (dtype == KVB_BF16 ? 4 : 0) | (out_dtype == KVB_BF16 ? 2 : 0) | (weight_dtype == KVB_BF16 ? 1 : 0);
   switch (code) {
     case 0: KVB_AR(float, float, float); break;

@@ -2108,6 +2108,24 @@ def moe_group(ids: torch.Tensor, experts: int, *, for_library: bool, identity: i
     return g
 
 
+def _rounded_rows(rows: int) -> int:
+    """An expert's rows rounded up to 64, and beyond 512 to an eighth of the power of two below: the library chooses a
+    kernel anew for every shape it has not met, about a millisecond each."""
+    unit = 64 if rows <= 512 else 1 << (rows.bit_length() - 4)
+    return -(-rows // unit) * unit
+
+
+_one_runs: dict[torch.device, torch.Tensor] = {}
+
+
+def _one_run(device: torch.device) -> torch.Tensor:
+    """Bounds of a single run of rows that begins at 0 and has no end (``moe_gather`` in the order of the grouping)."""
+    bounds = _one_runs.get(device)
+    if bounds is None:
+        bounds = _one_runs[device] = torch.tensor([0, 1 << 30], dtype=torch.int32, device=device)
+    return bounds
+
+
 def moe_path(x: torch.Tensor, pairs: int, ff: int) -> str:
     """Which way ``moe_experts`` takes for a batch of ``pairs`` (token, expert) pairs of ``x``'s type."""
     if x.dtype != torch.bfloat16:
@@ -2202,32 +2220,41 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_
     max_tiles, capacity = grouping.max_tiles, grouping.capacity
     if library:
         begins = grouping.begins()                # the one read-back: how many rows each expert got
+        if not begins[experts]:                   # every pair of the batch hands its input on: a row that nobody reads
+            return ExpertRows(torch.zeros((1, n), dtype=x.dtype, device=x.device), row_of_pair,
+                              None if weight_on_input else weights.reshape(-1), top, own)
         # the common stride: the fullest expert's rows, rounded up to 64 so that the library sees few
         # different shapes (it chooses a kernel anew for every shape it has not met: about a millisecond)
         stride = -(-max(begins[e + 1] - begins[e] for e in range(experts)) // 64) * 64
-        gathered = torch.empty((experts, stride, k), dtype=x.dtype, device=x.device)
-        _call("kvb_moe_gather", gathered.data_ptr(), x.data_ptr(), x.stride(0), top,
-              weights.data_ptr() if weight_on_input else None, sorted_pairs.data_ptr(), expert_begin.data_ptr(),
-              experts, stride, row_of_pair.data_ptr(), k, code, _stream())
         # every expert's rows at one stride: two batched library products over all experts (an expert with
         # fewer pairs multiplies zero rows; with one expert far fuller than the rest, expert by expert instead)
         if experts * stride <= 2 * capacity + experts * 64:
+            gathered = torch.empty((experts, stride, k), dtype=x.dtype, device=x.device)
+            _call("kvb_moe_gather", gathered.data_ptr(), x.data_ptr(), x.stride(0), top,
+                  weights.data_ptr() if weight_on_input else None, sorted_pairs.data_ptr(), expert_begin.data_ptr(),
+                  experts, stride, row_of_pair.data_ptr(), k, code, _stream())
             both = torch.bmm(gathered, gate_up.transpose(1, 2))
             hidden = activate(both.view(experts * stride, two_ff)).view(experts, stride, ff)
             out = torch.bmm(hidden, down.transpose(1, 2)).view(experts * stride, n)
         else:
-            # an expert's rows rounded up to 64 as well (the rows beyond its pairs are zeros): few shapes again
-            counts = [min(stride, -(-(begins[e + 1] - begins[e]) // 64) * 64) for e in range(experts)]
-            both = torch.zeros((experts, stride, two_ff), dtype=x.dtype, device=x.device)
-            for e in range(experts):
-                if counts[e]:
-                    torch.mm(gathered[e, : counts[e]], gate_up[e].t(), out=both[e, : counts[e]])
-            hidden = activate(both.view(experts * stride, two_ff)).view(experts, stride, ff)
-            out = torch.empty((experts, stride, n), dtype=x.dtype, device=x.device)
-            for e in range(experts):
-                if counts[e]:
-                    torch.mm(hidden[e, : counts[e]], down[e].t(), out=out[e, : counts[e]])
-            out = out.view(experts * stride, n)
+            # The rows expert by expert without gaps, as the grouping has them.  A product takes an expert's rows
+            # rounded up (few different shapes again) and so runs over into the rows behind, which belong to later
+            # experts and are written by their own products after it; the last rows are nobody's.
+            total = begins[experts]
+            counts = [_rounded_rows(begins[e + 1] - begins[e]) for e in range(experts)]
+            spare = max(begins[e] + counts[e] for e in range(experts)) - total
+            gathered = torch.empty((total + spare, k), dtype=x.dtype, device=x.device)
+            _call("kvb_moe_gather", gathered.data_ptr(), x.data_ptr(), x.stride(0), top,
+                  weights.data_ptr() if weight_on_input else None, sorted_pairs.data_ptr(),
+                  _one_run(x.device).data_ptr(), 1, total, row_of_pair.data_ptr(), k, code, _stream())
+            both = torch.empty((total + spare, two_ff), dtype=x.dtype, device=x.device)
+            out = torch.empty((total + spare, n), dtype=x.dtype, device=x.device)
+            spans = [(e, begins[e], begins[e] + counts[e]) for e in range(experts) if counts[e]]
+            for e, lo, hi in spans:
+                torch.mm(gathered[lo:hi], gate_up[e].t(), out=both[lo:hi])
+            hidden = activate(both)
+            for e, lo, hi in spans:
+                torch.mm(hidden[lo:hi], down[e].t(), out=out[lo:hi])
         return ExpertRows(out, row_of_pair, None if weight_on_input else weights.reshape(-1), top, own)
     hidden = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
     _call("kvb_moe_gemm", hidden.data_ptr(), x.data_ptr(), x.stride(0), top,

@@ -1,0 +1,725 @@
+"""The Tabopel decoder through the framework (configuration, loader, cache manager, step function, scheduler, entry
+point) against the plain statement in tests/plain_tabopel.py, on the host with the stand-in kernels and on the GPU with
+the CUDA kernels, in 32-bit and in bfloat16.
+
+Small configurations of their own and random weights: whole prompts against token-by-token decoding, portions down to one
+and two tokens, mixed batches against each request alone, pages and state slots used again (freed pages overwritten), the
+first tokens of a request (nothing in the convolution, little in the softmax beside the sink), long decoding across
+pages, a key that stands out far back and at page borders, the oldest input that a convolution still reads and the next
+one that it does not, a token that only the recurrence carries on, loops at the start, in the middle and at the end, sizes
+that make mechanisms coincide (one head, one tap, nothing turned, equal key and value widths, every expert chosen, none
+that hands its input on, one pass of the loop, no loop), and greedy generation through the entry point."""
+from __future__ import annotations
+
+import json
+import math
+
+import numpy as np
+import pytest
+import torch
+
+import plain_kernels
+import plain_tabopel as P
+import replay_cases as rc
+from kvcore_b200 import (CacheConfig, DeviceConfig, KVCoreConfig, ModelConfig, SamplingParams, SchedulerConfig)
+from kvcore_b200.config import ConfigError
+from kvcore_b200.config.registry import model_spec_from_config, model_spec_from_folder
+from kvcore_b200.engine.llm_engine import GenerationRequest, LLMEngine
+from kvcore_b200.weights.safetensors_io import write_safetensors
+
+BACKENDS = [pytest.param("cpu", id="host"), pytest.param("cuda:0", id="gpu", marks=pytest.mark.gpu)]
+# largest |difference| of a row over the request's largest |logit|; in bfloat16 also the root mean square of a
+# row's difference (its mean taken off) over that of the request's logits.  A wrong key, a lost state or a
+# convolution one token off moves a row by 1e-2 and more (test_each_mechanism_changes_the_logits); the 32-bit
+# runs hold every position to 5e-5.  In bfloat16 a single row may stray further than the median row.
+TOLERANCE = {"float32": 5e-5}
+BF16_ROW_TOLERANCE = 1e-1
+BF16_MEDIAN_RMS_TOLERANCE = 3.5e-2
+# a position where a router's choice hangs on less than this (relative to the score) is left out of the bfloat16 runs
+BF16_ROUTER_MARGIN = 0.1
+
+
+@pytest.fixture(params=BACKENDS)
+def device(request, monkeypatch):
+    if request.param == "cpu":
+        plain_kernels.install(monkeypatch)
+    return request.param
+
+
+A, C, R, rot = P.conv_attention, P.capped_attention, P.retention, P.rotation
+CONFIGS = {
+    # every mixer with either feed-forward or none, a loop over the middle layers that begins with a recurrence
+    "all_kinds": P.model_config([
+        C(heads=6, kv_heads=2, dim=16, vdim=24, rot=rot(10, 500.0), softcap=2.5, scale=0.4,
+          mlp=P.moe(experts=5, top=2, ff=20, identity=2)),
+        R(dim=12, vdim=20, decay=(0.6, 0.9, 0.98), rot=rot(8, 300.0), mlp=P.dense(28)),
+        A(heads=4, kv_heads=2, dim=14, vdim=6, conv=4, rot=rot(14, 10000.0, (4.0, 1.0, 3.0, 40)), mlp=None),
+        A(heads=3, kv_heads=1, dim=24, vdim=16, conv=2, rot=rot(6, 100.0), scale=0.3,
+          mlp=P.moe(experts=4, top=3, ff=12, identity=1)),
+        R(dim=20, vdim=8, decay=(0.97,), rot=rot(20, 1000.0), mlp=P.moe(experts=3, top=1, ff=16, identity=0)),
+    ], vocab=83, width=40, loop=(1, 3, 2), eps=1e-5, scale=0.7),
+    # what the first makes unequal is equal or 1 here and the other way round: one head, key and value heads of their own,
+    # one tap and more than a thread's window holds, two turned entries, a decay of one (nothing is lost), every expert
+    # chosen, a single expert, a loop over everything taken once, sizes no 16-byte vector fits
+    "coincide": P.model_config([
+        R(dim=10, vdim=14, decay=(1.0, 0.8), rot=rot(2, 10.0), mlp=P.moe(experts=3, top=4, ff=6, identity=1)),
+        C(heads=1, kv_heads=1, dim=10, vdim=10, rot=rot(10, 10000.0), softcap=60.0, mlp=P.moe(experts=1, top=1, ff=10, identity=0)),
+        A(heads=3, kv_heads=3, dim=6, vdim=7, conv=1, rot=rot(2, 50.0, (8.0, 1.0, 4.0, 32)), mlp=P.dense(9)),
+        A(heads=2, kv_heads=1, dim=8, vdim=5, conv=11, rot=rot(8, 50.0), mlp=None),
+    ], vocab=61, width=42, loop=(0, 4, 1), eps=1e-6),
+    # sizes the tensor-core attention and the streaming products take, contexts across several pages, state sizes that are
+    # shared by several threads a column, a loop at the end
+    "serving_sizes": P.model_config([
+        R(dim=64, vdim=48, decay=(0.9, 0.97, 0.99, 0.995), rot=rot(32, 10000.0), mlp=P.dense(128)),
+        A(heads=4, kv_heads=2, dim=32, vdim=64, conv=3, rot=rot(32, 20000.0, (2.0, 1.0, 4.0, 128)),
+          mlp=P.moe(experts=8, top=2, ff=32, identity=2)),
+        C(heads=8, kv_heads=2, dim=48, vdim=32, rot=rot(16, 5000.0), softcap=4.0, mlp=P.moe(experts=16, top=4, ff=16, identity=1)),
+    ], vocab=128, width=64, loop=(1, 3, 2), eps=1e-5, scale=2.0),
+}
+LENGTHS = {"all_kinds": (1, 23, 45, 70, 37, 2), "coincide": (64, 1, 30, 50), "serving_sizes": (150, 3, 97, 61)}
+
+
+def write_folder(folder, cfg, seed, weights=None):
+    weights = P.random_weights(cfg, seed) if weights is None else weights
+    folder.mkdir(parents=True, exist_ok=True)
+    (folder / "config.json").write_text(json.dumps(cfg))
+    write_safetensors(folder / "model.safetensors", {k: v.to(torch.bfloat16) for k, v in weights.items()})
+    return {k: v.to(torch.bfloat16).double() for k, v in weights.items()}
+
+
+def references(cfg, weights, requests):
+    reference, margins = {}, {}
+    for rid, toks in requests.items():
+        seen = []
+        reference[rid] = P.forward(cfg, weights, toks, margins=seen).numpy()
+        margins[rid] = seen[0].numpy()
+    return reference, margins
+
+
+@pytest.fixture(scope="module", params=list(CONFIGS))
+def case(request, tmp_path_factory):
+    name = request.param
+    cfg = CONFIGS[name]
+    folder = tmp_path_factory.mktemp(f"tabopel_{name}")
+    weights = write_folder(folder, cfg, seed=len(name))
+    requests = {f"q{i}": rc.random_tokens(cfg["vocab"], n, 30 + i) for i, n in enumerate(LENGTHS[name])}
+    reference, margins = references(cfg, weights, requests)
+    return dict(name=name, cfg=cfg, folder=folder, weights=weights, requests=requests, reference=reference,
+                margins=margins)
+
+
+def compare(rows, reference, dtype, margins=None):
+    """32-bit: every row within TOLERANCE.  bfloat16: rows whose own router margin is small are left out; a row
+    in front of which some router chose otherwise (these narrow models' streams carry a percent of rounding, and a
+    state or a cached key hands a changed row on) may stray, so up to 6 % of the rows may lie beyond the row
+    tolerance, while the median row must stay within BF16_MEDIAN_RMS_TOLERANCE: a kernel that is a little
+    wrong everywhere fails the second, a wrong key or a lost state the 32-bit runs and the kernels' own tests."""
+    assert rows
+    spread, beyond = [], []
+    for (rid, pos), row in sorted(rows.items()):
+        assert np.isfinite(row).all(), f"non-finite logits for {rid}@{pos}"
+        err = np.abs(row - reference[rid][pos]).max() / np.abs(reference[rid]).max()
+        if dtype == "float32":
+            assert err <= TOLERANCE[dtype], f"{rid}: first wrong position {pos} (error {err:.3e})"
+            continue
+        if margins is not None and margins[rid][pos] < BF16_ROUTER_MARGIN:
+            continue
+        diff = row - reference[rid][pos]
+        rms = np.sqrt(np.mean((diff - diff.mean()) ** 2)) / reference[rid].std()
+        spread.append(rms)
+        if max(err, rms) > BF16_ROW_TOLERANCE:
+            beyond.append((rid, pos, float(max(err, rms))))
+    if spread:
+        assert len(beyond) <= max(2, 0.06 * len(spread)), f"{len(beyond)} of {len(spread)} rows stray: {beyond[:8]}"
+        assert np.median(spread) <= BF16_MEDIAN_RMS_TOLERANCE, f"median rms error {np.median(spread):.3e}"
+
+
+# ---- configuration -----------------------------------------------------------------------------------
+def test_config_names_the_tensors_of_the_plain_statement(case):
+    from kvcore_b200.parts.model import build_model
+
+    spec = model_spec_from_folder(case["folder"])
+    assert spec.architecture == "Tabopel"
+    model = build_model(spec, dtype=torch.float32, device="meta")
+    assert {slot.name: slot.shape for slot in model.weight_slots()} == P.tensor_shapes(case["cfg"])
+
+
+def test_config_gives_every_constant_to_the_parts():
+    spec = model_spec_from_config(CONFIGS["all_kinds"])
+    assert [(e.layer, e.ahead, e.cache_of) for e in spec.schedule] == [
+        (0, None, None), (1, ("loop", 0), None), (2, None, None), (1, ("loop", 1), None), (2, None, None),
+        (3, None, None), (4, None, None)]
+    step = spec.stream_steps["loop"]
+    assert step.kind == "add_step" and (step.params["times"], step.params["hidden_size"]) == (2, 40)
+    assert spec.embedding.params["scale"] == 0.7 and spec.lm_head.params["tensor"] == "head"
+    p = spec.layers[0].mixer.params
+    assert (p["num_heads"], p["num_kv_heads"], p["head_dim"], p["value_dim"], p["scale"], p["softcap"], p["eps"]) == \
+        (6, 2, 16, 24, 0.4, 2.5, 1e-5)
+    assert (p["bias"], p["qk_norm"], p["sink"], p["gate"], p["conv_taps"]) == (True, True, "learned", False, 0)
+    assert dict(p["position"].params) == dict(head_dim=16, rotary_dim=10, theta=500.0)
+    p = spec.layers[1].mixer.params
+    assert (p["num_heads"], p["head_dim"], p["value_dim"], p["decay"]) == (3, 12, 20, (0.6, 0.9, 0.98))
+    p = spec.layers[2].mixer.params
+    assert (p["bias"], p["qk_norm"], p["sink"], p["gate"], p["conv_taps"], p["softcap"]) == (False, False, "one", True, 4, None)
+    assert dict(p["position"].params) == dict(head_dim=14, rotary_dim=14, theta=10000.0, rope_type="llama3", factor=4.0,
+                                              low_freq_factor=1.0, high_freq_factor=3.0, original_max_position_embeddings=40)
+    moe = spec.layers[0].feed_forward.params
+    assert (moe["num_experts"], moe["identity_experts"], moe["top_k"], moe["expert_size"], moe["activation"], moe["score"],
+            moe["weight_on"], moe["choice_correction"], moe["renormalize"]) == (5, 2, 2, 20, "squared_relu", "softmax", "output", True, False)
+    assert spec.layers[1].feed_forward.kind == "squared_relu" and spec.layers[1].feed_forward.params["intermediate_size"] == 28
+    assert spec.layers[2].feed_forward is None and set(spec.layers[2].norms) == {"mixer_norm", "mixer_out_norm"}
+    assert all(n.params["eps"] == 1e-5 for n in spec.layers[0].norms.values())
+    # keys that a model may leave out
+    bare = json.loads(json.dumps(CONFIGS["all_kinds"]))
+    bare.pop("loop")
+    bare["layers"][0]["mlp"]["router"].pop("identity")
+    bare["layers"][0]["mixer"].pop("softcap")
+    bare["layers"][1]["mixer"].pop("rot")
+    bare["layers"][2]["mixer"].pop("conv")
+    plain = model_spec_from_config(bare)
+    assert [(e.layer, e.ahead) for e in plain.schedule] == [(i, None) for i in range(5)] and not plain.stream_steps
+    assert plain.layers[0].feed_forward.params["identity_experts"] == 0 and plain.layers[0].mixer.params["softcap"] is None
+    assert plain.layers[1].mixer.params["position"] is None and plain.layers[2].mixer.params["conv_taps"] == 0
+
+
+@pytest.mark.parametrize("change,message", [
+    (lambda c: c["layers"][0].update(type="lightning"), "mixer of this design"),
+    (lambda c: c["layers"][0]["mlp"].update(kind="glu"), "feed-forward of this design"),
+    (lambda c: c["layers"][0]["mixer"].update(kv_heads=4), "multiple"),
+    (lambda c: c["layers"][0]["mixer"]["rot"].update(dims=9), "even"),
+    (lambda c: c["layers"][0]["mixer"]["rot"].update(dims=18), "at most dim"),
+    (lambda c: c["layers"][0]["mixer"].update(softcap=0.0), "softcap"),
+    (lambda c: c["layers"][0]["mixer"].pop("scale"), "scale"),
+    (lambda c: c["layers"][0]["mlp"]["router"].update(top=8), "exceeds experts"),
+    (lambda c: c["layers"][0]["mlp"]["router"].update(identity=-1), "identity"),
+    (lambda c: c["layers"][0]["mlp"].pop("expert"), "expert"),
+    (lambda c: c["layers"][1]["mixer"].update(decay=[0.5, 0.5]), "decay"),
+    (lambda c: c["layers"][1]["mixer"]["decay"].__setitem__(0, -0.1), "decay"),
+    (lambda c: c["layers"][1]["mlp"].update(ff=0), "ff"),
+    (lambda c: c["layers"][2]["mixer"].update(conv=0), "conv"),
+    (lambda c: c["layers"][2]["mixer"]["rot"]["scaling"].pop("low"), "low"),
+    (lambda c: c["layers"][2]["mixer"]["rot"]["scaling"].update(factor=0.0), "scaling"),
+    (lambda c: c["loop"].update(stop=6), "loop over layers"),
+    (lambda c: c["loop"].update(times=0), "times"),
+    (lambda c: c["embedding"].pop("scale"), "scale"),
+    (lambda c: c.pop("norm"), "norm"),
+])
+def test_config_refuses(change, message):
+    cfg = json.loads(json.dumps(CONFIGS["all_kinds"]))
+    change(cfg)
+    with pytest.raises(ConfigError, match=message):
+        model_spec_from_config(cfg)
+
+
+def test_cache_groups_and_state():
+    """A pass of the loop has pages and states of its own; attention layers of one row width share a page group; a
+    retention keeps no pages and one state row a request and pass; a convolution keeps pages and a state row."""
+    from kvcore_b200.cache.kv_manager import group_entries
+    from kvcore_b200.parts.model import build_model
+
+    model = build_model(model_spec_from_config(CONFIGS["all_kinds"]), dtype=torch.float32, device="meta")
+    requirements = model.entry_requirements()
+    groups, entry_group = group_entries(requirements)
+    assert [(g.planes, g.heads, g.width, g.window, g.entries) for g in groups] == [
+        (1, 1, 2 * (16 + 24), None, (0,)), (1, 1, 2 * (14 + 6), None, (2, 4, 5))]
+    assert entry_group == {0: 0, 2: 1, 4: 1, 5: 1}
+    memory, last = 3 * 12 * 20, 20 * 8
+    conv, short = (4 * 14 + 2 * 20) * 3, 3 * 24 + 24 + 16
+    assert [None if r.state_spec is None else r.state_spec.shape for r in requirements] == [
+        None, (memory,), (conv,), (memory,), (conv,), (short,), (last,)]
+
+
+def test_unused_tensors_of_a_checkpoint_are_accepted(device, tmp_path):
+    """A layer without a feed-forward may carry the norms around one."""
+    from kvcore_b200.engine.trace_replay import build_replay
+
+    cfg = CONFIGS["coincide"]
+    weights = P.random_weights(cfg, 3)
+    weights["l3.norm2"] = weights["l3.norm2b"] = torch.ones(cfg["width"])
+    write_folder(tmp_path / "m", cfg, 3, weights)
+    build_replay(str(tmp_path / "m"), "float32", 64, device=device)
+
+
+# ---- the cuttings ---------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_cuttings_match_the_plain_statement(case, dtype, device, tmp_path):
+    cfg, requests = case["cfg"], case["requests"]
+    traces = {
+        "whole": rc.trace_whole(requests),
+        "tail": rc.trace_decode_tail(requests, tail=26),
+        "chunks": rc.trace_chunks(requests, sizes=(7, 3, 16, 2, 5, 1, 9, 2, 31)),
+        "mixed": rc.trace_mixed(requests, max_live=4, seed=3),
+    }
+    results = {}
+    for name, steps in traces.items():
+        out = tmp_path / name
+        rc.run_inprocess(case["folder"], dtype, steps, out, rc.peak_tokens(steps), device=device,
+                         fill_freed_pages="poison" if name == "mixed" else None)
+        rows = rc.collect(steps, out, cfg["vocab"])
+        assert len(rows) == sum(len(t) for t in requests.values())
+        compare(rows, case["reference"], dtype, case["margins"])
+        results[name] = rows
+    if dtype == "float32" and device != "cpu":
+        # every kernel of the 32-bit path sums in an order that depends on the position only
+        for name in ("tail", "chunks", "mixed"):
+            for key, row in results["whole"].items():
+                assert np.array_equal(row, results[name][key]), f"{name} differs from whole at {key}"
+
+
+def test_residual_stream_after_every_layer(case, device):
+    """Layer by layer, every pass of the loop counted: the 32-bit stream plus what the block leaves to the kernel behind
+    it, against the plain statement's, in two portions (the second begins with a convolution and a state to carry over)."""
+    from kvcore_b200.engine.step import StepEntry
+    from kvcore_b200.engine.trace_replay import build_replay
+    from kvcore_b200.parts.norm import add_pending
+
+    tokens = case["requests"]["q1"] if len(case["requests"]["q1"]) > 2 else case["requests"]["q2"]
+    step_function, kv = build_replay(str(case["folder"]), "float32", 256, device=device)
+    seen = []
+    for block in step_function.model.blocks:
+        original = block.forward
+
+        def recording(h, residual, ctx, cache, original=original):
+            out = original(h, residual, ctx, cache)
+            seen.append(add_pending(out[1].clone(), out[0])[0].cpu())
+            return out
+        block.forward = recording
+    cut = len(tokens) // 3 + 1
+    runs = len(step_function.model.schedule)
+    assert kv.allocate_slots("x", cut)
+    step_function.step([StepEntry("x", tokens[:cut], [])])
+    assert kv.allocate_slots("x", len(tokens) - cut)
+    step_function.step([StepEntry("x", tokens[cut:], [len(tokens) - cut - 1])])
+    collected = []
+    P.forward(case["cfg"], case["weights"], tokens, streams=collected)
+    assert len(seen) == 2 * runs and len(collected) == runs
+    for index, want in enumerate(collected):
+        got = torch.cat([seen[index], seen[runs + index]])
+        assert got.dtype == torch.float32
+        torch.testing.assert_close(got.double(), want, rtol=5e-5, atol=1e-4, msg=lambda m: f"layer run {index}: {m}")
+
+
+def test_pages_and_slots_are_used_again(case, device, tmp_path):
+    """A pool for the largest live set only: the trace needs more pages over its life than the pool has and
+    more requests than state slots in a row, so a new request finds a page and a state row that another has
+    left (the row must read as zeros, the page must not be read before it is written)."""
+    requests = dict(case["requests"])
+    requests.update({f"again{i}": toks for i, toks in enumerate(case["requests"].values())})
+    steps = rc.trace_mixed(requests, max_live=3, seed=11)
+    peak = rc.peak_tokens(steps)
+    assert sum(-(-len(t) // 16) * 16 for t in requests.values()) > peak
+    out = tmp_path / "o"
+    step_function, kv = rc.run_inprocess(case["folder"], "float32", steps, out, peak, device=device,
+                                         fill_freed_pages="poison")
+    assert all(pool.num_free == pool.num_usable for pool in kv.pools)
+    reference = dict(case["reference"])
+    reference.update({f"again{i}": ref for i, ref in enumerate(case["reference"].values())})
+    compare(rc.collect(steps, out, case["cfg"]["vocab"]), reference, "float32")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_long_decoding(dtype, device, tmp_path):
+    """Two prompt tokens, then single tokens: pages fill up one after the other, the convolutions and the states run on
+    (on the GPU: decode graphs captured and replayed)."""
+    cfg = CONFIGS["serving_sizes"] if device != "cpu" else CONFIGS["all_kinds"]
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, seed=5)
+    tokens = rc.random_tokens(cfg["vocab"], 200 if device != "cpu" else 60, 77)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": tokens[:2], "want": [0, 1]}], "end": []}]
+    for pos in range(2, len(tokens)):
+        steps.append({"step": pos - 1, "entries": [{"id": "a", "tokens": [tokens[pos]], "want": [0]}],
+                      "end": ["a"] if pos == len(tokens) - 1 else []})
+    out = tmp_path / "o"
+    rc.run_inprocess(folder, dtype, steps, out, 256, device=device, fill_freed_pages="poison")
+    reference, margins = references(cfg, weights, {"a": tokens})
+    compare(rc.collect(steps, out, cfg["vocab"]), reference, dtype, margins)
+
+
+@pytest.mark.gpu
+def test_long_portions_beside_single_tokens(tmp_path):
+    """Portions whose experts go the way of prompts, beside short ones and single tokens, in bfloat16."""
+    cfg = CONFIGS["serving_sizes"]
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, seed=8)
+    requests = {rid: rc.random_tokens(cfg["vocab"], n, 300 + n) for rid, n in (("long", 700), ("short", 40), ("one", 5))}
+    parts = ([("long", 300)], [("long", 60), ("short", 30), ("one", 3)], [("long", 340), ("short", 10), ("one", 1)], [("one", 1)])
+    at, steps = {rid: 0 for rid in requests}, []
+    for portion in parts:
+        entries = []
+        for rid, n in portion:
+            entries.append({"id": rid, "tokens": requests[rid][at[rid]:at[rid] + n], "want": list(range(n))})
+            at[rid] += n
+        steps.append({"step": len(steps), "entries": entries, "end": []})
+    steps[-1]["end"] = list(requests)
+    assert at == {rid: len(t) for rid, t in requests.items()}
+    reference, margins = references(cfg, weights, requests)
+    for dtype in ("float32", "bfloat16"):
+        rc.run_inprocess(folder, dtype, steps, tmp_path / dtype, rc.peak_tokens(steps), device="cuda:0", fill_freed_pages="poison")
+        compare(rc.collect(steps, tmp_path / dtype, cfg["vocab"]), reference, dtype, margins)
+
+
+# ---- faults that random weights would hide ----------------------------------------------------------------
+def _bare_model(layer, seed):
+    """One layer of the mixer alone, every weight zero but the norms (ones), the output matrix, the values' matrix, the
+    head and the tokens' rows; the first two entries of the stream belong to tokens 1 and 2."""
+    cfg = P.model_config([layer], vocab=24, width=32)
+    w = {name: torch.zeros(shape) for name, shape in P.tensor_shapes(cfg).items()}
+    g = torch.Generator().manual_seed(seed)
+    w["embed"] = torch.randn(24, 32, generator=g)
+    w["embed"][:, :2] = 0.0
+    w["embed"][1, 0], w["embed"][2, 1] = 6.0, 6.0
+    for name in w:
+        if "norm" in name:
+            w[name] = torch.ones_like(w[name])
+    for name in ("head", "l0.mix.o", "l0.mix.v"):
+        w[name] = torch.randn(w[name].shape, generator=g)
+    return cfg, w
+
+
+def _standout_model(kind):
+    """Attention in which the query of token 2 meets the key of token 1 in a score that takes the whole softmax, along an
+    entry that does not turn."""
+    if kind == "attention":
+        cfg, w = _bare_model(A(heads=2, kv_heads=1, dim=16, vdim=20, conv=3, rot=rot(8, 100.0), scale=0.5), 3)
+        for n in "qkv":
+            w[f"l0.mix.{n}.conv"][:, -1] = 1.0
+    else:
+        cfg, w = _bare_model(C(heads=2, kv_heads=1, dim=16, vdim=20, rot=rot(8, 100.0), softcap=9.0, scale=1.0), 3)
+        w["l0.mix.sink"] = torch.tensor([1.0, -1.0])
+    w["l0.mix.q"][12, 1], w["l0.mix.k"][12, 0] = 4.0, 4.0      # entry 12 of head 0
+    return cfg, w
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("kind", ["attention", "attention_2"])
+def test_a_key_that_stands_out(kind, dtype, device, tmp_path):
+    """A dominating key far back, right in front, at page borders and at the first position, in prompts and decoded."""
+    cfg, w = _standout_model(kind)
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, 0, w)
+    requests = {}
+    for distance in (1, 2, 16, 90):
+        for place in (0, 3, 15, 16):                           # where the key stands
+            tokens = [t + 3 for t in rc.random_tokens(20, place + distance + 4, 7 * distance + place)]
+            tokens[place], tokens[place + distance] = 1, 2
+            requests[f"d{distance}p{place}"] = tokens
+    reference, _ = references(cfg, weights, requests)
+    for rid, tokens in requests.items():                       # without that key the query's logits are others
+        place, distance = int(rid.split("p")[1]), int(rid[1:].split("p")[0])
+        other = list(tokens)
+        other[place] = 3
+        moved = np.abs(P.forward(cfg, weights, other).numpy()[place + distance] - reference[rid][place + distance]).max()
+        assert moved > 0.2 * np.abs(reference[rid]).max()
+    for name, steps in (("whole", rc.trace_whole(requests)), ("tail", rc.trace_decode_tail(requests, tail=5)),
+                        ("chunks", rc.trace_chunks(requests, sizes=(5, 2, 16, 3)))):
+        out = tmp_path / name
+        rc.run_inprocess(folder, dtype, steps, out, rc.peak_tokens(steps), device=device, fill_freed_pages="poison")
+        for (rid, pos), row in rc.collect(steps, out, cfg["vocab"]).items():
+            err = np.abs(row - reference[rid][pos]).max() / np.abs(reference[rid]).max()
+            assert err <= (TOLERANCE[dtype] if dtype == "float32" else 4e-2), f"{name}: {rid}@{pos}: {err:.3e}"
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("taps", [2, 4, 6])
+def test_the_oldest_input_of_a_convolution(taps, dtype, device, tmp_path):
+    """A convolution whose oldest tap alone reads: the query turns to the key of the token ``taps - 1`` in front of which
+    token 1 stands, not one nearer or farther; with a portion's beginning at every place in between."""
+    cfg, w = _bare_model(A(heads=1, kv_heads=1, dim=8, vdim=12, conv=taps, rot=rot(4, 100.0), scale=0.5), 5)
+    for n in "qkv":
+        w[f"l0.mix.{n}.conv"][:, 0] = 1.0
+    w["l0.mix.q"][6, 1], w["l0.mix.k"][6, 0] = 4.0, 4.0
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, 0, w)
+    tokens = [t + 3 for t in rc.random_tokens(20, 30, 9)]
+    tokens[4], tokens[13] = 1, 2                               # acts at 4 + taps - 1, asks at 13 + taps - 1
+    requests = {f"c{n}": tokens for n in range(1, taps + 3)}
+    reference, _ = references(cfg, weights, requests)
+    at = 13 + taps - 1
+    for wrong in (1, -1):                                      # a convolution that reaches one token more or less
+        other = dict(weights)
+        for n in "qkv":
+            moved = torch.zeros(weights[f"l0.mix.{n}.conv"].shape[0], taps + 1, dtype=torch.float64)
+            moved[:, 0 if wrong > 0 else 2] = 1.0
+            other[f"l0.mix.{n}.conv"] = moved
+        off = P.forward(cfg, other, tokens).numpy()
+        assert np.abs(off[at] - reference["c1"][at]).max() > 0.1 * np.abs(reference["c1"]).max()
+    steps = []
+    for n, rid in enumerate(requests, start=1):                # portions that end n tokens into the reach
+        for begin, end in ((0, 4 + n), (4 + n, 13 + n), (13 + n, 14 + n), (14 + n, 30)):
+            steps.append({"step": len(steps), "end": [rid] if end == 30 else [],
+                          "entries": [{"id": rid, "tokens": tokens[begin:end], "want": list(range(end - begin))}]})
+    for name, trace in (("cut", steps), ("tail", rc.trace_decode_tail({"c1": tokens}, tail=28))):
+        out = tmp_path / name
+        rc.run_inprocess(folder, dtype, trace, out, rc.peak_tokens(trace), device=device)
+        for (rid, pos), row in rc.collect(trace, out, cfg["vocab"]).items():
+            err = np.abs(row - reference[rid][pos]).max() / np.abs(reference[rid]).max()
+            assert err <= (TOLERANCE[dtype] if dtype == "float32" else 4e-2), f"{name}: {rid}@{pos}: {err:.3e}"
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_token_far_back_that_only_the_state_carries(dtype, device, tmp_path):
+    """A retention that takes in one token (the keys of the others are zero) and reads it out at the end: a hundred tokens
+    on, in prompts, portions and decoded steps."""
+    cfg, w = _bare_model(R(dim=8, vdim=8, decay=(0.999, 0.99), rot=rot(4, 1000.0)), 4)
+    w["l0.mix.k"][6, 0] = w["l0.mix.k"][14, 0] = 6.0
+    w["l0.mix.q"][[6, 14]] = torch.randn(2, 32, generator=torch.Generator().manual_seed(2))
+    w["l0.mix.q"][[6, 14], 1] = 3.0
+    w["l0.mix.g"] = torch.randn(16, 32, generator=torch.Generator().manual_seed(6))
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, 0, w)
+    requests = {}
+    for place in (0, 9):
+        tokens = [t + 3 for t in rc.random_tokens(20, 110 + place, 50 + place)]
+        tokens[place] = 1
+        tokens[-1] = 2
+        requests[f"p{place}"] = tokens
+    reference, _ = references(cfg, weights, requests)
+    for rid, tokens in requests.items():                       # without that token the last logits are others
+        other = list(tokens)
+        other[int(rid[1:])] = 3
+        assert np.abs(P.forward(cfg, weights, other).numpy()[-1] - reference[rid][-1]).max() > 0.2 * np.abs(reference[rid]).max()
+    for name, steps in (("whole", rc.trace_whole(requests)), ("tail", rc.trace_decode_tail(requests, tail=100)),
+                        ("chunks", rc.trace_chunks(requests, sizes=(2, 13, 3, 1, 2))),
+                        ("mixed", rc.trace_mixed(requests, max_live=2, seed=2))):
+        out = tmp_path / name
+        rc.run_inprocess(folder, dtype, steps, out, rc.peak_tokens(steps), device=device)
+        for (rid, pos), row in rc.collect(steps, out, cfg["vocab"]).items():
+            err = np.abs(row - reference[rid][pos]).max() / np.abs(reference[rid]).max()
+            assert err <= (TOLERANCE[dtype] if dtype == "float32" else 8e-2), f"{name}: {rid}@{pos}: {err:.3e}"
+
+
+def test_the_first_tokens_feel_what_the_denominator_holds():
+    """The plain statement itself: a request's first token keeps e^s / (e^s + e^sink) of its own value and nothing else."""
+    cfg = P.model_config([C(heads=1, kv_heads=1, dim=4, vdim=4, rot=rot(2, 10.0), softcap=3.0, scale=0.5)], vocab=5, width=8)
+    w = P.random_weights(cfg, 1, dtype=torch.float64)
+    h = torch.randn(1, 8, dtype=torch.float64, generator=torch.Generator().manual_seed(1))
+    p = "l0.mix."
+    q = P.norm(h @ w[p + "q"].T + w[p + "q.b"], w[p + "q.norm"], 1e-5)
+    k = P.norm(h @ w[p + "k"].T + w[p + "k.b"], w[p + "k.norm"], 1e-5)
+    s = 3.0 * math.tanh(float((q * k).sum()) * 0.5 / 3.0)
+    share = math.exp(s) / (math.exp(s) + math.exp(float(w[p + "sink"][0])))
+    want = share * (h @ w[p + "v"].T + w[p + "v.b"]) @ w[p + "o"].T
+    torch.testing.assert_close(P.attention_2(h, cfg["layers"][0]["mixer"], w, p, 1e-5), want)
+
+
+def test_each_mechanism_changes_the_logits():
+    """The plain statement itself: leaving a mechanism out moves the logits by far more than any tolerance
+    here, so a test that passes has seen it.  (Guards the tests, not the product.)"""
+    cfg = CONFIGS["all_kinds"]
+    weights = P.random_weights(cfg, 9, dtype=torch.float64)
+    tokens = rc.random_tokens(cfg["vocab"], 40, 3)
+    base = P.forward(cfg, weights, tokens)
+
+    def distance(logits):
+        return float((logits - base).abs().max() / base.abs().max())
+
+    def moved(config=None, **tensors):
+        other = dict(weights)
+        other.update(tensors)
+        return distance(P.forward(config or cfg, other, tokens))
+
+    def changed(change):
+        other = json.loads(json.dumps(cfg))
+        change(other)
+        return other
+
+    for mechanism in ("loop.step", "conv", "scaling", "sink", "g", "b", "qk_norm", "softcap", "retention.rot", "correction",
+                      "identity"):
+        assert distance(P.forward(cfg, weights, tokens, leave_out=(mechanism,))) > 1e-3, mechanism
+    ones = torch.ones_like
+    mixer = lambda c, i: c["layers"][i]["mixer"]
+    for name in ("l0.norm1", "l0.norm1b", "l0.norm2", "l0.norm2b", "l2.norm1b", "final.norm", "l0.mix.q.norm", "l0.mix.k.norm"):
+        assert moved(**{name: ones(weights[name])}) > 1e-3, name
+    assert moved(**{"l0.mix.sink": torch.zeros_like(weights["l0.mix.sink"])}) > 1e-3
+    for key, value in (("dims", 8), ("base", 400.0)):
+        for layer in (0, 1, 3):
+            assert moved(changed(lambda c: mixer(c, layer)["rot"].update({key: value - 4 * (key == "dims" and layer == 1)}))) > 1e-3
+    for key, value in (("factor", 2.0), ("low", 0.5), ("high", 6.0), ("original", 80)):
+        assert moved(changed(lambda c: mixer(c, 2)["rot"]["scaling"].update({key: value}))) > 1e-4, key
+    assert moved(changed(lambda c: mixer(c, 0).update(scale=0.5))) > 1e-3
+    assert moved(changed(lambda c: mixer(c, 0).update(softcap=3.0))) > 1e-3
+    assert moved(changed(lambda c: mixer(c, 1).update(decay=[0.6, 0.9, 0.95]))) > 1e-3
+    assert moved(changed(lambda c: c["loop"].update(times=1)), **{"loop.step": weights["loop.step"][:1]}) > 1e-3
+    assert moved(changed(lambda c: c["layers"][0]["mlp"]["router"].update(top=1))) > 1e-3
+    assert moved(changed(lambda c: c["embedding"].update(scale=0.8))) > 1e-3
+    assert moved(changed(lambda c: c["norm"].update(eps=1e-2))) > 1e-3
+
+
+# ---- configurations drawn at random ------------------------------------------------------------------------
+def drawn_config(seed):
+    """Another model of the design: sizes, head counts, order of layers, loop and constants all drawn."""
+    import random
+
+    rng = random.Random(seed)
+    fast = seed % 2 == 0                       # every other model has widths the tensor-core attention takes
+    width = rng.choice([32, 48, 64, 96] if fast else [24, 40, 56, 72])
+    layers = []
+    for _ in range(rng.randrange(2, 6)):
+        mlp = None
+        draw = rng.random()
+        if draw < 0.3:
+            mlp = P.dense(rng.choice([16, 64, 72] if fast else [6, 10, 33]))
+        elif draw < 0.85:
+            count, identity = rng.randrange(1, 10), rng.randrange(0, 4)
+            mlp = P.moe(experts=count, top=rng.randrange(1, min(count + identity, 5) + 1), identity=identity,
+                        ff=rng.choice([8, 16, 24] if fast else [6, 12, 20]))
+        dim = rng.choice([16, 32, 48] if fast else [6, 10, 20])
+        turn = rot(rng.choice([dim, dim // 2 // 2 * 2, 2]), rng.choice([10.0, 1000.0, 500000.0]),
+                   rng.choice([None, (8.0, 1.0, 4.0, 64), (2.0, 0.5, 2.0, 30)]))
+        heads = rng.choice([1, 2, 3])
+        vdim = rng.choice([8, 16, 40] if fast else [5, 7, 12])
+        kind = rng.choice("acr")
+        if kind == "r":
+            turn.pop("scaling", None)
+            layers.append(R(dim=dim, vdim=vdim, decay=[rng.choice([0.5, 0.9, 0.99, 0.999]) for _ in range(heads)], rot=turn, mlp=mlp))
+        elif kind == "a":
+            layers.append(A(heads=heads * rng.choice([1, 2, 4]), kv_heads=heads, dim=dim, vdim=vdim, conv=rng.choice([1, 2, 3, 4, 5, 10]),
+                            rot=turn, scale=rng.choice([None, 0.2, 0.5]), mlp=mlp))
+        else:
+            turn.pop("scaling", None)
+            layers.append(C(heads=heads * rng.choice([1, 2, 4]), kv_heads=heads, dim=dim, vdim=vdim, rot=turn,
+                            softcap=rng.choice([1.0, 5.0, 40.0]), scale=rng.choice([None, 0.2, 0.5]), mlp=mlp))
+    start = rng.randrange(0, len(layers))
+    loop = (start, rng.randrange(start + 1, len(layers) + 1), rng.choice([1, 2, 3])) if rng.random() < 0.8 else None
+    return P.model_config(layers, vocab=rng.randrange(40, 160), width=width, loop=loop, eps=rng.choice([1e-6, 1e-5]),
+                          scale=rng.choice([1.0, 0.3, 4.0]))
+
+
+@pytest.mark.parametrize("seed", range(8))
+def test_configurations_drawn_at_random(seed, device, tmp_path):
+    """Eight other models of the design through the framework: in 32-bit every position of every cutting against
+    the plain statement (and, on the GPU, bit-equal between cuttings); in bfloat16 the mixed cutting."""
+    cfg = drawn_config(seed)
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, seed=100 + seed)
+    requests = {f"d{i}": rc.random_tokens(cfg["vocab"], n, 500 + 10 * seed + i) for i, n in enumerate((1, 2, 47, 90, 33))}
+    reference, margins = references(cfg, weights, requests)
+    traces = {"whole": rc.trace_whole(requests), "tail": rc.trace_decode_tail(requests, tail=40),
+              "chunks": rc.trace_chunks(requests, sizes=(2, 13, 1, 5, 32, 3)),
+              "mixed": rc.trace_mixed(requests, max_live=3, seed=seed)}
+    if device == "cpu":        # the stand-in kernels are slow, and the other configurations run every cutting there
+        traces.pop("whole")
+        traces.pop("tail")
+    results = {}
+    for name, steps in traces.items():
+        out = tmp_path / name
+        rc.run_inprocess(folder, "float32", steps, out, rc.peak_tokens(steps), device=device,
+                         fill_freed_pages="poison" if name == "mixed" else None)
+        results[name] = rc.collect(steps, out, cfg["vocab"])
+        compare(results[name], reference, "float32")
+    if device != "cpu":
+        for name in ("tail", "chunks", "mixed"):
+            for key, row in results["whole"].items():
+                assert np.array_equal(row, results[name][key]), f"{name} differs from whole at {key}"
+        steps = traces["mixed"]
+        rc.run_inprocess(folder, "bfloat16", steps, tmp_path / "b", rc.peak_tokens(steps), device=device, fill_freed_pages="poison")
+        compare(rc.collect(steps, tmp_path / "b", cfg["vocab"]), reference, "bfloat16", margins)
+
+
+# ---- the entry point and the scheduler -------------------------------------------------------------------
+def plain_greedy(cfg, weights, prompt, steps):
+    tokens = list(prompt)
+    for _ in range(steps):
+        tokens.append(int(P.forward(cfg, weights, tokens)[-1].argmax()))
+    return tokens[len(prompt):]
+
+
+def generate(folder, prompts, new_tokens, device, *, block_size, pages, seqs, budget, prefix=False):
+    config = KVCoreConfig(
+        model_config=ModelConfig(model=str(folder), dtype="float32", max_model_len=128 if block_size == 16 else 64),
+        cache_config=CacheConfig(block_size=block_size, num_gpu_blocks=pages, enable_prefix_caching=prefix),
+        scheduler_config=SchedulerConfig(max_num_seqs=seqs, max_num_scheduled_tokens=budget,
+                                         max_num_partial_prefills=seqs, max_long_partial_prefills=seqs),
+        device_config=DeviceConfig(device=device),
+    )
+    engine = LLMEngine(config)
+    requests = [GenerationRequest(f"g{i}", SamplingParams(max_tokens=new_tokens, temperature=0.0), tuple(p))
+                for i, p in enumerate(prompts)]
+    outputs = [list(output.output_token_ids) for output in engine.generate(requests)]
+    return engine, outputs
+
+
+@pytest.mark.parametrize("name,budget", [("all_kinds", 16), ("coincide", 7)])
+def test_greedy_generation_through_the_entry_point(device, tmp_path, name, budget):
+    cfg = CONFIGS[name]
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, seed=21)
+    prompts = [rc.random_tokens(cfg["vocab"], n, 60 + i) for i, n in enumerate((5, 19, 33))]
+    engine, outputs = generate(folder, prompts, 12, device, block_size=16, pages=24, seqs=4, budget=budget)
+    for prompt, output in zip(prompts, outputs):
+        assert output == plain_greedy(cfg, weights, prompt, 12)
+    kv = engine.engine_core.model_runner.kv_manager
+    kv.check_invariants()
+    assert not kv.live_requests()
+
+
+def test_generation_with_few_pages_and_preemption(device, tmp_path):
+    """So few pages that a running request is preempted and computed again from its first token: its state rows must
+    read as new, not as what it left."""
+    cfg = CONFIGS["all_kinds"]
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, seed=22)
+    prompts = [rc.random_tokens(cfg["vocab"], n, 90 + i) for i, n in enumerate((30, 28, 26))]
+    _, outputs = generate(folder, prompts, 10, device, block_size=4, pages=30, seqs=3, budget=32)
+    for prompt, output in zip(prompts, outputs):
+        assert output == plain_greedy(cfg, weights, prompt, 10)
+
+
+@pytest.mark.parametrize("stateless", [True, False])
+def test_prefix_reuse_where_pages_hold_all_that_a_request_needs(stateless, device, tmp_path):
+    """A model of capped attentions alone keeps nothing but pages, also in every pass of a loop: a later prompt takes over
+    those of an equal beginning.  With a convolution it does not."""
+    layers = [C(heads=2, kv_heads=1, dim=8, vdim=12, rot=rot(4, 100.0), softcap=4.0, mlp=P.dense(20))]
+    if not stateless:
+        layers.append(A(heads=2, kv_heads=1, dim=8, vdim=12, conv=2, rot=rot(4, 100.0)))
+    cfg = P.model_config(layers, vocab=50, width=24, loop=(0, 1, 2))
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, seed=23)
+    prompt = rc.random_tokens(50, 40, 1)
+    engine, outputs = generate(folder, [prompt, prompt + [3]], 4, device, block_size=16, pages=24, seqs=1, budget=64, prefix=True)
+    kv = engine.engine_core.model_runner.kv_manager
+    assert kv.prefix_caching == stateless and (kv.num_prefix_hits > 0) == stateless
+    assert outputs == [plain_greedy(cfg, weights, prompt, 4), plain_greedy(cfg, weights, prompt + [3], 4)]
+
+
+# ---- the programs, each in a process of its own ------------------------------------------------------------
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_trace_program_on_a_tabopel_folder(case, dtype, tmp_path):
+    """``bin/trace_run`` as a user drives it: a step, its ``done`` line, the next step."""
+    if case["name"] != "serving_sizes":
+        pytest.skip("one configuration is enough for the subprocess run")
+    steps = rc.trace_mixed(case["requests"], max_live=3, seed=5)
+    steps.insert(1, {"step": 1000, "entries": [], "end": []})      # a step that brings nothing
+    out = tmp_path / "out"
+    rc.run_subprocess(case["folder"], dtype, steps, out, rc.peak_tokens(steps))
+    rows = rc.collect(steps, out, case["cfg"]["vocab"])
+    assert len(rows) == sum(len(t) for t in case["requests"].values())
+    compare(rows, case["reference"], dtype, case["margins"])
+
+
+@pytest.mark.gpu
+def test_offline_batch_program_on_a_tabopel_folder(tmp_path):
+    import ast
+    import re
+    import subprocess
+    import sys
+
+    cfg = CONFIGS["serving_sizes"]
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, seed=4)
+    prompts = {f"req-{i}": rc.random_tokens(cfg["vocab"], n, 80 + i) for i, n in enumerate((70, 9, 33))}
+    (tmp_path / "requests.json").write_text(json.dumps(
+        [dict(request_id=rid, prompt_token_ids=tokens) for rid, tokens in prompts.items()]))
+    command = [sys.executable, str(rc.ROOT / "bin" / "kvcore_offline_batch"), "--model", str(folder), "--dtype", "float32",
+               "--prompt-tokens-file", str(tmp_path / "requests.json"), "--max-tokens", "6", "--block-size", "16",
+               "--num-gpu-blocks", "64", "--max-model-len", "256", "--max-num-seqs", "4",
+               "--max-num-scheduled-tokens", "48", "--max-num-partial-prefills", "4", "--max-long-partial-prefills", "4",
+               "--log-level", "WARNING"]
+    result = subprocess.run(command, capture_output=True, text=True, timeout=300)
+    assert result.returncode == 0, result.stderr[-2000:]
+    found = {m["id"]: list(ast.literal_eval(m["ids"])) for m in re.finditer(
+        r"^\[(?P<id>[^\]]+)\] finish_reason=\S+\ntoken_ids=(?P<ids>\(.*\))$", result.stdout, re.M)}
+    assert list(found) == list(prompts)
+    for rid, prompt in prompts.items():
+        assert found[rid] == plain_greedy(cfg, weights, prompt, 6)
