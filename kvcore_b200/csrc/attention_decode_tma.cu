@@ -15,7 +15,7 @@
 // with mma.sync m16n8k16, keeps a running 32-bit softmax, and accumulates its part of the
 // output; after an item's last tile the warps merge through shared memory (where q lay) and write
 // either the final rows (one split) or a partial (max, sum, output) to scratch that a second kernel
-// merges over the splits.
+// merges over the splits.  Optional: a smooth cap on the scores, and a sink per query head in the denominator.
 //
 // Every wait on an mbarrier is bounded: when the bound is hit the thread sets the
 // WAIT_TIMEOUT bit of the status word, the block stops waiting, drains the copies it
@@ -45,6 +45,8 @@ struct DecodeParams {
   const int* query_start; const int* context_lens;
   int num_reqs, H, KVH, G, page_size, num_pages, window;
   float scale_log2;
+  float cap_in, cap_out;     // capped scores (kvb_capped_score): 2 log2(e) scale / cap and cap log2(e); cap_out 0: none
+  const float* sink;         // optional [H]: a logit per query head that joins the softmax's denominator
   int num_splits;
   float* partial_o;   // [reqs, KVH, splits, 16, D]
   float* partial_ml;  // [reqs, KVH, splits, 16, 2]
@@ -398,6 +400,11 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
       row_pos[hh] = context + (row_valid[hh] ? r / p.G : 0);
       row_max[hh] = -INFINITY;
       row_sum[hh] = 0.0f;
+      // the sink joins the denominator once: in the first split's first warp (a row's sum is spread over a quad)
+      if (p.sink != nullptr && split == 0 && warp == 0 && row_valid[hh]) {
+        row_max[hh] = p.sink[kvh * p.G + r % p.G] * 1.4426950408889634f;
+        row_sum[hh] = (lane & 3) == 0 ? 1.0f : 0.0f;
+      }
     }
 #pragma unroll
     for (int j = 0; j < DBLOCKS; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
@@ -460,7 +467,10 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
 #pragma unroll
       for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[j][e] += s2[j][e];
+        for (int e = 0; e < 4; ++e) {
+          s[j][e] += s2[j][e];
+          s[j][e] = p.cap_out > 0.0f ? kvb_capped_score(s[j][e] * p.cap_in, p.cap_out) : s[j][e] * p.scale_log2;
+        }
       float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
@@ -470,7 +480,7 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
           const int key = (tile_begin + it) * TD_KEYS + wkey + j * 8 + (lane & 3) * 2 + (e & 1);
           const bool seen = row_valid[hh] && key >= key_lo && key < key_hi && key <= row_pos[hh] &&
                             (p.window <= 0 || key > row_pos[hh] - p.window);
-          const float v = seen ? s[j][e] * p.scale_log2 : -INFINITY;
+          const float v = seen ? s[j][e] : -INFINITY;
           s[j][e] = v;
           tile_max[hh] = fmaxf(tile_max[hh], v);
         }
@@ -692,7 +702,7 @@ extern "C" int kvb_flash_decode_tma(void* out, long long out_stride, const void*
                                     int num_reqs, int max_query_len, int H, int KVH, int D, int page_size,
                                     int num_pages, float scale, int window, int num_splits, float* scratch,
                                     const float* cos_sin, void* k_cache, void* v_cache, int* work, int max_blocks,
-                                    float* lse, cudaStream_t stream) {
+                                    float* lse, const float* sink, float cap, cudaStream_t stream) {
   if (num_reqs == 0) return 0;
   KVB_REQUIRE(D == 64 || D == 128, "decode attention (TMA): head_dim must be 64 or 128");
   KVB_REQUIRE((k_cache == nullptr) == (v_cache == nullptr), "decode attention (TMA): give both caches or none");
@@ -714,6 +724,9 @@ extern "C" int kvb_flash_decode_tma(void* out, long long out_stride, const void*
   p.num_reqs = num_reqs; p.H = H; p.KVH = KVH; p.G = H / KVH;
   p.page_size = page_size; p.num_pages = num_pages; p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.cap_in = cap > 0.0f ? 2.0f * 1.4426950408889634f * scale / cap : 0.0f;
+  p.cap_out = cap > 0.0f ? cap * 1.4426950408889634f : 0.0f;
+  p.sink = sink;
   p.num_splits = num_splits < 1 ? 1 : num_splits;
   KVB_REQUIRE(p.num_splits == 1 || scratch != nullptr, "decode attention (TMA): splits need scratch memory");
   p.partial_o = scratch;

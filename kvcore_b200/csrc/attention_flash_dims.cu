@@ -73,15 +73,6 @@ __device__ __forceinline__ unsigned fd_pack(float lo, float hi) {
   return *reinterpret_cast<const unsigned*>(&v);
 }
 
-// cap_out * tanh(x) for y = 2 log2(e) x, by tanh(x) = 1 - 2 / (1 + exp(2 x)): two approximate instructions (base-2
-// exponential, reciprocal), within a few units of 1e-7 of cap_out; both ends saturate without a special case.
-__device__ __forceinline__ float fd_capped(float y, float cap_out) {
-  float e, r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(y));
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
-  return fmaf(-2.0f * cap_out, r, cap_out);
-}
-
 // Element offsets of every key row (and value row) of a tile inside the cache, or -1: zero-fill.
 template <int KEYS>
 __device__ __forceinline__ void fd_lookup_rows(long long* k_rows, long long* v_rows, const FlashDimsParams& p,
@@ -270,7 +261,7 @@ flash_dims_kernel(const FlashDimsParams p) {
 #pragma unroll
       for (int j = 0; j < NB; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[j][e] = fd_capped(s[j][e] * p.cap_in, p.cap_out);
+        for (int e = 0; e < 4; ++e) s[j][e] = kvb_capped_score(s[j][e] * p.cap_in, p.cap_out);
     }
     // mask and online softmax (base-2 exponent)
     float tile_max[2] = {-INFINITY, -INFINITY};

@@ -11,7 +11,9 @@
 //              128 columns), masks where the tile needs it, keeps a running maximum and sum in 32-bit,
 //              writes P = exp2(...) as packed bf16 over the columns it read S from (tcgen05.st: the
 //              A operand of the second product is read from tensor memory, so P never touches shared
-//              memory), and rescales its row of O when its maximum moved by more than 2^8.
+//              memory), and rescales its row of O when its maximum moved by more than 2^8.  Optional: a smooth
+//              cap on the scores (the raw scores are capped as they come), and a sink per query head that starts
+//              the running maximum and sum.
 //              The two warps of a scheduler belong to different query tiles: while one waits for
 //              tensor memory or for the tensor pipe, the other works.
 //   warps 8, 9 producers of K and of V (separate, so that a wait for a V stage never holds back
@@ -58,6 +60,8 @@ struct Tc5Params {
   const int* query_start; const int* context_lens;
   int num_reqs, H, KVH, G, page_size, num_pages, window;
   float scale_log2;
+  float cap_in, cap_out;     // CAP: 2 log2(e) scale / cap and cap log2(e)
+  const float* sink;         // optional [H]: a logit per query head that joins the softmax's denominator
   int* status;
   float* lse;                // optional [tokens, H]: log2 of the sum of 2^(scaled score) over the keys seen (-inf: none)
   int q_by_tma;                // the query tiles are brought by TMA (q_map is valid)
@@ -95,6 +99,27 @@ __device__ __forceinline__ void t5_add2(float& s0, float& s1, float a0, float a1
 #define T5_ROUND_SHIFT 0.0028150156f          // log2(1 + 2^-9)
 #define T5_ROUND_FACTOR 1.001953125f          // 1 + 2^-9
 
+// Scores bounded smoothly, cap_out * tanh(x) for y = 2 log2(e) x, as in kvb_capped_score, four at a time: the four
+// reciprocals are one reciprocal of the product and eight multiplications (the softmax of a capped tile is bound by the
+// unit that takes exponentials and reciprocals).  y is cut at 30, where 1 - 2 / (1 + 2^30) is 1 in 32-bit, so the product
+// stays below 2^121.
+__device__ __forceinline__ void t5_cap4(float& s0, float& s1, float& s2, float& s3, float cap_in, float cap_out) {
+  float a0, a1, a2, a3, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a0) : "f"(fminf(s0 * cap_in, 30.0f)));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a1) : "f"(fminf(s1 * cap_in, 30.0f)));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a2) : "f"(fminf(s2 * cap_in, 30.0f)));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a3) : "f"(fminf(s3 * cap_in, 30.0f)));
+  a0 += 1.0f; a1 += 1.0f; a2 += 1.0f; a3 += 1.0f;
+  const float low = a0 * a1, high = a2 * a3;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(low * high));
+  const float inv_low = r * high, inv_high = r * low, minus = -2.0f * cap_out;
+  s0 = fmaf(minus, inv_low * a1, cap_out);
+  s1 = fmaf(minus, inv_low * a0, cap_out);
+  s2 = fmaf(minus, inv_high * a3, cap_out);
+  s3 = fmaf(minus, inv_high * a2, cap_out);
+}
+
+template <bool CAP>
 __global__ void __launch_bounds__(T5_THREADS, 1)
 flash_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                          const __grid_constant__ CUtensorMap q_map, const Tc5Params p) {
@@ -370,6 +395,11 @@ flash_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __grid
     const unsigned s_addr = tmem_base + lane_addr + x * T5_BN;
     const unsigned o_addr = tmem_base + lane_addr + 256 + x * T5_D;
     float row_max = -INFINITY, row_sum = 0.0f;            // row_max in the scaled (log2) domain
+    if (p.sink != nullptr && row_valid) {                 // counts once, raised like the probabilities it stands beside
+      row_max = p.sink[kvh * p.G + flat % p.G] * 1.4426950408889634f;
+      row_sum = T5_ROUND_FACTOR;
+    }
+    const float scale_log2 = CAP ? 1.0f : p.scale_log2;   // capped scores are in the log2 domain already
     bool ok = true;
     for (int j = 0; j < n_mine; ++j) {
       if (!kvb_mbar_wait<T5_SPIN_LIMIT, 4096>(&s_full[x], j & 1)) { ok = false; break; }
@@ -380,6 +410,12 @@ flash_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __grid
 #pragma unroll
       for (int c = 0; c < 4; ++c) kvb_tc5_ld32(s_addr + c * 32, s[c]);
       kvb_tc5_wait_ld();
+      if (CAP) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) t5_cap4(s[c][i], s[c][i + 1], s[c][i + 2], s[c][i + 3], p.cap_in, p.cap_out);
+      }
       // ---- pass 1: maximum of the raw scores of the row ----
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
       if (need_mask) {
@@ -409,7 +445,7 @@ flash_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __grid
           for (int i = 0; i < 32; i += 2) mx[(i >> 1) & 3] = t5_max3(mx[(i >> 1) & 3], s[c][i], s[c][i + 1]);
         }
       }
-      const float tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.scale_log2;   // scale > 0; -inf stays -inf
+      const float tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale_log2;   // scale > 0; -inf stays -inf
       const float new_max = fmaxf(row_max, tile_max);
       const bool grows = new_max > row_max + 8.0f || (row_max == -INFINITY && new_max > -INFINITY);
       const bool move = __any_sync(0xffffffffu, grows);
@@ -429,7 +465,7 @@ flash_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __grid
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
           float a0, a1, e0, e1;
-          t5_fma2(a0, a1, s[c][i], s[c][i + 1], p.scale_log2, shift);      // masked entries stay -inf
+          t5_fma2(a0, a1, s[c][i], s[c][i + 1], scale_log2, shift);      // masked entries stay -inf
           asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e0) : "f"(a0));
           asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e1) : "f"(a1));
           t5_add2(sm[i & 2], sm[(i & 2) + 1], e0, e1);
@@ -535,7 +571,7 @@ extern "C" int kvb_flash_prefill_tc5(void* out, long long out_stride, const void
                                      int table_stride, const int* query_start, const int* context_lens,
                                      int num_reqs, int max_query_len, int num_tokens, int H, int KVH, int D,
                                      int page_size, int num_pages, float scale, int window, float* lse,
-                                     cudaStream_t stream) {
+                                     const float* sink, float cap, cudaStream_t stream) {
   if (num_reqs == 0) return 0;
   KVB_REQUIRE(D == T5_D, "prefill attention (tcgen05): head_dim must be 128");
   KVB_REQUIRE(page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64,
@@ -553,6 +589,9 @@ extern "C" int kvb_flash_prefill_tc5(void* out, long long out_stride, const void
   p.num_reqs = num_reqs; p.H = H; p.KVH = KVH; p.G = H / KVH;
   p.page_size = page_size; p.num_pages = num_pages; p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.cap_in = cap > 0.0f ? 2.0f * 1.4426950408889634f * scale / cap : 0.0f;
+  p.cap_out = cap > 0.0f ? cap * 1.4426950408889634f : 0.0f;
+  p.sink = sink;
   p.status = kvb_status_word();
   p.lse = lse;
   KVB_REQUIRE(p.status != nullptr, "prefill attention (tcgen05): no status word");
@@ -580,14 +619,18 @@ extern "C" int kvb_flash_prefill_tc5(void* out, long long out_stride, const void
   constexpr size_t SMEM = 6 * T5_TILE_BYTES + 16 * 8;
   static bool configured = false;
   if (!configured) {
-    KVB_CHECK_CUDA(cudaFuncSetAttribute(flash_prefill_tc5_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM));
+    KVB_CHECK_CUDA(cudaFuncSetAttribute(flash_prefill_tc5_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM));
+    KVB_CHECK_CUDA(cudaFuncSetAttribute(flash_prefill_tc5_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM));
     configured = true;
   }
   const int max_rows = max_query_len * p.G;
   const int pairs = (max_rows + 2 * T5_BM - 1) / (2 * T5_BM);            // a block takes two query tiles
   KVB_REQUIRE(pairs <= 65535, "prefill attention (tcgen05): portion too long for one launch");
   dim3 grid(KVH, num_reqs, pairs);
-  KVB_CHECK_CUDA(kvb_launch((flash_prefill_tc5_kernel), dim3(grid), dim3(T5_THREADS), SMEM, stream, true, k_map, v_map, q_map, p));
+  if (cap > 0.0f)
+    KVB_CHECK_CUDA(kvb_launch((flash_prefill_tc5_kernel<true>), dim3(grid), dim3(T5_THREADS), SMEM, stream, true, k_map, v_map, q_map, p));
+  else
+    KVB_CHECK_CUDA(kvb_launch((flash_prefill_tc5_kernel<false>), dim3(grid), dim3(T5_THREADS), SMEM, stream, true, k_map, v_map, q_map, p));
   KVB_CHECK_LAUNCH();
   return 0;
 }

@@ -1,4 +1,5 @@
-// Between the projections and the attention of a mixer that caches one row [k of all heads | v of all heads] a token.
+// Between the projections and the attention of a mixer that caches keys and values, addressed by strides: side by side in
+// one row a token, or in two tensors [pages, heads, page, width].
 //
 //   attention_prepare: q [H, D], k [G, D] and v of a token's projected row, in this order, each step where asked for:
 //     a causal convolution over time per channel of q, k and v (taps [K, channels], the last tap on the current token,
@@ -63,8 +64,11 @@ struct AttentionPrepareParams {
   const float2* cos_sin; int rot;                    // [T, rot / 2]
   const int* positions; const int* req_index; const int* query_start; const int* state_slots;
   const int* table; int table_stride;
-  void* cache; int page_size, num_pages, write;
-  int tokens, H, G, D, v_width;
+  // where head g of the token in slot s of page n keeps its key: k_cache + n * k_page + g * k_head + s * k_row; values alike
+  void* k_cache; long long k_page, k_head, k_row;
+  void* v_cache; long long v_page, v_head, v_row;
+  int page_size, num_pages, write;
+  int tokens, H, G, D, V, v_width;                   // v_width = G * V
   const void* taps; int num_taps;                    // 0: no convolution
   float* state; long long state_stride, state_offset;
   int single;                                        // one token a request: the kept inputs are moved on here
@@ -85,13 +89,15 @@ attention_prepare_kernel(const AttentionPrepareParams p) {
     const int t = blockIdx.x;
     const T* row = (const T*)p.rows + (size_t)t * p.row_stride;
     const int pos = p.positions[t], req = p.req_index[t];
-    T* dst = nullptr;
+    T* k_dst = nullptr;                              // the token's place among the keys and among the values
+    T* v_dst = nullptr;
     if (p.write) {
       const int page = p.table[(size_t)req * p.table_stride + pos / p.page_size];
       if (page <= 0 || page >= p.num_pages) {
         if (threadIdx.x == 0) atomicOr(p.status, KVB_STATUS_BAD_PAGE);
       } else {
-        dst = (T*)p.cache + ((size_t)page * p.page_size + pos % p.page_size) * ((size_t)k_len + p.v_width);
+        k_dst = (T*)p.k_cache + (size_t)page * p.k_page + (size_t)(pos % p.page_size) * p.k_row;
+        v_dst = (T*)p.v_cache + (size_t)page * p.v_page + (size_t)(pos % p.page_size) * p.v_row;
       }
     }
     int back = 0;
@@ -190,7 +196,8 @@ attention_prepare_kernel(const AttentionPrepareParams p) {
           b[j] = w0 * cs.v[j].x + u0 * cs.v[j].y;
         }
       }
-      T* to = is_q ? (T*)p.q_out + (size_t)t * p.q_stride + at : dst == nullptr ? nullptr : dst + at;
+      T* to = is_q ? (T*)p.q_out + (size_t)t * p.q_stride + at
+                   : k_dst == nullptr ? nullptr : k_dst + (size_t)(head - p.H) * p.k_head + i;
       if (to == nullptr) return;
       store(to, a);
       if (mate) store(to + mate, b);
@@ -204,9 +211,10 @@ attention_prepare_kernel(const AttentionPrepareParams p) {
       float av[N], bv[N];
       fetch(q_len + k_len + i, av, true);
       if (cut.v_mate) fetch(q_len + k_len + i + cut.v_mate, bv, true);
-      if (dst == nullptr) return;
-      store(dst + k_len + i, av);
-      if (cut.v_mate) store(dst + k_len + i + cut.v_mate, bv);
+      if (v_dst == nullptr) return;
+      auto at = [&](int e) { return v_dst + (size_t)(e / p.V) * p.v_head + e % p.V; };
+      store(at(i), av);
+      if (cut.v_mate) store(at(i + cut.v_mate), bv);
     };
     float a[N], b[N];                                // this thread's first unit stays in registers
     ApPiece<T, N> w, w2;                             // (its weights are on their way before anybody waits for a sum)
@@ -254,6 +262,8 @@ attention_prepare_kernel(const AttentionPrepareParams p) {
   }
 }
 
+__device__ __forceinline__ int ap_kind(int u, int qk_units, int q_units) { return u < q_units ? 0 : u < qk_units ? 1 : 2; }
+
 // Without a norm.  A thread owns a unit for `run` tokens; K: taps the window is made for (the model's taps, right-aligned;
 // the places in front are zero), 1 also where nothing is convolved.
 template <typename T, int N, int K>
@@ -261,7 +271,7 @@ __global__ void __launch_bounds__(AP_RUN_THREADS, K <= 4 ? 4 : 2)
 attention_prepare_runs_kernel(const AttentionPrepareParams p) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_ATTN_PREPARE);
   extern __shared__ __align__(16) float2 run_cs[];   // [run][rot / 2]
-  __shared__ long long place_of[AP_RUN];             // where a token's cached row begins, or -1
+  __shared__ long long place_of[2][AP_RUN];          // where a token's key and its value begin, or -1
   const int q_len = p.H * p.D, k_len = p.G * p.D, channels = q_len + k_len + p.v_width, keep = p.num_taps - 1;
   const ApUnits<N> cut(p.D, p.rot, p.write ? p.H + p.G : p.H, p.v_width, p.write);
   const int half = cut.half;
@@ -273,20 +283,30 @@ attention_prepare_runs_kernel(const AttentionPrepareParams p) {
     const int page = p.table[(size_t)p.req_index[t] * p.table_stride + pos / p.page_size];
     const bool fine = page > 0 && page < p.num_pages;
     if (!fine && blockIdx.x == 0) atomicOr(p.status, KVB_STATUS_BAD_PAGE);
-    place_of[threadIdx.x] = fine ? ((long long)page * p.page_size + pos % p.page_size) * (k_len + p.v_width) : -1;
+    place_of[0][threadIdx.x] = fine ? page * p.k_page + pos % p.page_size * p.k_row : -1;
+    place_of[1][threadIdx.x] = fine ? page * p.v_page + pos % p.page_size * p.v_row : -1;
   }
   __syncthreads();
   const int u = blockIdx.x * AP_RUN_THREADS + threadIdx.x;
   if (u >= cut.units) return;
   int c, i = 0, mate;                                // first channel, its place in its head, where its second piece lies
   bool turns = false;
-  if (u < cut.qk_units) {
+  const int kind = ap_kind(u, cut.qk_units, p.H * cut.per_head);      // 0 a query, 1 a key, 2 values
+  long long inside[2] = {0, 0};                      // a key's or value's pieces behind the token's place
+  if (kind < 2) {
     int head;
     cut.locate(u, head, i, mate, turns);
     c = head * p.D + i;
+    if (kind == 1) {
+      inside[0] = (head - p.H) * p.k_head + i;
+      inside[1] = inside[0] + mate;
+    }
   } else {
-    c = q_len + k_len + (u - cut.qk_units) * N;
+    const int e = (u - cut.qk_units) * N;
+    c = q_len + k_len + e;
     mate = cut.v_mate;
+    inside[0] = e / p.V * p.v_head + e % p.V;
+    inside[1] = (e + mate) / p.V * p.v_head + (e + mate) % p.V;
   }
   ApPiece<T, N> taps[2][K];
   if (p.num_taps > 0) {
@@ -386,13 +406,16 @@ attention_prepare_runs_kernel(const AttentionPrepareParams p) {
           y[1][n] = w0 * cs.v[n].x + u0 * cs.v[n].y;
         }
       }
-      T* to;
-      if (c < q_len) {
-        to = (T*)p.q_out + (size_t)t * p.q_stride + c;
+      T* to[2];
+      if (kind == 0) {
+        to[0] = (T*)p.q_out + (size_t)t * p.q_stride + c;
+        to[1] = to[0] + mate;
       } else {
-        const long long place = place_of[t - t_begin];
+        const long long place = place_of[kind - 1][t - t_begin];
         if (place < 0) continue;
-        to = (T*)p.cache + place + (c - q_len);
+        T* at = (T*)(kind == 1 ? p.k_cache : p.v_cache) + place;
+        to[0] = at + inside[0];
+        to[1] = at + inside[1];
       }
 #pragma unroll
       for (int side = 0; side < 2; ++side) {
@@ -400,7 +423,7 @@ attention_prepare_runs_kernel(const AttentionPrepareParams p) {
         ApPiece<T, N> r;
 #pragma unroll
         for (int n = 0; n < N; ++n) r.v[n] = from_float<T>(y[side][n]);
-        *reinterpret_cast<ApPiece<T, N>*>(to + side * mate) = r;
+        *reinterpret_cast<ApPiece<T, N>*>(to[side]) = r;
       }
     }
   }
@@ -439,14 +462,16 @@ static cudaError_t launch_attention_prepare(AttentionPrepareParams& p, bool norm
 extern "C" int kvb_attention_prepare(const void* rows, long long row_stride, void* q_out, long long q_stride,
                                      const float* cos_sin, int rot, const int* positions, const int* req_index,
                                      const int* query_start, const int* state_slots, const int* table, int table_stride,
-                                     void* cache, int page_size, int num_pages, int write, int tokens, int num_reqs,
-                                     int H, int G, int D, int v_width, const void* taps, int num_taps, float* state,
+                                     void* k_cache, long long k_page, long long k_head, long long k_row, void* v_cache,
+                                     long long v_page, long long v_head, long long v_row, int page_size, int num_pages,
+                                     int write, int tokens, int num_reqs, int H, int G, int D, int V, const void* taps, int num_taps, float* state,
                                      long long state_stride, long long state_offset, const void* q_weight,
                                      const void* k_weight, float eps, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (cos_sin == nullptr) rot = 0;
   if (taps == nullptr) num_taps = 0;
-  KVB_REQUIRE(H > 0 && G > 0 && D > 0 && v_width > 0, "attention_prepare: bad sizes");
+  KVB_REQUIRE(H > 0 && G > 0 && D > 0 && V > 0, "attention_prepare: bad sizes");
+  const int v_width = G * V;
   KVB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= D, "attention_prepare: the turned entries are an even number within the head");
   KVB_REQUIRE((tokens + 3) / 4 <= 65535 || tokens == num_reqs, "attention_prepare: too many tokens for one launch");
   KVB_REQUIRE((long long)rot / 2 * 8 <= 40 * 1024, "attention_prepare: too many turned entries");
@@ -458,7 +483,9 @@ extern "C" int kvb_attention_prepare(const void* rows, long long row_stride, voi
   p.rows = rows; p.row_stride = row_stride; p.q_out = q_out; p.q_stride = q_stride;
   p.cos_sin = (const float2*)cos_sin; p.rot = rot; p.positions = positions; p.req_index = req_index;
   p.query_start = query_start; p.state_slots = state_slots; p.table = table; p.table_stride = table_stride;
-  p.cache = cache; p.page_size = page_size; p.num_pages = num_pages; p.write = write; p.tokens = tokens;
+  p.k_cache = k_cache; p.k_page = k_page; p.k_head = k_head; p.k_row = k_row;
+  p.v_cache = v_cache; p.v_page = v_page; p.v_head = v_head; p.v_row = v_row; p.V = V;
+  p.page_size = page_size; p.num_pages = num_pages; p.write = write; p.tokens = tokens;
   p.H = H; p.G = G; p.D = D; p.v_width = v_width; p.taps = taps; p.num_taps = num_taps; p.state = state;
   p.state_stride = state_stride; p.state_offset = state_offset; p.single = tokens == num_reqs;
   p.q_weight = q_weight; p.k_weight = k_weight; p.eps = eps; p.run = 1;
@@ -467,7 +494,9 @@ extern "C" int kvb_attention_prepare(const void* rows, long long row_stride, voi
   // entries a piece: 16 bytes where a block owns a token and nothing is convolved, else 4 entries
   const int n = q_weight != nullptr && num_taps == 0 && dtype != KVB_F32 ? 8 : 4;
   const bool vec = (rot / 2) % n == 0 && D % n == 0 && v_width % n == 0 && row_stride % n == 0 && q_stride % n == 0 &&
-                   aligned16(rows) && aligned16(q_out) && aligned16(cos_sin) && aligned16(cache) && aligned16(taps) &&
+                   (v_head == V || V % n == 0) && (k_page | k_head | k_row | v_page | v_head | v_row) % n == 0 &&
+                   aligned16(rows) && aligned16(q_out) && aligned16(cos_sin) && aligned16(k_cache) &&
+                   (uintptr_t)v_cache % (n * (dtype == KVB_F32 ? 4 : 2)) == 0 && aligned16(taps) &&
                    aligned16(q_weight) && aligned16(k_weight);
   cudaError_t err;
   const bool norm = q_weight != nullptr;

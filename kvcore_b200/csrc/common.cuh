@@ -233,6 +233,16 @@ struct Vec16 {
 // The 32-bit path uses the exact form.
 __device__ __forceinline__ float kvb_silu_for_bf16(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 
+// A smoothly bounded attention score in units of the base-2 exponent, cap_out * tanh(x) for y = 2 log2(e) x, by
+// tanh(x) = 1 - 2 / (1 + exp(2 x)): two approximate instructions (base-2 exponential, reciprocal), within a few units
+// of 1e-7 of cap_out; both ends saturate without a special case.
+__device__ __forceinline__ float kvb_capped_score(float y, float cap_out) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(y));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return fmaf(-2.0f * cap_out, r, cap_out);
+}
+
 __host__ __device__ __forceinline__ bool aligned16(const void* p) {
   return (reinterpret_cast<uintptr_t>(p) & 15) == 0;
 }

@@ -67,10 +67,10 @@ def ensure_built(verbose: bool = False) -> str:
                                  _int, _int, _float, _int, _int, _int, _vp],
         "kvb_make_kv_tensor_map": [_vp, _vp, _ll, _int, _int, _int],
         "kvb_flash_decode_tma": [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _int, _vp, _vp, _int, _int, _int, _int,
-                                 _int, _int, _int, _float, _int, _int, _vp, _vp, _vp, _vp, _vp, _int, _vp, _vp],
+                                 _int, _int, _int, _float, _int, _int, _vp, _vp, _vp, _vp, _vp, _int, _vp, _vp, _float, _vp],
         "kvb_make_kv_half_tensor_map": [_vp, _vp, _ll, _int, _int, _int],
         "kvb_flash_prefill_tc5": [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _int, _vp, _vp, _int, _int, _int, _int, _int,
-                                  _int, _int, _int, _float, _int, _vp, _vp],
+                                  _int, _int, _int, _float, _int, _vp, _vp, _float, _vp],
         "kvb_gemm_f32": [_vp, _vp, _vp, _vp, _int, _int, _int, _ll, _ll, _vp],
         "kvb_rms_norm_shift": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _int, _int, _float, _int, _int, _int, _vp],
         "kvb_stream_add_norm": [_vp, _vp, _vp, _vp, _int, _int, _float, _vp, _vp, _ll, _vp, _int, _vp, _int, _int, _vp],
@@ -104,8 +104,8 @@ def ensure_built(verbose: bool = False) -> str:
         "kvb_gated_group_norm": [_vp, _ll, _vp, _vp, _ll, _vp, _int, _int, _int, _float, _int, _vp],
         "kvb_stream_add_rows": [_vp, _vp, _int, _vp, _vp, _int, _vp, _int, _vp, _vp, _vp, _float, _vp, _vp, _vp, _float, _vp,
                                 _vp, _int, _vp, _vp, _int, _int, _int, _int, _vp],
-        "kvb_attention_prepare": [_vp, _ll, _vp, _ll, _vp, _int, _vp, _vp, _vp, _vp, _vp, _int, _vp, _int, _int, _int, _int,
-                                  _int, _int, _int, _int, _int, _vp, _int, _vp, _ll, _ll, _vp, _vp, _float, _int, _vp],
+        "kvb_attention_prepare": [_vp, _ll, _vp, _ll, _vp, _int, _vp, _vp, _vp, _vp, _vp, _int, _vp, _ll, _ll, _ll, _vp, _ll,
+                                  _ll, _ll, _int, _int, _int, _int, _int, _int, _int, _int, _int, _vp, _int, _vp, _ll, _ll, _vp, _vp, _float, _int, _vp],
         "kvb_retention_scan": [_vp, _vp, _vp, _vp, _vp, _ll, _vp, _int, _vp, _vp, _ll, _ll, _vp, _vp, _int, _int, _int, _int,
                                _int, _float, _int, _vp],
         "kvb_relu_squared": [_vp, _ll, _int, _vp],
@@ -504,6 +504,12 @@ def tc5_prefill_supported(dtype: torch.dtype, head_dim: int, page_size: int) -> 
     return dtype == torch.bfloat16 and head_dim == 128 and page_size in (8, 16, 32, 64)
 
 
+def paged_attention_takes_sinks(dtype: torch.dtype, head_dim: int, page_size: int) -> bool:
+    """Whether ``paged_attention`` takes sinks and capped scores on such a cache: where its decode batches go to the TMA
+    kernel and its prompts to the tcgen05 kernel."""
+    return tma_decode_supported(dtype, head_dim, page_size) and tc5_prefill_supported(dtype, head_dim, page_size)
+
+
 def paged_attention(
     qkv: torch.Tensor,
     k_cache: torch.Tensor,
@@ -523,6 +529,9 @@ def paged_attention(
     cos_sin: torch.Tensor | None = None,
     write_kv: bool | None = None,
     keep_first: int = 0,
+    sink: torch.Tensor | None = None,
+    softcap: float | None = None,
+    out: torch.Tensor | None = None,
 ) -> torch.Tensor:
     """Attention of the step's queries (the first ``H*D`` columns of ``qkv``) over the cache.
 
@@ -536,7 +545,22 @@ def paged_attention(
     ``cos_sin`` (``None``: no rotation) and, if ``write_kv``, writes this step's k and v into
     their pages: inside the decode kernel where that one runs (``qkv`` is then left as it
     was), through ``rope_kv_write`` in front of the other kernels.
+
+    ``sink [H]`` (32-bit): a logit per query head that joins the softmax's denominator.  ``softcap``: the scaled scores
+    become ``softcap * tanh(score / softcap)``.  Both only where ``paged_attention_takes_sinks`` says so.  ``out``: a
+    ``[T, H*D]`` tensor to fill.
     """
+    if sink is not None or softcap is not None:
+        if keep_first or window or not paged_attention_takes_sinks(qkv.dtype, head_dim, k_cache.shape[2]) or force_general:
+            raise KernelError("paged_attention: sinks and capped scores are for the TMA decode and the tcgen05 kernel")
+        if sink is not None:
+            _check(sink, "sink", dtype=torch.float32)
+            if sink.numel() != num_heads:
+                raise KernelError(f"paged_attention: {sink.numel()} sinks for {num_heads} query heads")
+        if softcap is not None and not softcap > 0:
+            raise KernelError(f"paged_attention: the scores' cap must be positive, got {softcap}")
+        if qkv.stride(0) % 8 or not (use_tma and use_tc5):
+            raise KernelError("paged_attention: sinks and capped scores need rows on 16-byte boundaries")
     if write_kv is not None:
         group = num_heads // num_kv_heads
         fused = (not force_general and not keep_first and use_tma and flash_attention_supported(qkv.dtype, head_dim)
@@ -561,7 +585,12 @@ def paged_attention(
         raise KernelError(f"cache shape {tuple(k_cache.shape)} does not match the head layout")
     if keep_first < 0 or (keep_first and not window):
         raise KernelError(f"kept first positions ({keep_first}) need a window")
-    out = torch.empty((tokens, num_heads * head_dim), dtype=qkv.dtype, device=qkv.device)
+    if out is None:
+        out = torch.empty((tokens, num_heads * head_dim), dtype=qkv.dtype, device=qkv.device)
+    _check(out, "out", dtype=qkv.dtype, contiguous=False)
+    if tuple(out.shape) != (tokens, num_heads * head_dim) or (tokens and (out.stride(1) != 1 or out.stride(0) % 8)):
+        raise KernelError(f"paged_attention: out {tuple(out.shape)} does not fit {tokens} tokens of {num_heads} heads")
+    bounded = (sink, softcap)
     if not force_general and flash_attention_supported(qkv.dtype, head_dim) and qkv.stride(0) % 8 == 0:
         group = num_heads // num_kv_heads
         geometry = (num_heads, num_kv_heads, head_dim, float(scale), int(window or 0))
@@ -591,11 +620,11 @@ def paged_attention(
                 for begin, end in ((0, long_count), (long_count, ctx.num_reqs)):
                     part = _RequestRun(ctx, begin, end)
                     _flash_attention_into(out, qkv, k_cache, v_cache, table[begin:end], part, geometry,
-                                          None, use_tma, use_tc5, None, None, lse)
+                                          None, use_tma, use_tc5, None, None, lse, *bounded)
                 add_kept_first()
                 return out
         _flash_attention_into(out, qkv, k_cache, v_cache, table, ctx, geometry, num_splits, use_tma, use_tc5,
-                              cos_sin, write_kv, lse)
+                              cos_sin, write_kv, lse, *bounded)
         add_kept_first()
         return out
     _call("kvb_paged_attention_rows", out.data_ptr(), out.stride(0), qkv.data_ptr(), qkv.stride(0),
@@ -623,7 +652,7 @@ class _RequestRun:
 
 
 def _flash_attention_into(out, qkv, k_cache, v_cache, table, ctx, geometry, num_splits, use_tma, use_tc5,
-                          cos_sin, write_kv, lse=None) -> None:
+                          cos_sin, write_kv, lse=None, sink=None, softcap=None) -> None:
     """The tensor-core attention kernels on one batch (or one run of requests of a batch): the TMA
     decode kernel for at most 16 rows a kv head, the tcgen05 kernel for portions of prompts, the
     ``mma.sync`` kernel for the shapes those two do not take."""
@@ -649,7 +678,8 @@ def _flash_attention_into(out, qkv, k_cache, v_cache, table, ctx, geometry, num_
               None if cos_sin is None else cos_sin.data_ptr(),
               k_cache.data_ptr() if write_kv else None, v_cache.data_ptr() if write_kv else None,
               _decode_work(qkv.device).data_ptr() if TMA_DECODE_SHARED_WORK else None,
-              sms * TMA_DECODE_BLOCKS_PER_SM, lse_ptr, _stream(),
+              sms * TMA_DECODE_BLOCKS_PER_SM, lse_ptr, None if sink is None else sink.data_ptr(), float(softcap or 0.0),
+              _stream(),
               kernels=2 if splits > 1 else 1)   # the splits are merged by a second kernel
         return
     if (not split_mode and use_tc5 and tc5_prefill_supported(qkv.dtype, head_dim, page_size)
@@ -659,7 +689,7 @@ def _flash_attention_into(out, qkv, k_cache, v_cache, table, ctx, geometry, num_
               ctypes.addressof(k_map), ctypes.addressof(v_map), table.data_ptr(), table.stride(0),
               ctx.query_start.data_ptr(), ctx.context_lens.data_ptr(), ctx.num_reqs, ctx.max_query_len,
               qkv.shape[0], num_heads, num_kv_heads, head_dim, page_size, num_pages, scale, window,
-              lse_ptr, _stream())
+              lse_ptr, None if sink is None else sink.data_ptr(), float(softcap or 0.0), _stream())
         return
     splits = 1
     if split_mode:
@@ -1789,7 +1819,7 @@ def _turned_entries(cos_sin: torch.Tensor | None, tokens: int, dim: int, who: st
 
 
 def attention_prepare(rows: torch.Tensor, q_out: torch.Tensor, cos_sin: torch.Tensor | None, ctx, table: torch.Tensor,
-                      cache: torch.Tensor, *, q_heads: int, k_heads: int, dim: int, value_width: int,
+                      cache, *, q_heads: int, k_heads: int, dim: int, value_width: int,
                       taps: torch.Tensor | None = None, state: torch.Tensor | None = None, state_offset: int = 0,
                       q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None, eps: float = 0.0,
                       write: bool = True) -> None:
@@ -1800,10 +1830,10 @@ def attention_prepare(rows: torch.Tensor, q_out: torch.Tensor, cos_sin: torch.Te
     ``k_weight``, one RMS norm over all of q and one over all of k; ``cos_sin [T, rot / 2, 2]``, a turn of the first
     ``rot`` entries of every q and k head in halves.  q goes to ``q_out [T, q_heads * dim]`` (a view; without taps it may
     be q's own columns); with ``write`` k and v go side by side into the token's row of
-    ``cache [pages, 1, page, k_heads * dim + value_width]``."""
+    ``cache [pages, 1, page, k_heads * dim + value_width]``, or, for ``cache = (keys, values)``, into the token's places
+    of ``keys [pages, k_heads, page, dim]`` and ``values [pages, k_heads, page, value_width / k_heads]``."""
     _check(rows, "rows", contiguous=False)
     _check(q_out, "q_out", dtype=rows.dtype, contiguous=False)
-    _check(cache, "cache", dtype=rows.dtype)
     _check(table, "block table", dtype=torch.int32, contiguous=False)
     tokens = rows.shape[0]
     q_len, k_len = q_heads * dim, k_heads * dim
@@ -1811,9 +1841,25 @@ def attention_prepare(rows: torch.Tensor, q_out: torch.Tensor, cos_sin: torch.Te
     if rows.shape[1] < channels or tuple(q_out.shape) != (tokens, q_len) or (tokens and (rows.stride(1) != 1 or q_out.stride(1) != 1)):
         raise KernelError(f"attention_prepare: rows {tuple(rows.shape)} / q_out {tuple(q_out.shape)} do not hold the heads")
     rot = _turned_entries(cos_sin, tokens, dim, "attention_prepare")
-    num_pages, one, page_size, width = cache.shape
-    if one != 1 or width != k_len + value_width or table.stride(1) != 1:
-        raise KernelError(f"attention_prepare: cache {tuple(cache.shape)} does not hold rows of {k_len} + {value_width}")
+    if value_width % k_heads or table.stride(1) != 1:
+        raise KernelError(f"attention_prepare: {value_width} value entries do not fall into {k_heads} heads")
+    vdim = value_width // k_heads
+    if isinstance(cache, tuple):
+        keys, values = cache
+        _check(keys, "keys", dtype=rows.dtype)
+        _check(values, "values", dtype=rows.dtype)
+        num_pages, _, page_size, _ = keys.shape
+        if tuple(keys.shape[1:]) != (k_heads, page_size, dim) or tuple(values.shape) != (num_pages, k_heads, page_size, vdim):
+            raise KernelError(f"attention_prepare: keys {tuple(keys.shape)} / values {tuple(values.shape)} do not fit the heads")
+        places = (keys.data_ptr(), k_heads * page_size * dim, page_size * dim, dim,
+                  values.data_ptr(), k_heads * page_size * vdim, page_size * vdim, vdim)
+    else:
+        _check(cache, "cache", dtype=rows.dtype)
+        num_pages, one, page_size, width = cache.shape
+        if one != 1 or width != k_len + value_width:
+            raise KernelError(f"attention_prepare: cache {tuple(cache.shape)} does not hold rows of {k_len} + {value_width}")
+        places = (cache.data_ptr(), page_size * width, dim, width,
+                  cache.data_ptr() + k_len * cache.element_size(), page_size * width, vdim, width)
     kept = (None, 0, None, 0, 0)
     if taps is not None:
         _check(taps, "taps", dtype=rows.dtype)
@@ -1834,8 +1880,8 @@ def attention_prepare(rows: torch.Tensor, q_out: torch.Tensor, cos_sin: torch.Te
     _call("kvb_attention_prepare", rows.data_ptr(), rows.stride(0), q_out.data_ptr(), q_out.stride(0),
           None if cos_sin is None else cos_sin.data_ptr(), rot, ctx.positions.data_ptr(), ctx.req_index.data_ptr(),
           ctx.query_start.data_ptr(), None if slots is None else slots.data_ptr(), table.data_ptr(), table.stride(0),
-          cache.data_ptr(), page_size, num_pages, int(bool(write)), tokens, ctx.num_reqs, q_heads, k_heads, dim,
-          value_width, *kept, None if q_weight is None else q_weight.data_ptr(),
+          *places, page_size, num_pages, int(bool(write)), tokens, ctx.num_reqs, q_heads, k_heads, dim,
+          vdim, *kept, None if q_weight is None else q_weight.data_ptr(),
           None if k_weight is None else k_weight.data_ptr(), float(eps), _dtype_code(rows), _stream(),
           kernels=2 if kept[2] is not None and tokens != ctx.num_reqs else 1)
 

@@ -9,7 +9,9 @@
              "one": 1; "learned": exp of one number a head
     o = sum of weights times values, times sigmoid(W_g x)               (``gate``: entry by entry)
 
-A token's keys and values are one cached row ``[k of all kv heads | v of all kv heads]``.  With a convolution the last
+A token's keys and values are one cached row ``[k of all kv heads | v of all kv heads]``; where both widths are the one
+that the TMA decode and the tcgen05 prompt kernels are made for (bfloat16), they are the two planes of those kernels
+instead (``CacheSpec.keys_and_values``).  With a convolution the last
 ``conv_taps - 1`` projected q, k and v of a request are per-request state (``[taps - 1, channels]``, 32-bit, oldest
 first).  Scores, softmax, angles, norms and the convolution's sums are 32-bit whatever the activation type.
 """
@@ -76,7 +78,13 @@ class GroupedAttention(ProjectedMixer):
     def graph_safe(self) -> bool:
         return self.position is None or self.position.graph_safe
 
+    # the page sizes of a cache do not count here: with one that those kernels do not take the planes are read by strides
+    def _two_planes(self) -> bool:
+        return self.head_dim == self.value_dim and K.paged_attention_takes_sinks(self.dtype, self.head_dim, 16)
+
     def cache_spec(self) -> CacheSpec:
+        if self._two_planes():
+            return CacheSpec.keys_and_values(self.num_kv_heads, self.head_dim)
         return CacheSpec(1, 1, self.k_cols + self.v_cols)
 
     def state_spec(self) -> StateSpec | None:
@@ -115,8 +123,6 @@ class GroupedAttention(ProjectedMixer):
             raise ValueError(f"{self.name}: grouped attention writes its output without a factor")
         tokens, heads = rows.shape[0], self.num_heads
         table = ctx.block_table(cache.group)
-        plane = cache.planes[0]                                # [pages, 1, page, k_cols + v_cols]
-        num_pages, _, page, width = plane.shape
         cos_sin = None
         if self.position is not None:
             cos_sin = self.position.cos_sin(ctx)
@@ -126,17 +132,30 @@ class GroupedAttention(ProjectedMixer):
         q_rows = rows[:, : self.q_cols]
         if self.taps is not None:
             q_rows = torch.empty((tokens, self.q_cols), dtype=rows.dtype, device=rows.device)
-        K.attention_prepare(rows, q_rows, cos_sin, ctx, table, plane, q_heads=heads, k_heads=self.num_kv_heads,
+        planes = len(cache.planes) == 2                        # [pages, kv heads, page, dim] each
+        keys, values = (cache.k, cache.v) if planes else (cache.planes[0], None)
+        K.attention_prepare(rows, q_rows, cos_sin, ctx, table, (keys, values) if planes else keys, q_heads=heads, k_heads=self.num_kv_heads,
                             dim=self.head_dim, value_width=self.v_cols, taps=self.taps,
                             state=cache.state if self.conv_taps > 1 else None, state_offset=self.state_offset,
                             q_weight=self.q_norm_weight, k_weight=self.k_norm_weight, eps=self.eps, write=cache.owner)
-        direct = out.unflatten(1, (heads, self.value_dim))
-        o = K.attention_dims(
-            q_rows.unflatten(1, (heads, self.head_dim)), plane, plane.view(-1)[self.k_cols:], table, ctx,
-            value_heads=self.num_kv_heads, group=heads // self.num_kv_heads, maps=1, key_width=self.head_dim,
-            value_width=self.value_dim, page_size=page, num_pages=num_pages,
-            key_strides=(page * width, self.head_dim, width), value_strides=(page * width, self.value_dim, width),
-            scale=self.scale, sink=self.sink, softcap=self.softcap, out=None if self.has_gate else direct)
+        num_pages, _, page, width = keys.shape
+        if planes and K.paged_attention_takes_sinks(rows.dtype, self.head_dim, page) and out.stride(0) % 8 == 0:
+            o = K.paged_attention(q_rows, keys, values, table, ctx, heads, self.num_kv_heads, self.head_dim, self.scale, None,
+                                  sink=self.sink, softcap=self.softcap, out=None if self.has_gate else out)
+            o = o.unflatten(1, (heads, self.value_dim))
+        else:
+            if planes:
+                key_strides = value_strides = (self.num_kv_heads * page * width, page * width, width)
+            else:
+                values = keys.view(-1)[self.k_cols:]
+                key_strides = (page * width, self.head_dim, width)
+                value_strides = (page * width, self.value_dim, width)
+            direct = out.unflatten(1, (heads, self.value_dim))
+            o = K.attention_dims(
+                q_rows.unflatten(1, (heads, self.head_dim)), keys, values, table, ctx, value_heads=self.num_kv_heads,
+                group=heads // self.num_kv_heads, maps=1, key_width=self.head_dim, value_width=self.value_dim,
+                page_size=page, num_pages=num_pages, key_strides=key_strides, value_strides=value_strides,
+                scale=self.scale, sink=self.sink, softcap=self.softcap, out=None if self.has_gate else direct)
         if self.has_gate:
             gate = rows[:, self.g_col:self.g_col + self.out_cols]
             if out.is_contiguous():

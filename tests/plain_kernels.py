@@ -117,16 +117,17 @@ def rope_kv_write(qkv, positions, req_index, cos_sin, table, k_cache, v_cache,
 
 def paged_attention(qkv, k_cache, v_cache, table, ctx, num_heads, num_kv_heads, head_dim, scale, window,
                     *, force_general=False, num_splits=None, use_tma=True, use_tc5=True, cos_sin=None,
-                    write_kv=None, keep_first=0):
+                    write_kv=None, keep_first=0, sink=None, softcap=None, out=None):
     if write_kv is not None:   # the call also rotates q, k and writes this step's k, v
         rope_kv_write(qkv, ctx.positions, ctx.req_index, cos_sin, table, k_cache, v_cache,
                       num_heads, num_kv_heads, head_dim, write_kv=write_kv)
-    return paged_attention_plain(qkv, k_cache, v_cache, table, ctx.positions, ctx.req_index,
-                                 num_heads, num_kv_heads, head_dim, scale, window, keep_first)
+    y = paged_attention_plain(qkv, k_cache, v_cache, table, ctx.positions, ctx.req_index,
+                              num_heads, num_kv_heads, head_dim, scale, window, keep_first, sink, softcap)
+    return y if out is None else out.copy_(y)
 
 
 def paged_attention_plain(qkv, k_cache, v_cache, table, positions, req_index,
-                          num_heads, num_kv_heads, head_dim, scale, window, keep_first=0):
+                          num_heads, num_kv_heads, head_dim, scale, window, keep_first=0, sink=None, softcap=None):
     tokens = qkv.shape[0]
     page_size = k_cache.shape[2]
     group = num_heads // num_kv_heads
@@ -146,7 +147,11 @@ def paged_attention_plain(qkv, k_cache, v_cache, table, positions, req_index,
         for h in range(num_heads):
             g = h // group
             scores = (k[:, g, :] @ q[t, h]) * scale
-            probs = torch.softmax(scores, dim=0)
+            if softcap is not None:
+                scores = softcap * torch.tanh(scores / softcap)
+            if sink is not None:                    # one more entry of the softmax, without a value
+                scores = torch.cat([scores, sink[h:h + 1].float()])
+            probs = torch.softmax(scores, dim=0)[:len(keys)]
             out[t, h * head_dim:(h + 1) * head_dim] = (probs @ v[:, g, :]).to(qkv.dtype)
     return out
 
@@ -724,7 +729,7 @@ def retention_scan(q, k, v, cos_sin, decay, state, ctx, *, heads, dim, value_dim
 
 def attention_prepare(rows, q_out, cos_sin, ctx, table, cache, *, q_heads, k_heads, dim, value_width, taps=None, state=None,
                       state_offset=0, q_weight=None, k_weight=None, eps=0.0, write=True):
-    tokens, page_size = rows.shape[0], cache.shape[2]
+    tokens, page_size = rows.shape[0], (cache[0] if isinstance(cache, tuple) else cache).shape[2]
     q_len, k_len = q_heads * dim, k_heads * dim
     channels = q_len + k_len + value_width
     x = rows[:, :channels].float()
@@ -753,6 +758,10 @@ def attention_prepare(rows, q_out, cos_sin, ctx, table, cache, *, q_heads, k_hea
         pos = int(ctx.positions[t])
         page = int(table[int(ctx.req_index[t]), pos // page_size])
         assert page > 0, "write through the null page"
+        if isinstance(cache, tuple):
+            cache[0][page, :, pos % page_size] = k[t].reshape(k_heads, dim)
+            cache[1][page, :, pos % page_size] = v[t].reshape(k_heads, -1)
+            continue
         cache[page, 0, pos % page_size, :k_len] = k[t]
         cache[page, 0, pos % page_size, k_len:] = v[t]
 

@@ -75,8 +75,15 @@ CONFIGS = {
           mlp=P.moe(experts=8, top=2, ff=32, identity=2)),
         C(heads=8, kv_heads=2, dim=48, vdim=32, rot=rot(16, 5000.0), softcap=4.0, mlp=P.moe(experts=16, top=4, ff=16, identity=1)),
     ], vocab=128, width=64, loop=(1, 3, 2), eps=1e-5, scale=2.0),
+    # heads of the width that the TMA decode and the tcgen05 prompt kernels are made for, keys and values in planes of their
+    # own: a convolution and a gate, capped scores and sinks, and a loop over both
+    "wide_heads": P.model_config([
+        A(heads=4, kv_heads=2, dim=128, vdim=128, conv=4, rot=rot(64, 10000.0, (4.0, 1.0, 4.0, 64)), mlp=P.dense(48)),
+        C(heads=6, kv_heads=2, dim=128, vdim=128, rot=rot(128, 3000.0), softcap=3.0, mlp=P.moe(experts=4, top=2, ff=24, identity=1)),
+    ], vocab=96, width=64, loop=(0, 2, 2), eps=1e-5),
 }
-LENGTHS = {"all_kinds": (1, 23, 45, 70, 37, 2), "coincide": (64, 1, 30, 50), "serving_sizes": (150, 3, 97, 61)}
+LENGTHS = {"all_kinds": (1, 23, 45, 70, 37, 2), "coincide": (64, 1, 30, 50), "serving_sizes": (150, 3, 97, 61),
+           "wide_heads": (140, 1, 33, 70)}
 
 
 def write_folder(folder, cfg, seed, weights=None):
@@ -229,6 +236,30 @@ def test_cache_groups_and_state():
         None, (memory,), (conv,), (memory,), (conv,), (short,), (last,)]
 
 
+def test_where_keys_and_values_lie():
+    """Side by side in one row a token, or in two planes where the kernels that read planes take the heads."""
+    from kvcore_b200.parts.model import build_model
+
+    spec = model_spec_from_config(CONFIGS["wide_heads"])
+    for dtype, want in ((torch.bfloat16, (2, 2, 128)), (torch.float32, (1, 1, 512))):
+        caches = [r.cache_spec for r in build_model(spec, dtype=dtype, device="meta").entry_requirements()]
+        assert [(c.planes, c.heads, c.width) for c in caches] == [want] * 4
+
+
+@pytest.mark.parametrize("page_size", [4, 8, 12, 64])
+def test_planes_under_other_page_sizes(page_size, device, tmp_path):
+    """Pages that the kernels for planes do not take are read by strides."""
+    cfg = CONFIGS["wide_heads"]
+    folder = tmp_path / "m"
+    weights = write_folder(folder, cfg, seed=31)
+    requests = {f"q{i}": rc.random_tokens(cfg["vocab"], n, 40 + i) for i, n in enumerate((37, 2, 70) if device != "cpu" else (20, 2))}
+    reference, margins = references(cfg, weights, requests)
+    steps = rc.trace_mixed(requests, max_live=3, seed=4)
+    out = tmp_path / "o"
+    rc.run_inprocess(folder, "bfloat16", steps, out, rc.peak_tokens(steps, page=192), device=device, page_size=page_size, fill_freed_pages="poison")
+    compare(rc.collect(steps, out, cfg["vocab"]), reference, "bfloat16", margins)
+
+
 def test_unused_tensors_of_a_checkpoint_are_accepted(device, tmp_path):
     """A layer without a feed-forward may carry the norms around one."""
     from kvcore_b200.engine.trace_replay import build_replay
@@ -376,25 +407,26 @@ def _bare_model(layer, seed):
     return cfg, w
 
 
-def _standout_model(kind):
+def _standout_model(kind, dim=16):
     """Attention in which the query of token 2 meets the key of token 1 in a score that takes the whole softmax, along an
     entry that does not turn."""
     if kind == "attention":
-        cfg, w = _bare_model(A(heads=2, kv_heads=1, dim=16, vdim=20, conv=3, rot=rot(8, 100.0), scale=0.5), 3)
+        cfg, w = _bare_model(A(heads=2, kv_heads=1, dim=dim, vdim=dim if dim > 16 else 20, conv=3, rot=rot(8, 100.0), scale=0.5), 3)
         for n in "qkv":
             w[f"l0.mix.{n}.conv"][:, -1] = 1.0
     else:
-        cfg, w = _bare_model(C(heads=2, kv_heads=1, dim=16, vdim=20, rot=rot(8, 100.0), softcap=9.0, scale=1.0), 3)
+        cfg, w = _bare_model(C(heads=2, kv_heads=1, dim=dim, vdim=dim if dim > 16 else 20, rot=rot(8, 100.0), softcap=9.0,
+                               scale=16.0 / dim), 3)
         w["l0.mix.sink"] = torch.tensor([1.0, -1.0])
     w["l0.mix.q"][12, 1], w["l0.mix.k"][12, 0] = 4.0, 4.0      # entry 12 of head 0
     return cfg, w
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("kind", ["attention", "attention_2"])
-def test_a_key_that_stands_out(kind, dtype, device, tmp_path):
+@pytest.mark.parametrize("kind,dim", [("attention", 16), ("attention_2", 16), ("attention", 128), ("attention_2", 128)])
+def test_a_key_that_stands_out(kind, dim, dtype, device, tmp_path):
     """A dominating key far back, right in front, at page borders and at the first position, in prompts and decoded."""
-    cfg, w = _standout_model(kind)
+    cfg, w = _standout_model(kind, dim)
     folder = tmp_path / "m"
     weights = write_folder(folder, cfg, 0, w)
     requests = {}

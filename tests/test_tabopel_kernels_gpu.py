@@ -24,7 +24,7 @@ def close(dtype):
 
 # ---- between the projections and the attention -------------------------------------------------------------
 #  q heads, k heads, dim, value entries, turned entries
-PREPARE_SIZES = [(4, 2, 16, 24, 16), (3, 1, 20, 14, 6), (6, 3, 24, 36, 0), (2, 2, 10, 7, 10), (8, 4, 64, 128, 32),
+PREPARE_SIZES = [(4, 2, 16, 24, 16), (3, 1, 20, 14, 6), (6, 3, 24, 36, 0), (2, 2, 10, 14, 10), (8, 4, 64, 128, 32),
                  (24, 6, 128, 96, 128), (40, 8, 128, 1024, 64), (2, 1, 40, 8, 24), (5, 5, 9, 10, 4), (16, 2, 256, 512, 256)]
 PREPARE_LENS = [(0, 1), (5, 19), (0, 2), (11, 37)]
 
@@ -79,6 +79,28 @@ def test_attention_prepare(sizes, dtype, taps, norm, lens):
         assert K().read_status() == 0
         if taps < 2:
             break
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("taps,norm", [(0, True), (0, False), (4, False), (3, True), (11, False)])
+@pytest.mark.parametrize("sizes", [(4, 2, 16, 24, 8), (6, 3, 24, 30, 24), (8, 2, 128, 256, 64), (5, 5, 9, 10, 4)])
+def test_keys_and_values_in_planes_of_their_own(sizes, taps, norm, dtype):
+    H, G, D, V, _ = sizes
+    c = _prepare_case(sizes, PREPARE_LENS, dtype, 23, taps=taps, norm=norm)
+    pages, page = c["cache"].shape[0], c["cache"].shape[2]
+    state, _ = _states(6, c["channels"] * max(0, taps - 1) + 4, seed=2)
+    rows_state = state.clone()
+    planes = (torch.zeros(pages, G, page, D, dtype=dtype, device=DEV), torch.zeros(pages, G, page, V // G, dtype=dtype, device=DEV))
+    cache = torch.zeros_like(c["cache"])
+    q = _run_prepare(K(), c, c["rows"], planes, state, c["batch"], c["table"])
+    q_rows = _run_prepare(K(), c, c["rows"], cache, rows_state, c["batch"], c["table"])
+    assert torch.equal(q, q_rows) and torch.equal(state, rows_state)
+    assert torch.equal(planes[0], cache[:, 0, :, :G * D].reshape(pages, page, G, D).transpose(1, 2))
+    assert torch.equal(planes[1], cache[:, 0, :, G * D:].reshape(pages, page, G, V // G).transpose(1, 2))
+    host = (torch.zeros(planes[0].shape, dtype=dtype), torch.zeros(planes[1].shape, dtype=dtype))
+    _run_prepare(P, c, c["rows"].cpu(), host, _states(6, c["channels"] * max(0, taps - 1) + 4, seed=2)[1], c["host"], c["table"].cpu())
+    for got, want in zip(planes, host):
+        torch.testing.assert_close(got.cpu(), want, **close(dtype))
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -171,6 +193,80 @@ def test_attention_with_capped_scores(dtype, heads, kv_heads, dim, vdim, page, l
     if dtype == torch.bfloat16 and batch.max_query_len == 1:
         for splits in (1, 3):
             torch.testing.assert_close(run(num_splits=splits).cpu(), want, **bound)
+
+
+# heads, kv heads, page, requests (cached, new, longest portion first), cap, sink, splits
+PLANE_CASES = [
+    (8, 2, 16, [(0, 300), (130, 140), (5, 40)], 2.0, True, None),              # prompts on tcgen05
+    (8, 2, 16, [(0, 129)], None, True, None),
+    (6, 2, 8, [(37, 200)], 30.0, False, None),                                  # three heads a key head: queries copied by rows
+    (16, 1, 32, [(0, 40), (77, 9)], 4.0, True, None),
+    (8, 2, 16, [(640, 1), (1000, 1), (3, 1), (0, 1)], 2.5, True, None),         # decoded
+    (8, 2, 16, [(640, 1), (1000, 1), (3, 1)], None, True, 3),
+    (8, 2, 16, [(640, 1), (1000, 1), (3, 1)], 1.0, True, 5),
+    (8, 8, 64, [(300, 1)] * 40, 6.0, False, None),                              # more items than blocks fit at once
+    (8, 2, 16, [(0, 300), (40, 9), (90, 1), (200, 1), (7, 1)], 3.0, True, None),  # portions beside single tokens
+]
+
+
+@pytest.mark.parametrize("heads,kv_heads,page,lens,cap,sink,splits", PLANE_CASES)
+def test_attention_over_planes_with_sinks_and_capped_scores(heads, kv_heads, page, lens, cap, sink, splits):
+    dim, dtype = 128, torch.bfloat16
+    case = _cache_case(dtype, heads, kv_heads, dim, page, lens, seed=5)
+    batch = _Batch(lens)
+    q = randn(batch.num_tokens, heads * dim, dtype=dtype, seed=6, scale=2.0)     # scores far beyond the smaller caps
+    sinks = randn(heads, dtype=torch.float32, seed=7, scale=3.0) if sink else None
+    args = (heads, kv_heads, dim, dim ** -0.5, None)
+    host = (q.cpu(), case["k_cache"].cpu(), case["v_cache"].cpu(), case["table"].cpu(), batch.positions.cpu(), batch.req_index.cpu(), *args)
+    host_sinks = None if sinks is None else sinks.cpu()
+    want = P.paged_attention_plain(*host, sink=host_sinks, softcap=cap)
+    assert (want - P.paged_attention_plain(*host)).abs().max() > 0.05, "neither moves anything in this case"
+    out = torch.zeros(batch.num_tokens, heads * dim + 8, dtype=dtype, device=DEV)
+    got = K().paged_attention(q, case["k_cache"], case["v_cache"], case["table"], batch, *args, sink=sinks, softcap=cap,
+                              num_splits=splits, out=out[:, :heads * dim])
+    assert K().read_status() == 0 and not out[:, heads * dim:].any()
+    torch.testing.assert_close(got.cpu(), want, rtol=2e-2, atol=2e-2)
+    # the same through the kernels that address any cache by strides
+    strides = (kv_heads * page * dim, page * dim, dim)
+    other = K().attention_dims(q.view(-1, heads, dim), case["k_cache"], case["v_cache"], case["table"], batch, value_heads=kv_heads,
+                               group=heads // kv_heads, maps=1, key_width=dim, value_width=dim, page_size=page,
+                               num_pages=case["k_cache"].shape[0], key_strides=strides, value_strides=strides, scale=dim ** -0.5,
+                               sink=sinks, softcap=cap)
+    torch.testing.assert_close(other.reshape(-1, heads * dim).cpu(), want, rtol=2e-2, atol=2e-2)
+
+
+@pytest.mark.parametrize("lens,splits", [((200, 1), None), ((200, 1), 3), ((0, 201), None), ((150, 51), None)])
+@pytest.mark.parametrize("place", [0, 15, 16, 127, 128, 180])
+@pytest.mark.parametrize("cap", [3.0, 25.0])
+def test_a_far_key_among_planes_keeps_the_weight_that_the_cap_leaves_it(cap, place, lens, splits):
+    """As below, on the TMA decode and the tcgen05 kernel: exp(cap) against the sink's exp(1.5) and one for every other key."""
+    heads, kv_heads, dim, page = 4, 2, 128, 16
+    case = _cache_case(torch.bfloat16, heads, kv_heads, dim, page, [lens], seed=3)
+    keys, values, batch = case["k_cache"].zero_(), case["v_cache"].zero_(), _Batch([lens])
+    q = torch.zeros(batch.num_tokens, heads * dim, dtype=torch.bfloat16, device=DEV)
+    q.view(-1, heads, dim)[:, :, 3] = 200.0
+    at = case["table"][0, place // page]
+    keys[at, :, place % page, 3], values[at, :, place % page] = 100.0, 1.0
+    sinks = torch.full((heads,), 1.5, dtype=torch.float32, device=DEV)
+    out = K().paged_attention(q, keys, values, case["table"], batch, heads, kv_heads, dim, 1.0, None, sink=sinks, softcap=cap, num_splits=splits)
+    e = torch.tensor([cap, 1.5], dtype=torch.float64).exp()
+    want = e[0] / (e[0] + e[1] + sum(lens) - 1)
+    torch.testing.assert_close(out[-1].cpu().double(), want.expand(heads * dim), rtol=8e-3, atol=0.0)
+    assert K().read_status() == 0
+
+
+def test_a_sink_that_dominates_or_vanishes_among_planes():
+    """A sink far above every score leaves nothing; far below, the ordinary softmax, bit for bit within rounding."""
+    heads, kv_heads, dim, page = 4, 2, 128, 16
+    for lens in ([(0, 150)], [(150, 1)]):
+        case = _cache_case(torch.bfloat16, heads, kv_heads, dim, page, lens, seed=9)
+        batch = _Batch(lens)
+        q = randn(batch.num_tokens, heads * dim, dtype=torch.bfloat16, seed=10)
+        run = lambda sinks: K().paged_attention(q, case["k_cache"], case["v_cache"], case["table"], batch, heads, kv_heads, dim,
+                                                dim ** -0.5, None, sink=sinks)
+        free = run(None)
+        assert run(torch.full((heads,), 80.0, device=DEV)).abs().max() < 1e-20
+        torch.testing.assert_close(run(torch.full((heads,), -80.0, device=DEV)), free, rtol=1e-2, atol=1e-3)
 
 
 @pytest.mark.parametrize("dtype,dim,lens", [(torch.float32, 16, (60, 1)), (torch.bfloat16, 64, (200, 1)), (torch.bfloat16, 64, (0, 201))])
@@ -459,6 +555,10 @@ def test_wrappers_refuse_what_does_not_fit():
     with pytest.raises(kernels.KernelError, match="cap"):
         K().attention_dims(x.view(2, 2, 8), cache, cache, table, batch, value_heads=1, group=2, maps=1, key_width=8, value_width=8,
                            page_size=4, num_pages=2, key_strides=(32, 0, 8), value_strides=(32, 0, 8), scale=1.0, softcap=0.0)
+    q = randn(2, 64, dtype=torch.bfloat16, seed=1)
+    planes = torch.zeros(2, 1, 16, 32, dtype=torch.bfloat16, device=DEV)
+    with pytest.raises(kernels.KernelError, match="sinks and capped scores"):
+        K().paged_attention(q, planes, planes, table, batch, 2, 1, 32, 1.0, None, softcap=5.0)
     with pytest.raises(kernels.KernelError, match="activation"):
         K().moe_experts(x, torch.zeros(2, 1, dtype=torch.int32, device=DEV), torch.ones(2, 1, device=DEV),
                         randn(1, 8, 16, dtype=torch.float32), randn(1, 16, 8, dtype=torch.float32), weight_on_input=False,
