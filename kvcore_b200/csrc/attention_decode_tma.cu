@@ -131,7 +131,8 @@ __device__ __forceinline__ TdStageHeader td_describe_item(const DecodeParams& p,
   return h;
 }
 
-template <int D>
+// BOUNDED: with sinks or capped scores
+template <int D, bool BOUNDED>
 __global__ void __launch_bounds__(TD_THREADS, 2)
 flash_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                         const DecodeParams p) {
@@ -401,7 +402,7 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
       row_max[hh] = -INFINITY;
       row_sum[hh] = 0.0f;
       // the sink joins the denominator once: in the first split's first warp (a row's sum is spread over a quad)
-      if (p.sink != nullptr && split == 0 && warp == 0 && row_valid[hh]) {
+      if (BOUNDED && p.sink != nullptr && split == 0 && warp == 0 && row_valid[hh]) {
         row_max[hh] = p.sink[kvh * p.G + r % p.G] * 1.4426950408889634f;
         row_sum[hh] = (lane & 3) == 0 ? 1.0f : 0.0f;
       }
@@ -469,7 +470,8 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           s[j][e] += s2[j][e];
-          s[j][e] = p.cap_out > 0.0f ? kvb_capped_score(s[j][e] * p.cap_in, p.cap_out) : s[j][e] * p.scale_log2;
+          if (BOUNDED && p.cap_out > 0.0f) s[j][e] = kvb_capped_score(s[j][e] * p.cap_in, p.cap_out);
+          else if (BOUNDED) s[j][e] *= p.scale_log2;
         }
       float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -480,7 +482,7 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
           const int key = (tile_begin + it) * TD_KEYS + wkey + j * 8 + (lane & 3) * 2 + (e & 1);
           const bool seen = row_valid[hh] && key >= key_lo && key < key_hi && key <= row_pos[hh] &&
                             (p.window <= 0 || key > row_pos[hh] - p.window);
-          const float v = seen ? s[j][e] : -INFINITY;
+          const float v = seen ? (BOUNDED ? s[j][e] : s[j][e] * p.scale_log2) : -INFINITY;
           s[j][e] = v;
           tile_max[hh] = fmaxf(tile_max[hh], v);
         }
@@ -672,7 +674,7 @@ extern "C" int kvb_make_kv_tensor_map(void* map_out, const void* cache, long lon
   return 0;
 }
 
-template <int D>
+template <int D, bool BOUNDED>
 static int launch_decode_tma(const CUtensorMap& k_map, const CUtensorMap& v_map, const DecodeParams& p,
                              int max_rows, int blocks, cudaStream_t stream) {
   constexpr size_t SMEM = 1024 + TD_STAGES * 2 * TD_KEYS * D * 2 + 16 * (D + 8) * 2 +
@@ -680,12 +682,12 @@ static int launch_decode_tma(const CUtensorMap& k_map, const CUtensorMap& v_map,
                           TD_STAGES * sizeof(TdStageHeader) + 2 * TD_STAGES * 8 + 16;
   static bool configured = false;
   if (!configured) {
-    KVB_CHECK_CUDA(cudaFuncSetAttribute(flash_decode_tma_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    KVB_CHECK_CUDA(cudaFuncSetAttribute(flash_decode_tma_kernel<D, BOUNDED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                         (int)SMEM));
     configured = true;
   }
   dim3 grid(blocks);
-  KVB_CHECK_CUDA(kvb_launch((flash_decode_tma_kernel<D>), dim3(grid), dim3(TD_THREADS), SMEM, stream, true, k_map, v_map, p));
+  KVB_CHECK_CUDA(kvb_launch((flash_decode_tma_kernel<D, BOUNDED>), dim3(grid), dim3(TD_THREADS), SMEM, stream, true, k_map, v_map, p));
   KVB_CHECK_LAUNCH();
   if (p.num_splits > 1) {
     const int rows = max_rows < 16 ? max_rows : 16;
@@ -749,8 +751,11 @@ extern "C" int kvb_flash_decode_tma(void* out, long long out_stride, const void*
   const bool shared = work != nullptr && max_blocks > 0 && p.total_items > max_blocks;
   p.work = shared ? work : nullptr;
   const int blocks = shared ? max_blocks : p.total_items;
-  if (D == 64) return launch_decode_tma<64>(k_map, v_map, p, max_rows, blocks, stream);
-  return launch_decode_tma<128>(k_map, v_map, p, max_rows, blocks, stream);
+  if (sink != nullptr || cap > 0.0f)
+    return D == 64 ? launch_decode_tma<64, true>(k_map, v_map, p, max_rows, blocks, stream)
+                   : launch_decode_tma<128, true>(k_map, v_map, p, max_rows, blocks, stream);
+  return D == 64 ? launch_decode_tma<64, false>(k_map, v_map, p, max_rows, blocks, stream)
+                 : launch_decode_tma<128, false>(k_map, v_map, p, max_rows, blocks, stream);
 }
 
 KVB_TRACE_TU(attention_decode_tma)
