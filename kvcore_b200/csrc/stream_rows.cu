@@ -40,13 +40,30 @@ struct AddRowsParams {
   int width;
 };
 
-// THREADS a block, by the width alone (so are the sums): a wide row with a norm behind the sub-layer has two sums in a
-// chain, which more threads with fewer pieces each shorten
+// With a norm behind the sub-layer (AFTER) a row has two sums in a chain, which more threads with fewer pieces each
+// shorten where there are few rows; many rows run better in blocks of 256.  So that a row's bits are the same either way,
+// its sums are taken as if 1,024 threads had a piece each: one butterfly for every 32 of those, then one over the 32.
+#define SR_VIRTUAL 1024
+template <int THREADS, int PIECES>
+__device__ __forceinline__ float virtual_sum(const float (&part)[PIECES], float* scratch) {
+  static_assert(THREADS * PIECES == SR_VIRTUAL, "a thread stands for PIECES virtual ones");
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float sums[PIECES];
+#pragma unroll
+  for (int s = 0; s < PIECES; ++s) sums[s] = warp_sum(part[s]);
+  __syncthreads();
+  if (lane == 0)
+#pragma unroll
+    for (int s = 0; s < PIECES; ++s) scratch[s * (THREADS / 32) + warp] = sums[s];
+  __syncthreads();
+  return warp_sum(scratch[lane]);
+}
+
 template <typename T, typename OUT, typename W, int N, bool AFTER, int THREADS>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(THREADS, AFTER && THREADS == 256 ? 3 : 1)
 stream_add_rows_kernel(const AddRowsParams p) {
   KVB_KERNEL_PROLOGUE(KVB_TAG_ADD_ROWS);
-  constexpr int PIECES = THREADS > SR_THREADS ? 1 : SR_PIECES;
+  constexpr int PIECES = AFTER ? SR_VIRTUAL / THREADS : SR_PIECES;
   __shared__ float scratch[32];
   const int n = blockIdx.x, t = p.token_rows != nullptr ? p.token_rows[n] : n;
   const int width = p.width;
@@ -76,6 +93,9 @@ stream_add_rows_kernel(const AddRowsParams p) {
   };
   float kept[PIECES][N];
   float ss = 0.0f, inv_a = 1.0f;
+  float parts[PIECES];                               // AFTER: the squares' sums of the virtual threads
+#pragma unroll
+  for (int s = 0; s < PIECES; ++s) parts[s] = 0.0f;
   // the new stream from what is added
   auto join = [&](int i, const RowPiece<float, N>& s, const RowPiece<W, N>& g, float (&v)[N]) {
     if (AFTER) {
@@ -113,8 +133,10 @@ stream_add_rows_kernel(const AddRowsParams p) {
       *reinterpret_cast<RowPiece<OUT, N>*>(dst) = now;
       *reinterpret_cast<RowPiece<OUT, N>*>(dst + width) = start;
     }
+  };
+  auto squares = [&](const float (&v)[N], float& sum) {
 #pragma unroll
-    for (int j = 0; j < N; ++j) ss = fmaf(v[j], v[j], ss);
+    for (int j = 0; j < N; ++j) sum = fmaf(v[j], v[j], sum);
   };
   // the kept pieces: the stream's, the weights' and a slot's loads are each in flight together
   RowPiece<float, N> xs[PIECES];
@@ -151,19 +173,21 @@ stream_add_rows_kernel(const AddRowsParams p) {
     }
   }
   const int rest = (threadIdx.x + PIECES * THREADS) * N;
-  if (AFTER) {                                       // the root mean square of what is added
-    float sa = 0.0f;
+  if constexpr (AFTER) {                             // the root mean square of what is added
+    float sa[PIECES];
 #pragma unroll
-    for (int s = 0; s < PIECES; ++s)              // (pieces beyond the width are zeros)
-#pragma unroll
-      for (int j = 0; j < N; ++j) sa = fmaf(kept[s][j], kept[s][j], sa);
-    for (int i = rest; i < width; i += THREADS * N) {
+    for (int s = 0; s < PIECES; ++s) {               // (pieces beyond the width are zeros)
+      sa[s] = 0.0f;
+      squares(kept[s], sa[s]);
+    }
+    for (int i = rest, s = 0; i < width; i += THREADS * N, s = s + 1 < PIECES ? s + 1 : 0) {
       float a[N];
       added(i, a);
 #pragma unroll
-      for (int j = 0; j < N; ++j) sa = fmaf(a[j], a[j], sa);
+      for (int k = 0; k < PIECES; ++k)               // (an array indexed by a variable would leave the registers)
+        if (k == s) squares(a, sa[k]);
     }
-    inv_a = 1.0f / sqrtf(block_sum(sa, scratch) / (float)width + p.after_eps);
+    inv_a = 1.0f / sqrtf(virtual_sum<THREADS, PIECES>(sa, scratch) / (float)width + p.after_eps);
   }
 #pragma unroll
   for (int s = 0; s < PIECES; ++s) {
@@ -171,16 +195,27 @@ stream_add_rows_kernel(const AddRowsParams p) {
     if (i < width) {
       join(i, xs[s], gs[AFTER ? s : 0], kept[s]);
       first_pass(i, kept[s]);
+      squares(kept[s], AFTER ? parts[s] : ss);
     }
   }
   // rows wider than the registers hold: the sum goes through `stream`, which the same thread reads again
-  for (int i = rest; i < width; i += THREADS * N) {
+  for (int i = rest, s = 0; i < width; i += THREADS * N, s = s + 1 < PIECES ? s + 1 : 0) {
     float v[N];
     summed(i, v);
     first_pass(i, v);
+    if (AFTER) {
+#pragma unroll
+      for (int k = 0; k < PIECES; ++k)
+        if (k == s) squares(v, parts[k]);
+    } else {
+      squares(v, ss);
+    }
   }
   if (p.normed == nullptr) return;
-  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + p.eps);
+  float total;
+  if constexpr (AFTER) total = virtual_sum<THREADS, PIECES>(parts, scratch);
+  else total = block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(total / (float)width + p.eps);
   const W* weight = (const W*)p.weight;
   OUT* dst = (OUT*)p.normed + (size_t)n * width;
   auto put = [&](int i, const float (&v)[N], const RowPiece<W, N>& w) {
@@ -235,11 +270,14 @@ extern "C" int kvb_stream_add_rows(const float* x, const void* rows, int top, co
   cudaError_t err;
 #define KVB_AR_SHAPE(T, OUT, W, N, A, TH) \
   kvb_launch((stream_add_rows_kernel<T, OUT, W, N, A, TH>), dim3(count), dim3(TH), 0, cuda_stream, true, p)
+  // few rows: as many threads as a row has pieces (the bits of a row are the same for each number of them)
+  const int few = kvb_sm_count() > 0 ? 2 * kvb_sm_count() : 256;
+  const int threads = !quads || count > few || width <= 1024 ? 256 : width <= 2048 ? 512 : 1024;
 #define KVB_AR(T, OUT, W)                                                                                        \
   err = after == nullptr ? (quads ? KVB_AR_SHAPE(T, OUT, W, 4, false, 256) : KVB_AR_SHAPE(T, OUT, W, 1, false, 256)) \
         : !quads         ? KVB_AR_SHAPE(T, OUT, W, 1, true, 256)                                                  \
-        : width <= 1024  ? KVB_AR_SHAPE(T, OUT, W, 4, true, 256)                                                  \
-        : width <= 2048  ? KVB_AR_SHAPE(T, OUT, W, 4, true, 512)                                                  \
+        : threads == 256 ? KVB_AR_SHAPE(T, OUT, W, 4, true, 256)                                                  \
+        : threads == 512 ? KVB_AR_SHAPE(T, OUT, W, 4, true, 512)                                                  \
                          : KVB_AR_SHAPE(T, OUT, W, 4, true, 1024)
   const int code = (dtype == KVB_BF16 ? 4 : 0) | (out_dtype == KVB_BF16 ? 2 : 0) | (weight_dtype == KVB_BF16 ? 1 : 0);
   switch (code) {

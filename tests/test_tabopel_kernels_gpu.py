@@ -418,6 +418,20 @@ def test_norm_sum_step_and_norm(width, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("width", [1000, 1028, 2048, 4096, 9000])
+def test_a_row_under_a_norm_has_the_same_bits_in_a_long_batch(width, dtype):
+    """Few rows take more threads each than many rows do; the sums are the same."""
+    x, a = randn(900, width, dtype=torch.float32, seed=71), randn(900, width, dtype=dtype, seed=72, scale=3.0)
+    behind, front = (randn(width, dtype=dtype, seed=73 + n) + 1.0 for n in range(2))
+    stream, y, _ = K().stream_add_rows(x.clone(), a, weight=front, eps=1e-5, after=(behind, 1e-3))
+    few, y_few, _ = K().stream_add_rows(x[400:408].clone(), a[400:408].clone(), weight=front, eps=1e-5, after=(behind, 1e-3))
+    assert torch.equal(few, stream[400:408]) and torch.equal(y_few, y[400:408])
+    want = P.stream_add_rows(x[400:408].cpu(), a[400:408].cpu(), weight=front.cpu(), eps=1e-5, after=(behind.cpu(), 1e-3))
+    torch.testing.assert_close(few.cpu(), want[0], **F32)
+    torch.testing.assert_close(y_few.cpu(), want[1], **close(dtype))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("width", [44, 777, 2000, 5000])
 def test_experts_rows_under_a_norm_with_pairs_that_have_none(width, dtype):
     """The rows of a token's experts, weighted or already weighted, some pairs with an expert that hands the token's own
